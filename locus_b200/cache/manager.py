@@ -4,10 +4,11 @@ group of layers with the same needs, and slots for per-request state of fixed si
 The reference keeps one geometry for all layers and one table per sequence
 (``PagedKvCache``, src/locus/kv/paged_cache.hpp:24-202; ``ensure_capacity`` all-or-nothing,
 paged_cache.cpp:62-77; ``release`` paged_cache.cpp:79-85).  Here layers are sorted into
-groups by what they keep -- all keys, or a window of them, of some (kv heads, head size) --
+groups by what they keep -- all keys, a window or a chunk of them, of some (kv heads, head size) --
 and every group has pages and a free list of its own; a request holds one table per group.
 Pages go back to their pool when the request is released and, in a window group, as soon
-as every position they hold has fallen out of the window.  A request also takes one state
+as every position they hold has fallen out of the window (in a group with chunks: out of the
+chunk that the next token lies in).  A request also takes one state
 slot when it is opened; layers with per-request state keep a tensor
 [n_state_slots, *shape] that the slot indexes.
 
@@ -139,8 +140,9 @@ class CacheManager:
         self.max_step_tokens = max(0, int(max_step_tokens))
         for g in self.groups:
             g.n_pages = n_pages
-            if g.spec.window > 0 and self.max_step_tokens > 0:
-                per_request = -(-(g.spec.window + self.max_step_tokens) // page_tokens) + 1 + -(-g.spec.keep_first // page_tokens)
+            reach = g.spec.window or g.spec.chunk
+            if reach > 0 and self.max_step_tokens > 0:
+                per_request = -(-(reach + self.max_step_tokens) // page_tokens) + 1 + -(-g.spec.keep_first // page_tokens)
                 g.n_pages = min(n_pages, n_state_slots * per_request)
         windows = (ctypes.c_int * max(1, len(self.groups)))(*[g.spec.window for g in self.groups])
         group_pages = (ctypes.c_int * max(1, len(self.groups)))(*[g.n_pages for g in self.groups])
@@ -151,6 +153,8 @@ class CacheManager:
         for g in self.groups:
             if g.spec.window > 0 and g.spec.keep_first > 0:
                 self._lib.locus_cache_set_keep(self._core, g.gid, g.spec.keep_first)
+            if g.spec.chunk > 0 and self._lib.locus_cache_set_aligned(self._core, g.gid, g.spec.chunk) != 0:
+                raise ValueError("a cache group has either a window or chunks, not both")
         assert self._lib.locus_cache_table_width(self._core) == self.table_width
         self.state_slots = _StateSlots(self)
         # (group, page) pairs that a commit or a release made free
@@ -296,7 +300,8 @@ class CacheManager:
     def commit(self, seq: SeqCache, n: int) -> None:
         """``n`` tokens were written after the cached ones.  Gives back window pages that no
         later query can see: a query at position p sees keys t > p - window, the next query
-        is at position n_tokens, so pages wholly below n_tokens - window + 1 are dead."""
+        is at position n_tokens, so pages wholly below n_tokens - window + 1 are dead (with chunks: those
+        below the start of the chunk that position n_tokens lies in)."""
         self._check_open(seq)
         r = self._lib.locus_cache_commit(self._core, seq._handle, int(n), self._freed, len(self._freed))
         if r == -3:

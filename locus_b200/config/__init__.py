@@ -4,3 +4,4 @@ from .qwen2_moe import Qwen2MoeConfig  # noqa: F401
 from .lalepel import LalepelConfig  # noqa: F401
 from .pozozen import PozozenConfig  # noqa: F401
 from .gugozen import GugozenConfig  # noqa: F401
+from .bebovik import BebovikConfig  # noqa: F401

@@ -7,7 +7,8 @@
 //             absolute positions, partial results merged in ascending order.
 //
 // Both read K and V through the request's block table, honour an optional window (a query
-// at position p sees keys t with p - window < t <= p; window 0 = all keys) and take any head
+// at position p sees keys t with p - window < t <= p; window 0 = all keys) or aligned chunks (a query
+// sees the keys of its own chunk of positions, mask.cuh), and take any head
 // size that is a multiple of 16 up to 256, any number of heads and any group ratio.
 // A window may keep a request's first tokens in sight (keep_first > 0: keys t < keep_first stay
 // visible to every later query, at their true positions), and the softmax may have a sink (sink != 0:
@@ -28,7 +29,7 @@ struct AttnArgs {
     int table_stride;
     const int* items;         // chunk: [n_items, 2] (segment, first query of the tile within it)
                               // decode: [n_items] segment ids
-    int nh, nkv, hd, page_tokens, window;
+    int nh, nkv, hd, page_tokens, window, chunk;
     int keep_first, sink;     // see the head of the file
     const float* sink_val;    // with sink: a learned score per query head in its place (null: the score 0)
     float scale;
@@ -80,6 +81,7 @@ __global__ void __launch_bounds__(128) attn_chunk_kernel(AttnArgs a) {
     float* m_s = sc + CHUNK_BQ * (CHUNK_TK + 1);   // [BQ]
     float* l_s = m_s + CHUNK_BQ;                   // [BQ]
     float* al_s = l_s + CHUNK_BQ;                  // [BQ]
+    __shared__ int lo_s[CHUNK_BQ];                 // first key that a query of the tile sees
 
     // the late tiles of a prompt see the most keys: the grid takes them first, for all heads (its fast index)
     const int item = gridDim.y - 1 - blockIdx.y;
@@ -100,9 +102,10 @@ __global__ void __launch_bounds__(128) attn_chunk_kernel(AttnArgs a) {
     if (tid < CHUNK_BQ) {
         m_s[tid] = -INFINITY;
         l_s[tid] = 0.f;
+        lo_s[tid] = first_key(a.window, a.chunk, p0 + tid);
     }
     const int t_hi = p0 + nq - 1;
-    const int t_lo = a.window > 0 ? max(0, p0 - a.window + 1) : 0;
+    const int t_lo = first_key(a.window, a.chunk, p0);
     const int nd = hd / 8;
     const int my_q = tid >> 3, dl = tid & 7;
     float acc[32];
@@ -135,7 +138,7 @@ __global__ void __launch_bounds__(128) attn_chunk_kernel(AttnArgs a) {
             const int qi = i / CHUNK_TK, kj = i % CHUNK_TK;
             const int t = tile0 + kj, p = p0 + qi;
             float s = -INFINITY;
-            if (qi < nq && t <= p && (a.window == 0 || t > p - a.window || t < a.keep_first)) {
+            if (qi < nq && t <= p && (t >= lo_s[qi] || t < a.keep_first)) {
                 float dot = 0.f;
                 const float* qr = qs + qi * hd;
                 const float* kr = ks + kj * (hd + 1);
@@ -240,7 +243,7 @@ __global__ void __launch_bounds__(128) attn_decode_split_kernel(AttnArgs a) {
     const int kvh = h / (a.nh / a.nkv);
     const int p = a.seg_ctx[seg];  // position of the single query
     const int row = a.seg_q0[seg];
-    const int t_lo = a.window > 0 ? max(0, p - a.window + 1) : 0;
+    const int t_lo = first_key(a.window, a.chunk, p);
     // splits in front of the window's that hold kept first tokens
     const int kept = a.window > 0 ? min(a.keep_first, t_lo) : 0;
     const int s0 = t_lo / DEC_SPLIT;
@@ -458,7 +461,7 @@ __global__ void __launch_bounds__(32 * DS_WARPS, DEEP ? 2 : 4) attn_decode_strea
     // The cut reads only the step's descriptors, which were on the device before the step's first kernel: under
     // programmatic dependent launch it is made while the kernel in front of this one (which writes q and the newest
     // keys and values) still runs; the wait for that kernel comes after it.
-    plan_key_ranges(kr, a.items, a.seg_ctx, a.seg_q0, a.window, n_items, a.nh, max_units, n_warps, cost_range, cost_merge,
+    plan_key_ranges(kr, a.items, a.seg_ctx, a.seg_q0, a.window, a.chunk, n_items, a.nh, max_units, n_warps, cost_range, cost_merge,
                     a.keep_first);
     bool waited = false;  // whether this warp has waited for the kernel in front (every path does before it leaves)
     int* const s_first = kr.first;
@@ -499,7 +502,7 @@ __global__ void __launch_bounds__(32 * DS_WARPS, DEEP ? 2 : 4) attn_decode_strea
         const int kept = kr.kept[item];
         const bool kept_range = kept > 0 && r == s_pref[item];
         const int split = r - s_pref[item] - (kept > 0);
-        const int t_lo = kept_range ? 0 : (a.window > 0 ? max(0, p - a.window + 1) : 0);
+        const int t_lo = kept_range ? 0 : first_key(a.window, a.chunk, p);
         const int k_begin = kept_range ? 0 : s_first[item] + split * len;  // a multiple of 32: chunks do not straddle pages
         const int k_end = kept_range ? kept : min(p + 1, k_begin + len);   // exclusive
         const int keep = a.keep_first;
@@ -772,22 +775,22 @@ extern "C" void locus_attn_decode_set_cost(int range_overhead, int merge_per_ran
     g_ds_cost_merge = merge_per_range;
 }
 
-static int check_common(int nh, int nkv, int hd, int page_tokens, int window, int keep_first = 0) {
-    if (nh <= 0 || nkv <= 0 || nh % nkv != 0 || keep_first < 0) return LOCUS_ERR_UNSUPPORTED;
+static int check_common(int nh, int nkv, int hd, int page_tokens, int window, int chunk, int keep_first = 0) {
+    if (nh <= 0 || nkv <= 0 || nh % nkv != 0 || !mask_ok(window, chunk, keep_first)) return LOCUS_ERR_UNSUPPORTED;
     if (hd <= 0 || hd % 16 != 0 || hd > 256) return LOCUS_ERR_UNSUPPORTED;
-    if (page_tokens <= 0 || window < 0) return LOCUS_ERR_UNSUPPORTED;
+    if (page_tokens <= 0) return LOCUS_ERR_UNSUPPORTED;
     return 0;
 }
 
 static AttnArgs make_args(const void* q, const void* pool, void* out, const int* seg_q0,
                           const int* seg_qn, const int* seg_ctx, const int* block_table,
                           int table_stride, const int* items, int nh, int nkv, int hd,
-                          int page_tokens, int window, float scale, int keep_first = 0, int sink = 0,
+                          int page_tokens, int window, int chunk, float scale, int keep_first = 0, int sink = 0,
                           const float* sink_val = nullptr) {
     AttnArgs a;
     a.q = q; a.pool = pool; a.out = out; a.seg_q0 = seg_q0; a.seg_qn = seg_qn; a.seg_ctx = seg_ctx;
     a.block_table = block_table; a.table_stride = table_stride; a.items = items; a.nh = nh;
-    a.nkv = nkv; a.hd = hd; a.page_tokens = page_tokens; a.window = window; a.scale = scale;
+    a.nkv = nkv; a.hd = hd; a.page_tokens = page_tokens; a.window = window; a.chunk = chunk; a.scale = scale;
     a.keep_first = window > 0 ? keep_first : 0; a.sink = sink; a.sink_val = sink ? sink_val : nullptr;
     a.part_o = nullptr; a.part_ml = nullptr; a.counters = nullptr; a.max_splits = 0;
     return a;
@@ -796,13 +799,13 @@ static AttnArgs make_args(const void* q, const void* pool, void* out, const int*
 extern "C" int locus_attn_chunk(const void* q, int dt, const void* pool, void* out,
                                 const int* seg_q0, const int* seg_qn, const int* seg_ctx,
                                 const int* block_table, int table_stride, const int* items,
-                                int n_items, int nh, int nkv, int hd, int page_tokens, int window,
+                                int n_items, int nh, int nkv, int hd, int page_tokens, int window, int chunk,
                                 float scale, int keep_first, int sink, const float* sink_val, cudaStream_t stream) {
     if (n_items <= 0) return 0;
-    if (int e = check_common(nh, nkv, hd, page_tokens, window, keep_first)) return e;
+    if (int e = check_common(nh, nkv, hd, page_tokens, window, chunk, keep_first)) return e;
     if (n_items > 65535) return LOCUS_ERR_UNSUPPORTED;
     AttnArgs a = make_args(q, pool, out, seg_q0, seg_qn, seg_ctx, block_table, table_stride, items,
-                           nh, nkv, hd, page_tokens, window, scale, keep_first, sink, sink_val);
+                           nh, nkv, hd, page_tokens, window, chunk, scale, keep_first, sink, sink_val);
     const size_t smem = sizeof(float) * (CHUNK_BQ * hd + CHUNK_TK * (hd + 1) + CHUNK_TK * hd +
                                          CHUNK_BQ * (CHUNK_TK + 1) + 3 * CHUNK_BQ);
     dim3 grid(nh, n_items);
@@ -826,15 +829,15 @@ extern "C" int locus_attn_chunk(const void* q, int dt, const void* pool, void* o
 extern "C" int locus_attn_decode(const void* q, int dt, const void* pool, void* out,
                                  const int* seg_q0, const int* seg_qn, const int* seg_ctx,
                                  const int* block_table, int table_stride, const int* items,
-                                 int n_items, int nh, int nkv, int hd, int page_tokens, int window,
+                                 int n_items, int nh, int nkv, int hd, int page_tokens, int window, int chunk,
                                  float scale, float* part_o, float* part_ml, int* counters, int max_splits,
                                  long long max_units, int keep_first, int sink, const float* sink_val,
                                  cudaStream_t stream) {
     if (n_items <= 0) return 0;
-    if (int e = check_common(nh, nkv, hd, page_tokens, window, keep_first)) return e;
+    if (int e = check_common(nh, nkv, hd, page_tokens, window, chunk, keep_first)) return e;
     if (nh > 65535 || max_splits <= 0 || max_splits > 65535) return LOCUS_ERR_UNSUPPORTED;
     AttnArgs a = make_args(q, pool, out, seg_q0, seg_qn, seg_ctx, block_table, table_stride, items,
-                           nh, nkv, hd, page_tokens, window, scale, keep_first, sink, sink_val);
+                           nh, nkv, hd, page_tokens, window, chunk, scale, keep_first, sink, sink_val);
     a.part_o = part_o; a.part_ml = part_ml; a.counters = counters; a.max_splits = max_splits;
     if (counters == nullptr) return LOCUS_ERR_UNSUPPORTED;
     // (one partial result per request and head at least; two where kept first tokens are a range of their own)
@@ -918,7 +921,7 @@ extern "C" int locus_attn_decode_static(const void* q, int dt, const void* pool,
                                         int n_items, int nh, int nkv, int hd, int page_tokens,
                                         int window, float scale, int max_splits, cudaStream_t stream) {
     if (n_items <= 0) return 0;
-    if (int e = check_common(nh, nkv, hd, page_tokens, window)) return e;
+    if (int e = check_common(nh, nkv, hd, page_tokens, window, 0)) return e;
     if (max_splits <= 0) return LOCUS_ERR_UNSUPPORTED;
     // part_o: n_items * nh * max_splits * hd floats, then part_ml: 2 floats per (item, head, split)
     const long long units = static_cast<long long>(n_items) * nh * max_splits;
@@ -948,6 +951,6 @@ extern "C" int locus_attn_decode_static(const void* q, int dt, const void* pool,
     // Nothing to clear: the kernel writes the sums, m and l of every split that it later reads,
     // and the counters are zero between calls.
     return locus_attn_decode(q, dt, pool, out, seg_q0, seg_qn, seg_ctx, block_table, table_stride,
-                             items, n_items, nh, nkv, hd, page_tokens, window, scale, part_o, part_ml,
+                             items, n_items, nh, nkv, hd, page_tokens, window, 0, scale, part_o, part_ml,
                              g_attn_static_cnt_ptr[dev], max_splits, cap, 0, 0, nullptr, stream);
 }

@@ -42,7 +42,7 @@ struct GqaArgs {
     const int* block_table;
     int table_stride;
     const int* items;         // [n_items] segments with one new token
-    int nh, nkv, page_tokens, window;
+    int nh, nkv, page_tokens, window, chunk;  // (mask.cuh)
     const float* sink_val;    // with sink: a learned score per query head in its place (null: the score 0)
     int keep_first, sink;     // with a window: a request's first tokens stay in sight; one more term of score 0 in the denominator
     float scale;
@@ -178,7 +178,7 @@ __global__ void __launch_bounds__(32 * GQW, 1) attn_decode_gqa_kernel(GqaArgs a,
     uint32_t parity = 0;  // bit i: the phase of stage i's barrier that the next wait on it looks for
     const int n_warps = gridDim.x * GQW;
     // a unit (range, kv head) leaves G partial results: the scratch holds max_units of them
-    const int len = plan_key_ranges(kr, a.items, a.seg_ctx, a.seg_q0, a.window, n_items, a.nkv, max_units / G, n_warps,
+    const int len = plan_key_ranges(kr, a.items, a.seg_ctx, a.seg_q0, a.window, a.chunk, n_items, a.nkv, max_units / G, n_warps,
                                     cost_range, cost_merge, a.keep_first);
     // (the cut read only the step's descriptors; q and the newest keys and values come from the kernel in front)
     pdl_entry();
@@ -199,7 +199,7 @@ __global__ void __launch_bounds__(32 * GQW, 1) attn_decode_gqa_kernel(GqaArgs a,
         const int kept = kr.kept[item], keep = a.keep_first;
         const bool kept_range = kept > 0 && r == kr.pref[item];
         const int split = r - kr.pref[item] - (kept > 0);
-        const int t_lo = kept_range ? 0 : (a.window > 0 ? max(0, p - a.window + 1) : 0);
+        const int t_lo = kept_range ? 0 : first_key(a.window, a.chunk, p);
         const int k_begin = kept_range ? 0 : kr.first[item] + split * len;   // a multiple of 32
         const int k_end = kept_range ? kept : min(p + 1, k_begin + len);      // exclusive
         const int* table = a.block_table + static_cast<size_t>(seg) * a.table_stride;
@@ -461,14 +461,13 @@ extern "C" void locus_attn_decode_gqa_set_deep(int deep) { g_gqa_deep = deep; }
 // n_items * nh), part_ml two floats each, counters n_items * nh ints that are zero before and after the call.
 extern "C" int locus_attn_decode_gqa(const void* q, const void* pool, void* out, const int* seg_q0, const int* seg_ctx,
                                      const int* block_table, int table_stride, const int* items, int n_items, int nh,
-                                     int nkv, int hd, int page_tokens, int window, float scale, float* part_o,
+                                     int nkv, int hd, int page_tokens, int window, int chunk, float scale, float* part_o,
                                      float* part_ml, int* counters, long long max_units, int cost_range,
                                      int cost_merge, int keep_first, int sink, const float* sink_val,
                                      cudaStream_t stream) {
     if (n_items <= 0) return 0;
-    if (!locus_attn_decode_gqa_takes(LOCUS_DT_BF16, nh, nkv, hd, page_tokens, n_items) || window < 0 || counters == nullptr)
+    if (!locus_attn_decode_gqa_takes(LOCUS_DT_BF16, nh, nkv, hd, page_tokens, n_items) || !mask_ok(window, chunk, keep_first) || counters == nullptr)
         return LOCUS_ERR_UNSUPPORTED;
-    if (keep_first < 0) return LOCUS_ERR_UNSUPPORTED;
     if (window == 0) keep_first = 0;
     // (one partial result per request and head at least; two where kept first tokens are a range of their own)
     if (max_units < static_cast<long long>(n_items) * nh * (keep_first > 0 ? 2 : 1)) return LOCUS_ERR_UNSUPPORTED;
@@ -486,7 +485,7 @@ extern "C" int locus_attn_decode_gqa(const void* q, const void* pool, void* out,
     a.pool = static_cast<const bf16*>(pool);
     a.out = static_cast<bf16*>(out);
     a.seg_q0 = seg_q0; a.seg_ctx = seg_ctx; a.block_table = block_table; a.table_stride = table_stride; a.items = items;
-    a.nh = nh; a.nkv = nkv; a.page_tokens = page_tokens; a.window = window; a.scale = scale;
+    a.nh = nh; a.nkv = nkv; a.page_tokens = page_tokens; a.window = window; a.chunk = chunk; a.scale = scale;
     a.keep_first = keep_first; a.sink = sink; a.sink_val = sink ? sink_val : nullptr;
     a.part_o = part_o; a.part_ml = part_ml; a.counters = counters;
     const dim3 grid(n_sm);

@@ -20,6 +20,7 @@
 // caller uses the CUDA-core kernel.  Rows in shared memory are
 // padded by 16 bytes so that ldmatrix reads no bank twice.
 #include "common.cuh"
+#include "mask.cuh"
 #include "sink.cuh"
 
 #define MQ 64    // queries per block
@@ -35,7 +36,7 @@ struct MmaAttnArgs {
     const int* block_table;
     int table_stride;
     const int* items;
-    int nh, nkv, page_tokens, window;
+    int nh, nkv, page_tokens, window, chunk;  // (mask.cuh)
     const float* sink_val;  // with sink: a learned score per query head in its place (null: the score 0)
     int keep_first, sink;   // a window that keeps a request's first tokens in sight; one more term of score 0 in the denominator
     float scale;
@@ -47,10 +48,10 @@ struct MmaAttnArgs {
 // Key tiles of an item: the first tile's first position and their number (the same in both kernels).
 // With kept first tokens the tiles that hold them and lie in front of the window's first tile come first
 // (kept_tiles of them, from position 0); tile number i of the item starts at tile_pos(i).
-__device__ __forceinline__ void item_tiles(int p0, int nq, int window, int keep_first, int& first_tile, int& n_tiles,
+__device__ __forceinline__ void item_tiles(int p0, int nq, int window, int chunk, int keep_first, int& first_tile, int& n_tiles,
                                            int& kept_tiles) {
     const int t_hi = p0 + nq - 1;
-    const int t_lo = window > 0 ? max(0, p0 - window + 1) : 0;
+    const int t_lo = first_key(window, chunk, p0);
     first_tile = (t_lo / MK) * MK;
     kept_tiles = window > 0 ? min(first_tile / MK, (min(keep_first, t_lo) + MK - 1) / MK) : 0;
     n_tiles = (t_hi - first_tile) / MK + 1 + kept_tiles;
@@ -111,14 +112,14 @@ __global__ void __launch_bounds__(128) attn_chunk_mma_kernel(MmaAttnArgs a) {
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int g = lane >> 2, qd = lane & 3;
     const int t_hi = p0 + nq - 1;
-    const int t_lo = a.window > 0 ? max(0, p0 - a.window + 1) : 0;
+    const int t_lo = first_key(a.window, a.chunk, p0);
     const int P = a.page_tokens;
     const int pshift = (P & (P - 1)) == 0 ? __ffs(P) - 1 : -1;  // pages of 2^k tokens: shifts instead of divisions
     const float scale_log2 = a.scale * 1.4426950408889634f;
 
     // this block's range of the item's key tiles
     int first_tile, n_tiles_all, kept_tiles;
-    item_tiles(p0, nq, a.window, a.keep_first, first_tile, n_tiles_all, kept_tiles);
+    item_tiles(p0, nq, a.window, a.chunk, a.keep_first, first_tile, n_tiles_all, kept_tiles);
     const int kept = a.window > 0 ? min(a.keep_first, t_lo) : 0;
     const int split = blockIdx.z;
     const int per_split = (n_tiles_all + a.n_splits - 1) / a.n_splits;
@@ -174,7 +175,11 @@ __global__ void __launch_bounds__(128) attn_chunk_mma_kernel(MmaAttnArgs a) {
 #pragma unroll
         for (int i = 0; i < 4; ++i) o[d][i] = 0.f;
     float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
-    const int pq[2] = {p0 + warp * 16 + g, p0 + warp * 16 + g + 8};  // positions of this lane's two query rows
+    const int p_first = p0 + warp * 16;                              // position of the warp's first query row
+    const int pq[2] = {p_first + g, p_first + g + 8};                // positions of this lane's two query rows
+    // the first key that each of the two sees, and that the warp's last row sees
+    const int lo_q[2] = {first_key(a.window, a.chunk, pq[0]), first_key(a.window, a.chunk, pq[1])};
+    const int lo_last = first_key(a.window, a.chunk, p_first + 15);
 
     for (int it = 0; it < n_tiles; ++it) {
         const int tile0 = tile_pos(first_idx + it, first_tile, kept_tiles);
@@ -213,9 +218,7 @@ __global__ void __launch_bounds__(128) attn_chunk_mma_kernel(MmaAttnArgs a) {
         // exp(x * scale - m) = exp2(x * scale * log2(e) - m').  The mask test runs only on tiles that
         // can hold a masked key for one of this warp's rows (the diagonal, the window's edge, the start).
         float mx[2] = {m_run[0], m_run[1]};
-        const int p_first = p0 + warp * 16;
-        const bool need_mask = tile0 + MK - 1 > p_first || tile0 < t_lo ||
-                               (a.window > 0 && tile0 <= p_first + 15 - a.window);
+        const bool need_mask = tile0 + MK - 1 > p_first || tile0 < lo_last;
         if (need_mask) {
 #pragma unroll
             for (int j = 0; j < MK / 8; ++j) {
@@ -223,8 +226,7 @@ __global__ void __launch_bounds__(128) attn_chunk_mma_kernel(MmaAttnArgs a) {
                 for (int i = 0; i < 4; ++i) {
                     const int rr = i >> 1;
                     const int t = tile0 + j * 8 + qd * 2 + (i & 1);
-                    const int p = pq[rr];
-                    const bool ok = t <= p && (a.window == 0 || t > p - a.window || t < a.keep_first);
+                    const bool ok = t <= pq[rr] && (t >= lo_q[rr] || t < a.keep_first);
                     const float v = ok ? s[j][i] * scale_log2 : -INFINITY;
                     s[j][i] = v;
                     mx[rr] = fmaxf(mx[rr], v);
@@ -338,7 +340,7 @@ __global__ void __launch_bounds__(128) attn_chunk_merge_kernel(MmaAttnArgs a, in
     const int r = i / half, d = (i - r * half) * 2;
     const int row0 = a.seg_q0[seg] + qoff;
     int first_tile, n_tiles, kept_tiles;
-    item_tiles(a.seg_ctx[seg] + qoff, nq, a.window, a.keep_first, first_tile, n_tiles, kept_tiles);
+    item_tiles(a.seg_ctx[seg] + qoff, nq, a.window, a.chunk, a.keep_first, first_tile, n_tiles, kept_tiles);
     const int per_split = (n_tiles + a.n_splits - 1) / a.n_splits;
     const int live = (n_tiles + per_split - 1) / per_split;
     const size_t unit0 = (static_cast<size_t>(item) * a.nh + h) * a.n_splits;
@@ -389,11 +391,11 @@ static int launch(const MmaAttnArgs& a, int n_items, cudaStream_t stream) {
 // n_splits > 1: part_o holds n_items * nh * n_splits * 64 * hd floats, part_ml n_items * nh * n_splits * 128.
 extern "C" int locus_attn_chunk_mma(const void* q, const void* pool, void* out, const int* seg_q0, const int* seg_qn,
                                     const int* seg_ctx, const int* block_table, int table_stride, const int* items,
-                                    int n_items, int nh, int nkv, int hd, int page_tokens, int window, float scale,
+                                    int n_items, int nh, int nkv, int hd, int page_tokens, int window, int chunk, float scale,
                                     int n_splits, float* part_o, float* part_ml, int keep_first, int sink, const float* sink_val,
                                     cudaStream_t stream) {
     if (n_items <= 0) return 0;
-    if (nh <= 0 || nkv <= 0 || nh % nkv != 0 || nh > 65535 || page_tokens <= 0 || window < 0 || keep_first < 0)
+    if (nh <= 0 || nkv <= 0 || nh % nkv != 0 || nh > 65535 || page_tokens <= 0 || !mask_ok(window, chunk, keep_first))
         return LOCUS_ERR_UNSUPPORTED;
     if (n_splits < 1 || n_splits > MERGE_MAX_SPLITS || (n_splits > 1 && n_items > 65535) || (n_splits > 1 && (part_o == nullptr || part_ml == nullptr)) ||
         ((reinterpret_cast<uintptr_t>(part_o) | reinterpret_cast<uintptr_t>(part_ml)) & 7))
@@ -402,7 +404,7 @@ extern "C" int locus_attn_chunk_mma(const void* q, const void* pool, void* out, 
     a.q = static_cast<const bf16*>(q); a.pool = static_cast<const bf16*>(pool); a.out = static_cast<bf16*>(out);
     a.seg_q0 = seg_q0; a.seg_qn = seg_qn; a.seg_ctx = seg_ctx; a.block_table = block_table;
     a.table_stride = table_stride; a.items = items; a.nh = nh; a.nkv = nkv; a.page_tokens = page_tokens;
-    a.window = window; a.scale = scale; a.keep_first = window > 0 ? keep_first : 0; a.sink = sink; a.sink_val = sink ? sink_val : nullptr;
+    a.window = window; a.chunk = chunk; a.scale = scale; a.keep_first = window > 0 ? keep_first : 0; a.sink = sink; a.sink_val = sink ? sink_val : nullptr;
     a.n_splits = n_splits; a.part_o = part_o; a.part_ml = part_ml;
     switch (hd) {
         case 16: return launch<16>(a, n_items, stream);

@@ -28,6 +28,7 @@
 #include <string.h>
 
 #include "common.cuh"
+#include "mask.cuh"
 #include "sink.cuh"
 
 #define AT_HD 128        // head size
@@ -47,7 +48,7 @@ struct TcAttnArgs {
     const int* block_table;
     int table_stride;
     const int* items;
-    int nh, nkv, page_tokens, window;
+    int nh, nkv, page_tokens, window, chunk;  // (mask.cuh)
     const float* sink_val;  // with sink: a learned score per query head in its place (null: the score 0)
     int keep_first, sink;   // with a window: a request's first tokens stay in sight; one more term of score 0 in the denominator
     float scale;
@@ -63,10 +64,10 @@ struct TcAttnArgs {
 // tokens that lie wholly in front of the window's first tile (tile j at position j * AT_MK), then the window's
 // (tile j at first_tile + (j - n_keep) * AT_MK); their number, and how they are cut into ranges (the same in both
 // kernels).
-__device__ __forceinline__ void at_tiles(int p0, int nq, int window, int keep_first, int n_splits, int& first_tile,
+__device__ __forceinline__ void at_tiles(int p0, int nq, int window, int chunk, int keep_first, int n_splits, int& first_tile,
                                          int& n_keep, int& n_tiles, int& per_split) {
     const int t_hi = p0 + nq - 1;
-    const int t_lo = window > 0 ? max(0, p0 - window + 1) : 0;
+    const int t_lo = first_key(window, chunk, p0);
     first_tile = (t_lo / AT_MK) * AT_MK;
     n_keep = (window > 0 && keep_first > 0) ? min((keep_first + AT_MK - 1) / AT_MK, first_tile / AT_MK) : 0;
     n_tiles = n_keep + (t_hi - first_tile) / AT_MK + 1;
@@ -236,11 +237,11 @@ attn_chunk_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
     const int row0 = a.seg_q0[seg] + qoff;
     const int p0 = a.seg_ctx[seg] + qoff;
     const int t_hi = p0 + nq - 1;
-    const int t_lo = a.window > 0 ? max(0, p0 - a.window + 1) : 0;
+    const int t_lo = first_key(a.window, a.chunk, p0);
     const int P = a.page_tokens;
     // this block's range of the key tiles (all of them when the keys are not cut)
     int first_tile, n_keep, n_tiles_all, per_split;
-    at_tiles(p0, nq, a.window, a.keep_first, a.n_splits, first_tile, n_keep, n_tiles_all, per_split);
+    at_tiles(p0, nq, a.window, a.chunk, a.keep_first, a.n_splits, first_tile, n_keep, n_tiles_all, per_split);
     const int split = blockIdx.z;
     const int j0 = split * per_split;  // this block's first tile in the list of all
     const int n_tiles = max(0, min(per_split, n_tiles_all - j0));
@@ -379,7 +380,8 @@ attn_chunk_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
         uint8_t* gP0 = at_generic + (sP - base) + half * AT_HALF_BYTES + r * 128;
         float* xch = reinterpret_cast<float*>(at_generic + (slot + 16 - base));  // [2 tile parities][2 halves][128 rows]
         bool ok = true;
-        const int lo = a.window > 0 ? max(0, pq - a.window + 1) : 0;  // first key this row sees
+        const int lo = first_key(a.window, a.chunk, pq);                    // first key this row sees ...
+        const int lo_last = first_key(a.window, a.chunk, p0 + AT_MQ - 1);   // ... and the block's last row
         const uint32_t tOmine = tO + lane_bits + 64 * half;           // this thread's 64 columns of the row's sum
 
         // the two threads of a row exchange a value through shared memory (a barrier of their two warps)
@@ -404,8 +406,7 @@ attn_chunk_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
             asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
             // a key t counts for this row when lo <= t <= pq, or when it is one of the kept first tokens; only tiles
             // at an edge need the test (a tile of kept tokens lies in front of t_lo, so it is always tested)
-            const bool need_mask = tile_first + AT_MK - 1 > p0 || tile_first < t_lo ||
-                                   (a.window > 0 && tile_first <= p0 + AT_MQ - 1 - a.window);
+            const bool need_mask = tile_first + AT_MK - 1 > p0 || tile_first < lo_last;
             float mx = -INFINITY;
             if (need_mask) {
 #pragma unroll
@@ -558,7 +559,7 @@ __global__ void __launch_bounds__(128) attn_chunk_tc_merge_kernel(TcAttnArgs a) 
     const int r = i / (AT_HD / 4), d = (i - r * (AT_HD / 4)) * 4;
     const int row = a.seg_q0[seg] + qoff + r;
     int first_tile, n_keep, n_tiles, per_split;
-    at_tiles(a.seg_ctx[seg] + qoff, nq, a.window, a.keep_first, a.n_splits, first_tile, n_keep, n_tiles, per_split);
+    at_tiles(a.seg_ctx[seg] + qoff, nq, a.window, a.chunk, a.keep_first, a.n_splits, first_tile, n_keep, n_tiles, per_split);
     const int live = (n_tiles + per_split - 1) / per_split;
     const size_t unit0 = (static_cast<size_t>(row) * a.nh + h) * a.n_splits;
     float2 ml[AT_MAX_SPLITS];
@@ -634,7 +635,7 @@ static bool at_make_map(CUtensorMap* map, const void* ptr, long long rows, long 
 extern "C" int locus_attn_chunk_tc(const void* q, long long T, const void* pool, long long n_pages, void* out,
                                    const int* seg_q0, const int* seg_qn, const int* seg_ctx, const int* block_table,
                                    int table_stride, const int* items, int n_items, int nh, int nkv, int hd,
-                                   int page_tokens, int window, float scale, int n_splits, float* part_o,
+                                   int page_tokens, int window, int chunk, float scale, int n_splits, float* part_o,
                                    float* part_ml, int keep_first, int sink, const float* sink_val,
                                    cudaStream_t stream) {
     if (n_items <= 0) return 0;
@@ -642,7 +643,7 @@ extern "C" int locus_attn_chunk_tc(const void* q, long long T, const void* pool,
     if (n_splits > 1 && (part_o == nullptr || part_ml == nullptr ||
                          ((reinterpret_cast<uintptr_t>(part_o) | reinterpret_cast<uintptr_t>(part_ml)) & 15)))
         return LOCUS_ERR_UNSUPPORTED;
-    if (hd != AT_HD || page_tokens <= 0 || page_tokens % 64 != 0 || window < 0 || keep_first < 0) return LOCUS_ERR_UNSUPPORTED;
+    if (hd != AT_HD || page_tokens <= 0 || page_tokens % 64 != 0 || !mask_ok(window, chunk, keep_first)) return LOCUS_ERR_UNSUPPORTED;
     if (nh <= 0 || nkv <= 0 || nh % nkv != 0 || nh > 65535) return LOCUS_ERR_UNSUPPORTED;
     const long long pool_rows = n_pages * 2 * nkv * page_tokens;
     if (T <= 0 || n_pages <= 0 || pool_rows >= (1LL << 31) || T >= (1LL << 31)) return LOCUS_ERR_UNSUPPORTED;
@@ -655,7 +656,7 @@ extern "C" int locus_attn_chunk_tc(const void* q, long long T, const void* pool,
     TcAttnArgs a;
     a.out = static_cast<bf16*>(out); a.seg_q0 = seg_q0; a.seg_qn = seg_qn; a.seg_ctx = seg_ctx;
     a.block_table = block_table; a.table_stride = table_stride; a.items = items; a.nh = nh; a.nkv = nkv;
-    a.page_tokens = page_tokens; a.window = window; a.scale = scale;
+    a.page_tokens = page_tokens; a.window = window; a.chunk = chunk; a.scale = scale;
     a.keep_first = window > 0 ? keep_first : 0; a.sink = sink ? 1 : 0; a.sink_val = sink ? sink_val : nullptr;
     a.n_splits = n_splits; a.part_o = part_o; a.part_ml = part_ml;
     const size_t smem = 7 * AT_TILE_BYTES + 160 + 2 * 2 * 128 * 4;

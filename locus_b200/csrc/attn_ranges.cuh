@@ -3,6 +3,8 @@
 // context lengths.
 #pragma once
 
+#include "mask.cuh"
+
 #define DS_CAND 256       // candidate range lengths looked at
 #define DS_MAX_ITEMS 1024
 
@@ -25,14 +27,14 @@ struct KeyRanges {
 // more range of the item, in front of the others (kr.kept keys from position 0; the caller walks it like any other).
 __device__ __forceinline__ int plan_key_ranges(KeyRanges& kr, const int* __restrict__ items,
                                                const int* __restrict__ seg_ctx, const int* __restrict__ seg_q0,
-                                               int window, int n_items, int per_range, long long max_units,
+                                               int window, int chunk, int n_items, int per_range, long long max_units,
                                                int n_warps, int cost_range, int cost_merge, int keep_first = 0) {
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, n_block_warps = blockDim.x >> 5;
     int longest = 0;
     for (int i = tid; i < n_items; i += blockDim.x) {
         const int seg = items[i];
         const int p = seg_ctx[seg];
-        const int t_lo = window > 0 ? max(0, p - window + 1) : 0;
+        const int t_lo = first_key(window, chunk, p);
         const int first = t_lo & ~31;
         kr.first[i] = first;
         kr.nkeys[i] = p - first + 1;

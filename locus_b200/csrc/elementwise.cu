@@ -4,27 +4,33 @@
 #include "common.cuh"
 
 // ---------------------------------------------------------------------------
-// Embedding: out[t, :] = table[tokens[t], :] as float32 (the residual stream is float32).
+// Embedding: out[t, :] = table[tokens[t], :] as float32 (the residual stream is float32), optionally through a Dynamic
+// Tanh (see below): tanh(alpha v) w + b.
 __global__ void embed_rows_kernel(const int* __restrict__ tokens, const void* __restrict__ table,
-                                  int table_dt, float* __restrict__ out, int H, int copies, float scale) {
+                                  int table_dt, float* __restrict__ out, int H, int copies, float scale,
+                                  const void* __restrict__ alpha, const void* __restrict__ w, const void* __restrict__ b,
+                                  int norm_dt) {
     pdl_entry();
     pdl_trigger();
     const int t = blockIdx.x;
     const size_t row = static_cast<size_t>(tokens[t]) * H;
     float* o = out + static_cast<size_t>(t) * H * copies;
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
-        const float v = ld_dyn(table, table_dt, row + i) * scale;
+        float v = ld_dyn(table, table_dt, row + i) * scale;
+        if (w) v = fmaf(tanhf(ld_dyn(alpha, norm_dt, 0) * v), ld_dyn(w, norm_dt, i), ld_dyn(b, norm_dt, i));
         for (int c = 0; c < copies; ++c) o[c * H + i] = v;
     }
 }
 
 // scale: a factor on the row (1: none).  copies > 1: a row of out holds the table's row that many times, one behind the other (a model that keeps
-// several copies of the residual stream starts them all from the embedding).
+// several copies of the residual stream starts them all from the embedding).  alpha [1], w [H], b [H] (element type
+// norm_dt) or null: a Dynamic Tanh behind the factor.
 extern "C" int locus_embed_rows(const int* tokens, const void* table, int table_dt, float* out,
-                                int T, int H, int copies, float scale, cudaStream_t stream) {
+                                int T, int H, int copies, float scale, const void* alpha, const void* w, const void* b,
+                                int norm_dt, cudaStream_t stream) {
     if (T <= 0) return 0;
-    if (copies < 1) return LOCUS_ERR_UNSUPPORTED;
-    locus_launch(embed_rows_kernel, T, 256, 0, stream, tokens, table, table_dt, out, H, copies, scale);
+    if (copies < 1 || (w != nullptr && (alpha == nullptr || b == nullptr))) return LOCUS_ERR_UNSUPPORTED;
+    locus_launch(embed_rows_kernel, T, 256, 0, stream, tokens, table, table_dt, out, H, copies, scale, alpha, w, b, norm_dt);
     return locus_launch_status();
 }
 
@@ -778,5 +784,144 @@ extern "C" int locus_span_rmsnorm(float* x, int ld, int T, int off0, int n0, con
         return LOCUS_ERR_UNSUPPORTED;
     locus_launch(span_rmsnorm_kernel, dim3(T, w1 != nullptr ? 2 : 1), dim3(256), 0, stream, x, ld, off0, n0, w0, off1, n1, w1,
                  w_dt, eps);
+    return locus_launch_status();
+}
+
+// ---------------------------------------------------------------------------
+// Dynamic Tanh, a norm without statistics: D(z) = tanh(alpha z) w + b with a scalar alpha, elementwise.  Because no
+// element needs another one of its row, the norm behind a sublayer, its layer scale, the addition to the residual stream
+// and the norm in front of the next sublayer are one pass:
+//     u = x[r, :] + ls * D_y(y[r, :])      (without y: u = x[r, :]);   x[r, :] = u unless rows are gathered
+//     out[i, :] = D(u)                     (out null: only the addition)
+// r = rows ? rows[i] : i.  A thread keeps the parameters of its V columns and walks the block's rows.
+struct DytArgs {
+    float* x;
+    const float* y;
+    const void* ya;   // D_y's alpha, weight, bias and the layer scale (null: 1), element type y_dt
+    const void* yw;
+    const void* yb;
+    const void* ls;
+    int y_dt, ls_dt;
+    void* out;
+    const void* a;    // D's
+    const void* w;
+    const void* b;
+    int dt;
+    const int* rows;
+    int n, H, rows_per_block;
+};
+
+template <int V>
+__device__ __forceinline__ void dyt_params(const void* p, int dt, int c, float* o) {
+    if (V == 4) {
+        if (dt == LOCUS_DT_F32) {
+            const float4 v = *reinterpret_cast<const float4*>(static_cast<const float*>(p) + c);
+            o[0] = v.x; o[1 % V] = v.y; o[2 % V] = v.z; o[3 % V] = v.w;
+        } else {
+            const uint2 v = *reinterpret_cast<const uint2*>(static_cast<const bf16*>(p) + c);
+            const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.x));
+            const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.y));
+            o[0] = lo.x; o[1 % V] = lo.y; o[2 % V] = hi.x; o[3 % V] = hi.y;
+        }
+    } else {
+        o[0] = ld_dyn(p, dt, c);
+    }
+}
+
+template <typename TO, int V>
+__global__ void __launch_bounds__(256) dyt_kernel(const DytArgs a) {
+    const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V;
+    const int i0 = blockIdx.y * a.rows_per_block, i1 = min(a.n, i0 + a.rows_per_block);
+    const bool in = c < a.H;
+    // (the parameters are weights: read before the wait for the kernel in front)
+    float w[V], b[V], yw[V], yb[V], ls[V], alpha = 0.f, y_alpha = 0.f;
+#pragma unroll
+    for (int k = 0; k < V; ++k) {
+        w[k] = b[k] = yw[k] = yb[k] = 0.f;
+        ls[k] = 1.f;
+    }
+    if (in && a.out != nullptr) {
+        alpha = ld_dyn(a.a, a.dt, 0);
+        dyt_params<V>(a.w, a.dt, c, w);
+        dyt_params<V>(a.b, a.dt, c, b);
+    }
+    if (in && a.y != nullptr) {
+        y_alpha = ld_dyn(a.ya, a.y_dt, 0);
+        dyt_params<V>(a.yw, a.y_dt, c, yw);
+        dyt_params<V>(a.yb, a.y_dt, c, yb);
+        if (a.ls != nullptr) dyt_params<V>(a.ls, a.ls_dt, c, ls);
+    }
+    pdl_entry();
+    pdl_trigger();
+    if (!in) return;
+#pragma unroll 2
+    for (int i = i0; i < i1; ++i) {
+        const size_t src = static_cast<size_t>(a.rows ? a.rows[i] : i) * a.H + c;
+        float u[V], z[V];
+        if (V == 4) {
+            const float4 v = *reinterpret_cast<const float4*>(a.x + src);
+            u[0] = v.x; u[1 % V] = v.y; u[2 % V] = v.z; u[3 % V] = v.w;
+            if (a.y != nullptr) {
+                const float4 t = *reinterpret_cast<const float4*>(a.y + src);
+                z[0] = t.x; z[1 % V] = t.y; z[2 % V] = t.z; z[3 % V] = t.w;
+            }
+        } else {
+            u[0] = a.x[src];
+            if (a.y != nullptr) z[0] = a.y[src];
+        }
+        if (a.y != nullptr) {
+#pragma unroll
+            for (int k = 0; k < V; ++k) u[k] = fmaf(ls[k], fmaf(tanhf(y_alpha * z[k]), yw[k], yb[k]), u[k]);
+            if (a.rows == nullptr) {
+                if (V == 4) *reinterpret_cast<float4*>(a.x + src) = make_float4(u[0], u[1 % V], u[2 % V], u[3 % V]);
+                else a.x[src] = u[0];
+            }
+        }
+        if (a.out == nullptr) continue;
+#pragma unroll
+        for (int k = 0; k < V; ++k) u[k] = fmaf(tanhf(alpha * u[k]), w[k], b[k]);
+        TO* dst = static_cast<TO*>(a.out) + static_cast<size_t>(i) * a.H + c;
+        if (V == 4 && sizeof(TO) == 4) {
+            *reinterpret_cast<float4*>(dst) = make_float4(u[0], u[1 % V], u[2 % V], u[3 % V]);
+        } else if (V == 4) {
+            __nv_bfloat162 lo = __floats2bfloat162_rn(u[0], u[1 % V]), hi = __floats2bfloat162_rn(u[2 % V], u[3 % V]);
+            *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
+        } else {
+            dst[0] = from_f<TO>(u[0]);
+        }
+    }
+}
+
+// x [*, H] float32; y like x or null; ya [1], yw, yb [H] (element type y_dt), ls [H] (element type ls_dt) or null; out
+// [n, H] (element type out_dt; it may be x itself when y is null and rows too) or null; a [1], w, b [H] (element type dt).
+extern "C" int locus_dyt(float* x, const float* y, const void* ya, const void* yw, const void* yb, int y_dt,
+                         const void* ls, int ls_dt, void* out, int out_dt, const void* alpha, const void* w, const void* b,
+                         int dt, const int* rows, int n, int H, cudaStream_t stream) {
+    if (n <= 0) return 0;
+    if (H <= 0 || x == nullptr || (y == nullptr && out == nullptr)) return LOCUS_ERR_UNSUPPORTED;
+    if (y != nullptr && (ya == nullptr || yw == nullptr || yb == nullptr)) return LOCUS_ERR_UNSUPPORTED;
+    if (out != nullptr && (alpha == nullptr || w == nullptr || b == nullptr)) return LOCUS_ERR_UNSUPPORTED;
+    if (out != nullptr && out_dt != LOCUS_DT_F32 && out_dt != LOCUS_DT_BF16) return LOCUS_ERR_UNSUPPORTED;
+    DytArgs a;
+    a.x = x; a.y = y; a.ya = ya; a.yw = yw; a.yb = yb; a.ls = ls; a.y_dt = y_dt; a.ls_dt = ls_dt; a.out = out;
+    a.a = alpha; a.w = w; a.b = b; a.dt = dt; a.rows = rows; a.n = n; a.H = H;
+    uintptr_t all = 0;
+    const void* ptrs[] = {x, y, yw, yb, ls, out, w, b};
+    for (const void* p : ptrs) all |= reinterpret_cast<uintptr_t>(p);
+    const bool vec = H % 4 == 0 && (all & 15) == 0;
+    const int cols = vec ? H / 4 : H;
+    const int threads = cols >= 256 ? 256 : ceil_div(cols, 32) * 32;
+    const int col_blocks = ceil_div(cols, threads);
+    // about eight blocks per SM, sixteen rows each at most
+    long long rpb = static_cast<long long>(n) * col_blocks / (148 * 8);
+    a.rows_per_block = static_cast<int>(rpb < 1 ? 1 : (rpb > 16 ? 16 : rpb));
+    const int row_blocks = ceil_div(n, a.rows_per_block);
+    if (row_blocks > 65535) return LOCUS_ERR_UNSUPPORTED;
+    const dim3 grid(col_blocks, row_blocks);
+    const bool f32 = out == nullptr || out_dt == LOCUS_DT_F32;
+    if (vec && f32) locus_launch(dyt_kernel<float, 4>, grid, dim3(threads), 0, stream, a);
+    else if (vec) locus_launch(dyt_kernel<bf16, 4>, grid, dim3(threads), 0, stream, a);
+    else if (f32) locus_launch(dyt_kernel<float, 1>, grid, dim3(threads), 0, stream, a);
+    else locus_launch(dyt_kernel<bf16, 1>, grid, dim3(threads), 0, stream, a);
     return locus_launch_status();
 }

@@ -31,7 +31,8 @@ struct GemmArgs {
     int act;                 // 0: none; 1: relu(v)^2 (after the bias, before the row scale); 2 (with w2): the clamped
                              // gated unit g' sigmoid(1.702 g') (u' + 1), g' = min(s g, limit), u' = clamp(s u, +-limit),
                              // s the row's scale, which then stands for a factor on the input
-    float act_param;         // the limit of act 2
+    float act_param;         // the limit of act 2; the cap of act 3 (without w2): cap tanh(act_scale v / cap), behind everything else
+    float act_scale;
     const float* row_scale;  // or null: row m is scaled by row_scale[scale_rows ? scale_rows[m] : m]
     const int* scale_rows;
     const int* x_rows;       // [M] or null
@@ -153,6 +154,7 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(GemmArgs a) {
                 v *= v;
             }
             if (a.row_scale && a.act != 2) v *= rs;
+            if (a.act == 3) v = a.act_param * tanhf(v * a.act_scale / a.act_param);
             const size_t o = static_cast<size_t>(r) * a.ldo + n;
             if (a.accumulate) {
                 static_cast<float*>(a.out)[o] += v;
@@ -177,11 +179,12 @@ static int launch(const GemmArgs& a, int max_tiles, bool swiglu, cudaStream_t st
 }
 
 // x_dt / w_dt: element types of x and of W (and W2).  flags: bit 0 = add the result into the float32 out,
-// bits 1-2 = the activation: 1 squared ReLU (not with W2), 2 the clamped gated unit with limit act_param (with W2).  max_tiles: number of 64-row tiles
+// bits 1-2 = the activation: 1 squared ReLU (not with W2), 2 the clamped gated unit with limit act_param (with W2),
+// 3 act_param tanh(act_scale v / act_param) (not with W2).  max_tiles: number of 64-row tiles
 // to launch; for a grouped product an upper bound (tiles past *n_tiles return at once).
 extern "C" int locus_gemm_simt(const void* x, int x_dt, const void* w, const void* w2, int w_dt,
                                const void* bias, int bias_dt, void* out, int out_dt,
-                               int flags, float act_param, const float* row_scale, const int* scale_rows,
+                               int flags, float act_param, float act_scale, const float* row_scale, const int* scale_rows,
                                const int* x_rows,
                                int x_row_div, int M, int N, int K, long long ldx, long long ldo,
                                const int* tile_expert, const int* tile_row0,
@@ -189,12 +192,12 @@ extern "C" int locus_gemm_simt(const void* x, int x_dt, const void* w, const voi
                                long long w_expert_stride, cudaStream_t stream) {
     if (N <= 0 || K <= 0) return LOCUS_ERR_UNSUPPORTED;
     const int accumulate = flags & 1, act = (flags >> 1) & 3;
-    if ((act == 1 && w2 != nullptr) || (act == 2 && w2 == nullptr) || act == 3) return LOCUS_ERR_UNSUPPORTED;
+    if ((act == 1 && w2 != nullptr) || (act == 2 && w2 == nullptr) || (act == 3 && (w2 != nullptr || !(act_param > 0.f)))) return LOCUS_ERR_UNSUPPORTED;
     if (accumulate && out_dt != LOCUS_DT_F32) return LOCUS_ERR_UNSUPPORTED;
     if (x_rows != nullptr && x_row_div <= 0) return LOCUS_ERR_UNSUPPORTED;
     GemmArgs a;
     a.x = x; a.w = w; a.w2 = w2; a.bias = bias; a.bias_dt = bias_dt; a.out = out;
-    a.out_dt = out_dt; a.accumulate = accumulate; a.act = act; a.act_param = act_param; a.row_scale = row_scale; a.scale_rows = scale_rows; a.x_rows = x_rows;
+    a.out_dt = out_dt; a.accumulate = accumulate; a.act = act; a.act_param = act_param; a.act_scale = act_scale; a.row_scale = row_scale; a.scale_rows = scale_rows; a.x_rows = x_rows;
     a.x_row_div = x_row_div; a.M = M; a.N = N; a.K = K; a.ldx = ldx; a.ldo = ldo;
     a.tile_expert = tile_expert; a.tile_row0 = tile_row0; a.tile_rows = tile_rows;
     a.n_tiles = n_tiles; a.w_expert_stride = w_expert_stride;

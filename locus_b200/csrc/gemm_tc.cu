@@ -65,7 +65,8 @@ struct TcArgs {
     int act;  // 1: relu(v)^2 after the bias, before the row scale (never with a product split along K); 2 (two weights):
               // the clamped gated unit g' sigmoid(1.702 g') (u' + 1), g' = min(s g, limit), u' = clamp(s u, +-limit), s the
               // row's scale (then a factor on the input)
-    float act_param;  // the limit of act 2
+    float act_param;  // the limit of act 2; the cap of act 3 (one weight, never split): cap tanh(act_scale v / cap), behind everything else
+    float act_scale;
     void* out;
     int out_dt;
     long long ldo;
@@ -454,6 +455,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                         x *= x;
                     }
                     if (a.row_scale) x *= scales[c0 + j];
+                    if (a.act == 3) x = a.act_param * tanhf(x * a.act_scale / a.act_param);
                     val[j] = x;
                 }
                 if (wide) {
@@ -614,13 +616,15 @@ static int pow2_at_least(int v) {
 // kernel adds them in order and does the epilogue.  The splits are renumbered so that none is empty.
 extern "C" int locus_gemm_tc(const void* x, long long x_rows_total, long long ldx, const void* w, const void* w2,
                              long long w_rows_total, const void* bias, int bias_dt, void* out, int out_dt,
-                             int flags, float act_param, const float* row_scale, const int* scale_rows, int M, int N, int K,
+                             int flags, float act_param, float act_scale, const float* row_scale, const int* scale_rows, int M, int N, int K,
                              long long ldo, int TN, const int* tile_expert, const int* tile_row0,
                              const int* tile_rows, const int* n_tiles, int max_tiles, float* split_scratch,
                              int splits, cudaStream_t stream) {
     const int dual = w2 != nullptr ? 1 : 0;
     const int accumulate = flags & 1, act = (flags >> 1) & 3;  // bit 0: add into out; bits 1-2: the activation
-    if ((act == 1 && (dual || splits > 1)) || (act == 2 && (!dual || splits > 1)) || act == 3) return LOCUS_ERR_UNSUPPORTED;
+    if ((act == 1 && (dual || splits > 1)) || (act == 2 && (!dual || splits > 1)) ||
+        (act == 3 && (dual || splits > 1 || !(act_param > 0.f))))
+        return LOCUS_ERR_UNSUPPORTED;
     if (N <= 0 || K <= 0 || K % 8 != 0 || ldx % 8 != 0) return LOCUS_ERR_UNSUPPORTED;
     if (TN < 16 || TN > 256 || TN % 16 != 0 || (dual && TN > 256)) return LOCUS_ERR_UNSUPPORTED;
     if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(w2)) & 15)
@@ -676,6 +680,7 @@ extern "C" int locus_gemm_tc(const void* x, long long x_rows_total, long long ld
     a.accumulate = split ? 0 : accumulate;
     a.act = act;
     a.act_param = act_param;
+    a.act_scale = act_scale;
     a.out = split ? split_scratch : out;
     a.out_dt = split ? LOCUS_DT_F32 : out_dt;
     a.ldo = split ? N : ldo;

@@ -65,6 +65,7 @@ struct Cache {
     int page_tokens, n_pages, max_seq_tokens, table_width;  // n_pages: of the largest group
     std::vector<int> window;  // per group, 0 = all keys
     std::vector<int> keep;    // per group with a window: a request's first tokens that stay in sight (their pages never go back)
+    std::vector<int> aligned;  // per group without a window: > 0, queries see the keys of their own chunk of that many positions
     std::vector<Pool> pools;
     Pool slots;
     std::vector<Seq> seqs;
@@ -78,16 +79,17 @@ struct Cache {
         for (int g = 0; g < n_groups; ++g) {
             window.push_back(windows[g]);
             keep.push_back(0);
+            aligned.push_back(0);
             pools.emplace_back(group_pages[g]);
             n_pages = group_pages[g] > n_pages ? group_pages[g] : n_pages;
         }
     }
     int n_groups() const { return static_cast<int>(pools.size()); }
     // Pages that a request of n_tokens tokens holds in group g at most, when no step feeds it more than
-    // step_tokens at once: all of them, or in a group with a window those that cover the window and the step.
+    // step_tokens at once: all of them, or in a group with a window (or chunks) those that cover it and the step.
     int pages_needed(int g, int n_tokens, int step_tokens) const {
         const int all = pages_of(n_tokens, page_tokens);
-        const int w = window[static_cast<size_t>(g)];
+        const int w = window[static_cast<size_t>(g)] > 0 ? window[static_cast<size_t>(g)] : aligned[static_cast<size_t>(g)];
         if (w <= 0 || step_tokens <= 0) return all;
         const int span = pages_of(w + step_tokens, page_tokens) + 1 + pages_of(keep[static_cast<size_t>(g)], page_tokens);
         return all < span ? all : span;
@@ -238,9 +240,18 @@ int locus_cache_set_keep(void* cv, int g, int keep_first) {
     return 0;
 }
 
-// n tokens were written after the cached ones.  In a group with a window, pages that no later
-// query can see go back: a query at position p sees keys t > p - window and the next query is at
-// position n_tokens, so pages wholly below n_tokens - window + 1 are dead.  Writes the (group,
+// A group's queries see the keys of their own chunk of `size` positions (counted from position 0) up to themselves.
+// Set before the first request opens, for a group without a window.  0 ok; -1 no such group, a negative size or a window.
+int locus_cache_set_aligned(void* cv, int g, int size) {
+    Cache* c = as_cache(cv);
+    if (g < 0 || g >= c->n_groups() || size < 0 || c->window[static_cast<size_t>(g)] > 0) return -1;
+    c->aligned[static_cast<size_t>(g)] = size;
+    return 0;
+}
+
+// n tokens were written after the cached ones.  In a group with a window or chunks, pages that no later
+// query can see go back: the next query is at position n_tokens; with a window it sees keys t > n_tokens - window, with
+// chunks those from its chunk's start on, and pages wholly below that are dead.  Writes the (group,
 // page) pairs that became free to freed (cap ints) and returns their number; -1 not open; -3 the
 // tokens do not fit the capacity.
 int locus_cache_commit(void* cv, int64_t h, int n, int* freed, int cap) {
@@ -251,11 +262,11 @@ int locus_cache_commit(void* cv, int64_t h, int n, int* freed, int cap) {
     s->n_tokens += n;
     int n_freed = 0;
     for (int g = 0; g < c->n_groups(); ++g) {
-        const int w = c->window[static_cast<size_t>(g)];
-        if (w <= 0) continue;
+        const int w = c->window[static_cast<size_t>(g)], chunk = c->aligned[static_cast<size_t>(g)];
+        if (w <= 0 && chunk <= 0) continue;
         auto& t = s->tables[static_cast<size_t>(g)];
-        int dead = (s->n_tokens - w + 1) / c->page_tokens;
-        if (s->n_tokens - w + 1 < 0) dead = 0;
+        const int first = w > 0 ? s->n_tokens - w + 1 : s->n_tokens - s->n_tokens % chunk;  // the first key in sight
+        int dead = first > 0 ? first / c->page_tokens : 0;
         if (dead > static_cast<int>(t.size())) dead = static_cast<int>(t.size());
         // (the pages that hold a request's kept first tokens stay)
         for (int i = pages_of(c->keep[static_cast<size_t>(g)], c->page_tokens); i < dead; ++i) {

@@ -5,10 +5,11 @@
 //   head_prep        one warp per (token, q | k | v, head).  The head's channels pass, in this order and each only
 //                    if asked for: the convolution y_t = sum_j w[c, j] u_(t - taps + 1 + j) (a portion's first
 //                    tokens read the inputs of the tokens before it from the request's state slot; zeros at a
-//                    request's start, since a slot is zeroed when a request opens), silu, the rotation of the pairs
-//                    (i, i + rot/2) of the first `rot` channels of a q or k head by position * inv_freq[i], and
-//                    for q and k the division by sqrt(mean(x^2) + eps) (norm 1) or sqrt(sum(x^2) + eps) (norm 2)
-//                    and q's factor.  The result goes, in the output's element type, to q's rows and to k's and
+//                    request's start, since a slot is zeroed when a request opens), silu, for q and k an RMS norm over
+//                    the head with a weight per channel (norm 3), the rotation of the pairs (i, i + rot/2), or of the
+//                    adjacent pairs (2i, 2i + 1), of the first `rot` channels of a q or k head by position *
+//                    inv_freq[i], and for q and k the division by sqrt(mean(x^2) + eps) (norm 1) or sqrt(sum(x^2) +
+//                    eps) (norm 2) and q's factor.  The result goes, in the output's element type, to q's rows and to k's and
 //                    v's rows or cache pages, laid out at `laid` elements per head (zeros behind the head's own).
 //                    With gates (a gated delta rule's), one more warp per token forms beta = sigmoid(b) and
 //                    decay = exp(-exp(A_log) * softplus(a + dt_bias)) for every head.
@@ -35,7 +36,9 @@ struct PrepArgs {
     const int* seg_qn;
     const int* positions;     // [T]
     const float* inv_freq;    // [rot / 2] or null
-    int rot, norm;
+    int rot, adjacent, norm;
+    const void* norm_w[2];    // norm 3: q's and k's weights [dim], shared by the heads
+    int norm_w_dt;
     float eps, q_scale;
     void* q_out;              // [T, heads[0] * laid[0]]
     void* k_out;              // rows [T, heads[1] * laid[1]] and v_out alike, or, with pool set, unused
@@ -102,20 +105,28 @@ __global__ void __launch_bounds__(128) head_prep_kernel(const PrepArgs a) {
         buf[i] = a.act ? sc_silu(acc) : acc;
     }
     __syncwarp();
+    if (which < 2 && a.norm == 3) {
+        float ss = 0.f;
+        for (int i = lane; i < d; i += 32) ss = fmaf(buf[i], buf[i], ss);
+        const float rms = 1.0f / sqrtf(warp_sum(ss) / static_cast<float>(d) + a.eps);
+        for (int i = lane; i < d; i += 32) buf[i] *= rms * ld_dyn(a.norm_w[which], a.norm_w_dt, i);
+        __syncwarp();
+    }
     if (which < 2 && a.rot > 0 && a.inv_freq != nullptr) {
         const int half = a.rot / 2;
         const float pos = static_cast<float>(a.positions[row]);
         for (int i = lane; i < half; i += 32) {
             float sn, cs;
             sincosf(pos * a.inv_freq[i], &sn, &cs);
-            const float u = buf[i], v = buf[i + half];
-            buf[i] = u * cs - v * sn;
-            buf[i + half] = v * cs + u * sn;
+            const int iu = a.adjacent ? 2 * i : i, iv = a.adjacent ? 2 * i + 1 : i + half;
+            const float u = buf[iu], v = buf[iv];
+            buf[iu] = u * cs - v * sn;
+            buf[iv] = v * cs + u * sn;
         }
         __syncwarp();
     }
     float r = 1.0f;
-    if (which < 2 && a.norm != 0) {
+    if (which < 2 && (a.norm == 1 || a.norm == 2)) {
         float ss = 0.f;
         for (int i = lane; i < d; i += 32) ss = fmaf(buf[i], buf[i], ss);
         ss = warp_sum(ss);
@@ -161,11 +172,13 @@ __global__ void __launch_bounds__(256) conv_state_move_kernel(const float* __res
 // sizes [12]: off, heads, dim, laid of q, k, v.  conv [channels, taps] (element type conv_dt) or null; conv_state: the
 // address of the convolution's part of slot 0, moved on by the call when move_state is set.  out_dt: the element type
 // of q_out, k_out, v_out and the pool.  pool: the layer's pages (k and v go there, at slots[t]) or null (k_out, v_out).
-// gates: beta, decay [T, gate_heads] float32 from columns off_b, off_a of proj, or beta null.
+// adjacent: rotate the pairs (2i, 2i + 1) instead of (i, i + rot/2).  norm 3: q_norm_w, k_norm_w [dim] of element type
+// norm_w_dt.  gates: beta, decay [T, gate_heads] float32 from columns off_b, off_a of proj, or beta null.
 extern "C" int locus_head_prep(const float* proj, int ld, const int* sizes, const void* conv, int conv_dt, int taps, int act,
                                float* conv_state, long long slot_stride, int move_state, const int* state_slots,
                                const int* seg_q0, const int* seg_qn, int n_seg, int longest_new, const int* positions,
-                               const float* inv_freq, int rot, int norm, float eps, float q_scale, void* q_out, void* k_out,
+                               const float* inv_freq, int rot, int adjacent, int norm, const void* q_norm_w,
+                               const void* k_norm_w, int norm_w_dt, float eps, float q_scale, void* q_out, void* k_out,
                                void* v_out, void* pool, const int* slots, int page_tokens, int write_kv, int out_dt,
                                float* beta, float* decay, int off_b, int off_a, int gate_heads, const void* a_log,
                                const void* dt_bias, int gate_dt, cudaStream_t stream) {
@@ -180,11 +193,13 @@ extern "C" int locus_head_prep(const float* proj, int ld, const int* sizes, cons
     if (taps < 1 || taps > PREP_MAX_TAPS || n_seg > 65535 || longest_new > 65535) return LOCUS_ERR_UNSUPPORTED;
     if (rot < 0 || rot % 2 || rot > a.dim[0] || rot > a.dim[1] || (rot > 0 && inv_freq == nullptr)) return LOCUS_ERR_UNSUPPORTED;
     if (conv != nullptr && taps > 1 && conv_state == nullptr) return LOCUS_ERR_UNSUPPORTED;
+    if (norm < 0 || norm > 3 || (norm == 3 && (q_norm_w == nullptr || (k_norm_w == nullptr && a.heads[1] > 0)))) return LOCUS_ERR_UNSUPPORTED;
     if (pool != nullptr && (a.laid[1] != a.laid[2] || page_tokens <= 0 || slots == nullptr)) return LOCUS_ERR_UNSUPPORTED;
     if (beta != nullptr && (decay == nullptr || gate_heads <= 0 || a_log == nullptr || dt_bias == nullptr)) return LOCUS_ERR_UNSUPPORTED;
     a.proj = proj; a.ld = ld; a.conv = conv; a.conv_dt = conv_dt; a.taps = conv ? taps : 1; a.act = act;
     a.conv_state = conv_state; a.slot_stride = slot_stride; a.state_slots = state_slots; a.seg_q0 = seg_q0; a.seg_qn = seg_qn;
-    a.positions = positions; a.inv_freq = inv_freq; a.rot = rot; a.norm = norm; a.eps = eps; a.q_scale = q_scale;
+    a.positions = positions; a.inv_freq = inv_freq; a.rot = rot; a.adjacent = adjacent; a.norm = norm;
+    a.norm_w[0] = q_norm_w; a.norm_w[1] = k_norm_w; a.norm_w_dt = norm_w_dt; a.eps = eps; a.q_scale = q_scale;
     a.q_out = q_out; a.k_out = k_out; a.v_out = v_out; a.pool = pool; a.slots = slots; a.page_tokens = page_tokens;
     a.write_kv = write_kv; a.beta = beta; a.decay = decay; a.off_b = off_b; a.off_a = off_a; a.gate_heads = gate_heads;
     a.a_log = a_log; a.dt_bias = dt_bias; a.gate_dt = gate_dt;

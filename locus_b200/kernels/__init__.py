@@ -199,9 +199,10 @@ F = ctypes.c_float
 
 
 # ---------------------------------------------------------------------------
-def embed_rows(tokens: torch.Tensor, table: torch.Tensor, out: torch.Tensor, copies: int = 1, scale: float = 1.0) -> None:
+def embed_rows(tokens: torch.Tensor, table: torch.Tensor, out: torch.Tensor, copies: int = 1, scale: float = 1.0,
+               dyt_norm=None) -> None:
     """out[t, :] = table[tokens[t], :] * scale as float32; ``copies`` > 1: the row that many times, one behind the
-    other (``out`` [T, copies * H])."""
+    other (``out`` [T, copies * H]).  ``dyt_norm`` = (alpha, weight, bias): the row through :func:`dyt`'s norm."""
     _i32(tokens, "tokens")
     _cuda_c(table, "table")
     _cuda_c(out, "out")
@@ -209,9 +210,55 @@ def embed_rows(tokens: torch.Tensor, table: torch.Tensor, out: torch.Tensor, cop
     _need(out.dtype == torch.float32, "embed_rows: out must be float32")
     _need(tokens.numel() == T and copies >= 1 and out.shape[1] == H * copies, "embed_rows: shape mismatch")
     code = _lib("elementwise").locus_embed_rows(
-        _p(tokens), _p(table), I(dtype_code(table.dtype)), _p(out), I(T), I(H), I(copies), F(scale), _stream()
+        _p(tokens), _p(table), I(dtype_code(table.dtype)), _p(out), I(T), I(H), I(copies), F(scale),
+        *_dyt_args(dyt_norm, H), _stream()
     )
     _check(code, "embed_rows")
+
+
+def _dyt_args(norm, H: int):
+    """(alpha, weight, bias, element type) of a Dynamic Tanh norm for the entry points; None: no norm."""
+    if norm is None:
+        return None, None, None, I(0)
+    alpha, w, b = norm
+    for t, n in ((alpha, 1), (w, H), (b, H)):
+        _need(t.is_cuda and t.is_contiguous() and t.numel() == n and t.dtype == w.dtype,
+              "dyt: alpha [1], weight and bias [H] of one element type on the device")
+    return _p(alpha), _p(w), _p(b), I(dtype_code(w.dtype))
+
+
+def dyt(x: torch.Tensor, norm=None, out: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None,
+        add=None) -> None:
+    """Dynamic Tanh, D(z) = tanh(alpha z) * weight + bias elementwise, ``norm`` = (alpha, weight, bias): out[i] = D(u) with
+    u = x[rows[i] if rows else i] (float32 rows).  ``add`` = (y, (alpha, weight, bias), scale or None): u = x + scale *
+    D_y(y) instead, D_y with those parameters and ``y`` rows like ``x``; without ``rows`` u is written back to ``x``.
+    ``out`` may be absent (only the addition), or ``x`` itself (neither ``rows`` nor ``add``)."""
+    _f32c(x, "dyt: x")
+    H = x.shape[-1]
+    n = x.shape[0] if out is None else out.shape[0]
+    _need(x.is_contiguous() and (out is not None or add is not None) and (norm is None) == (out is None), "dyt: norm and out go together")
+    if out is not None:
+        _cuda_c(out, "out")
+        _need(out.shape[-1] == H, "dyt: out width")
+        _need(out.data_ptr() != x.data_ptr() or (rows is None and add is None), "dyt: out is x")
+    if rows is not None:
+        _i32(rows, "rows")
+        _need(rows.numel() == n and out is not None, "dyt: rows/out mismatch")
+    else:
+        _need(x.shape[0] >= n, "dyt: x/out mismatch")
+    y = ls = None
+    y_norm = None
+    if add is not None:
+        y, y_norm, ls = add
+        _f32c(y, "dyt: y")
+        _need(y.is_contiguous() and y.shape[-1] == H and y.shape[0] >= (x.shape[0] if rows is not None else n), "dyt: y rows")
+        if ls is not None:
+            _cuda_c(ls, "scale")
+            _need(ls.numel() == H, "dyt: scale [H]")
+    code = _lib("elementwise").locus_dyt(
+        _p(x), _p(y), *_dyt_args(y_norm, H), _p(ls), I(dtype_code(ls.dtype) if ls is not None else 0), _p(out),
+        I(dtype_code(out.dtype) if out is not None else 0), *_dyt_args(norm, H), _p(rows), I(n), I(H), _stream())
+    _check(code, "dyt")
 
 
 def rmsnorm_adds(x: torch.Tensor) -> bool:
@@ -432,7 +479,7 @@ def expert_tile(n_pairs: int, n_experts: int) -> int:
 
 
 # activations of a product's epilogue, by their code in the kernels' flags
-ACTIVATIONS = {None: 0, "relu2": 1, "glu_clamp": 2}
+ACTIVATIONS = {None: 0, "relu2": 1, "glu_clamp": 2, "softcap": 3}
 
 
 def tc_error() -> int:
@@ -446,13 +493,14 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, w2: Optional[
            row_scale: Optional[torch.Tensor] = None, scale_rows: Optional[torch.Tensor] = None,
            x_rows: Optional[torch.Tensor] = None, x_row_div: int = 1, layout: Optional[ExpertLayout] = None,
            n_rows: Optional[int] = None, lists_ready: bool = False, second_tiles: bool = False,
-           act: Optional[str] = None, act_limit: float = 0.0) -> None:
+           act: Optional[str] = None, act_limit: float = 0.0, act_scale: float = 1.0) -> None:
     """out = x . w^T with float32 accumulation on CUDA cores (see csrc/gemm_simt.cu).
 
     ``w2``: out = silu(x . w^T) * (x . w2^T).  ``act`` = "relu2": out = max(x . w^T + bias, 0)^2 (not with ``w2``).
     ``act`` = "glu_clamp" (with ``w2``): the clamped gated unit out = g sigmoid(1.702 g) (u + 1) with g = min(s x . w^T,
     ``act_limit``), u = clamp(s x . w2^T, -act_limit, act_limit), where s is the row's ``row_scale`` (1 without): the
-    scale then stands for a factor on the row of x and is not applied once more behind the activation.  ``bias`` [N] is added, ``row_scale`` [M]
+    scale then stands for a factor on the row of x and is not applied once more behind the activation.  ``act`` =
+    "softcap" (not with ``w2``): ``act_limit`` * tanh(``act_scale`` * v / ``act_limit``) behind everything else.  ``bias`` [N] is added, ``row_scale`` [M]
     multiplies the row (``scale_rows``: row m uses row_scale[scale_rows[m]]), ``accumulate`` adds the result into the float32 ``out``.
     ``x_rows``: logical row m reads x[x_rows[m] // x_row_div].  ``layout``: grouped product,
     ``w`` is [E, N, K] and logical rows are the expert-sorted pairs of the layout.
@@ -478,8 +526,10 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, w2: Optional[
         _need(w2.shape == w.shape and w2.dtype == w.dtype and w2.is_contiguous(), "linear: w2 must match w")
     if accumulate:
         _need(out.dtype == torch.float32, "linear: accumulate needs a float32 out")
-    _need(act in ACTIVATIONS and not (act == "relu2" and w2 is not None) and not (act == "glu_clamp" and (w2 is None or not act_limit > 0)),
-          f"linear: activation {act!r} (known: relu2 without w2; glu_clamp with w2 and a positive act_limit)")
+    _need(act in ACTIVATIONS and not (act == "relu2" and w2 is not None) and not (act == "glu_clamp" and (w2 is None or not act_limit > 0))
+          and not (act == "softcap" and (w2 is not None or not act_limit > 0)),
+          f"linear: activation {act!r} (known: relu2 without w2; glu_clamp with w2 and a positive act_limit; softcap without "
+          "w2 and with a positive act_limit)")
     flags = I((1 if accumulate else 0) | (ACTIVATIONS[act] << 1))
     if bias is not None:
         _need(bias.numel() == N and bias.is_contiguous(), "linear: bias size")
@@ -508,7 +558,7 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, w2: Optional[
             max_tiles = stride = 0
         code = _lib("gemm_skinny").locus_gemm_skinny(
             _p(x), _p(w), _p(w2), _p(bias), I(dtype_code(bias.dtype) if bias is not None else 0), _p(out),
-            I(dtype_code(out.dtype)), flags, F(act_limit), _p(row_scale), _p(scale_rows), _p(x_rows),
+            I(dtype_code(out.dtype)), flags, F(act_limit), F(act_scale), _p(row_scale), _p(scale_rows), _p(x_rows),
             I(x_row_div), I(M), I(N), I(K), LL(x.stride(0)), LL(out.stride(0)), I(tile), _p(te), _p(t0), _p(tr),
             _p(nt), I(max_tiles), LL(stride), I(1 if (lists_ready and layout is not None) else 0), _stream()
         )
@@ -526,7 +576,7 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, w2: Optional[
         code = _lib("gemv").locus_gemv(
             _p(x), I(dtype_code(x.dtype)), _p(w), _p(w2), I(dtype_code(w.dtype)), _p(bias),
             I(dtype_code(bias.dtype) if bias is not None else 0), _p(out), I(dtype_code(out.dtype)),
-            flags, F(act_limit), _p(row_scale), _p(scale_rows), _p(x_rows), I(x_row_div), I(M), I(N), I(K),
+            flags, F(act_limit), F(act_scale), _p(row_scale), _p(scale_rows), _p(x_rows), I(x_row_div), I(M), I(N), I(K),
             LL(x.stride(0)), LL(out.stride(0)), _p(te), _p(t0), _p(tr), _p(nt), I(max_tiles), LL(stride), _stream()
         )
         _check(code, "linear", f"(few rows; M={M}, N={N}, K={K}, x {x.dtype}, w {w.dtype})")
@@ -554,7 +604,7 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, w2: Optional[
         code = _lib("gemm_tc").locus_gemm_tc(
             _p(x), LL(M), LL(x.stride(0)), _p(w), _p(w2), LL(w.numel() // K), _p(bias),
             I(dtype_code(bias.dtype) if bias is not None else 0), _p(out), I(dtype_code(out.dtype)),
-            flags, F(act_limit), _p(row_scale), _p(scale_rows), I(M), I(N), I(K), LL(out.stride(0)), I(TN),
+            flags, F(act_limit), F(act_scale), _p(row_scale), _p(scale_rows), I(M), I(N), I(K), LL(out.stride(0)), I(TN),
             _p(te), _p(t0), _p(tr), _p(nt), I(max_tiles), _p(scratch if splits > 1 else None), I(splits), _stream()
         )
         if splits > 1 and code == 0:
@@ -574,7 +624,7 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, w2: Optional[
     code = _lib("gemm_simt").locus_gemm_simt(
         _p(x), I(dtype_code(x.dtype)), _p(w), _p(w2), I(dtype_code(w.dtype)), _p(bias),
         I(dtype_code(bias.dtype) if bias is not None else 0), _p(out), I(dtype_code(out.dtype)),
-        flags, F(act_limit), _p(row_scale), _p(scale_rows), _p(x_rows), I(x_row_div), I(M), I(N), I(K),
+        flags, F(act_limit), F(act_scale), _p(row_scale), _p(scale_rows), _p(x_rows), I(x_row_div), I(M), I(N), I(K),
         LL(x.stride(0)), LL(out.stride(0)), _p(te), _p(t0), _p(tr), _p(nt), I(max_tiles), LL(stride),
         _stream()
     )
@@ -624,12 +674,13 @@ def _sink_args(sink, n_heads: int):
 def attn_chunk(q: torch.Tensor, pool: torch.Tensor, out: torch.Tensor, *, seg_q0: torch.Tensor,
                seg_qn: torch.Tensor, seg_ctx: torch.Tensor, block_table: torch.Tensor,
                items: torch.Tensor, n_items: int, n_heads: int, n_kv_heads: int, head_dim: int,
-               page_tokens: int, window: int, scale: float, keep_first: int = 0, sink=False) -> None:
+               page_tokens: int, window: int, scale: float, keep_first: int = 0, sink=False, chunk: int = 0) -> None:
     """Attention of portions of prompts: ``items`` [n_items, 2] = (segment, first query of a
     16-query tile).  Keys come from the cache through ``block_table`` [n_seg, width].  ``keep_first``: with a
     window, a request's first that many tokens stay in sight of every later query; ``sink``: the softmax has one
     more term in its denominator that has no value: True for the score 0, a float32 tensor [n_heads] for a learned
-    score per head (taken as it is, not multiplied by ``scale``)."""
+    score per head (taken as it is, not multiplied by ``scale``).  ``chunk`` > 0 (without a window): a query sees the keys of
+    its own chunk of that many positions, counted from position 0, up to itself."""
     _cuda_c(q, "q")
     _cuda_c(out, "out")
     _cuda_c(pool, "pool")
@@ -639,7 +690,7 @@ def attn_chunk(q: torch.Tensor, pool: torch.Tensor, out: torch.Tensor, *, seg_q0
     code = _lib("attention").locus_attn_chunk(
         _p(q), I(dtype_code(q.dtype)), _p(pool), _p(out), _p(seg_q0), _p(seg_qn), _p(seg_ctx),
         _p(block_table), I(block_table.shape[1]), _p(items), I(n_items), I(n_heads), I(n_kv_heads),
-        I(head_dim), I(page_tokens), I(window), F(scale), I(keep_first), *_sink_args(sink, n_heads), _stream()
+        I(head_dim), I(page_tokens), I(window), I(chunk), F(scale), I(keep_first), *_sink_args(sink, n_heads), _stream()
     )
     _check(code, "attn_chunk", f"(heads {n_heads}/{n_kv_heads}, head_dim {head_dim})")
 
@@ -682,7 +733,7 @@ def attn_chunk_mma(q: torch.Tensor, pool: torch.Tensor, out: torch.Tensor, *, se
                    items: torch.Tensor, n_items: int, n_heads: int, n_kv_heads: int, head_dim: int,
                    page_tokens: int, window: int, scale: float, n_splits: int = 1,
                    part_o: Optional[torch.Tensor] = None, part_ml: Optional[torch.Tensor] = None,
-                   keep_first: int = 0, sink=False) -> None:
+                   keep_first: int = 0, sink=False, chunk: int = 0) -> None:
     """Attention of portions of prompts on the tensor cores: ``items`` [n_items, 2] =
     (segment, first query of a 64-query tile); otherwise as :func:`attn_chunk`.  ``n_splits`` > 1
     (:func:`attn_chunk_mma_splits`) with scratch of :func:`attn_chunk_mma_scratch` floats: the keys of
@@ -700,7 +751,7 @@ def attn_chunk_mma(q: torch.Tensor, pool: torch.Tensor, out: torch.Tensor, *, se
               "attn_chunk_mma: scratch too small for these ranges")
     code = _lib("attention_mma").locus_attn_chunk_mma(
         _p(q), _p(pool), _p(out), _p(seg_q0), _p(seg_qn), _p(seg_ctx), _p(block_table), I(block_table.shape[1]),
-        _p(items), I(n_items), I(n_heads), I(n_kv_heads), I(head_dim), I(page_tokens), I(window), F(scale),
+        _p(items), I(n_items), I(n_heads), I(n_kv_heads), I(head_dim), I(page_tokens), I(window), I(chunk), F(scale),
         I(n_splits), _p(part_o if n_splits > 1 else None), _p(part_ml if n_splits > 1 else None), I(keep_first),
         *_sink_args(sink, n_heads), _stream()
     )
@@ -755,13 +806,13 @@ def attn_chunk_tc(q: torch.Tensor, pool: torch.Tensor, out: torch.Tensor, *, seg
                   items: torch.Tensor, n_items: int, n_heads: int, n_kv_heads: int, head_dim: int,
                   page_tokens: int, window: int, scale: float, n_splits: int = 1,
                   part_o: Optional[torch.Tensor] = None, part_ml: Optional[torch.Tensor] = None,
-                  keep_first: int = 0, sink=False) -> None:
+                  keep_first: int = 0, sink=False, chunk: int = 0) -> None:
     """Attention of portions of prompts with tcgen05 tensor cores (scores and sums in tensor memory):
     ``items`` as for :func:`attn_chunk_mma` (tiles of 64 queries; a block takes an even one and the 64 queries
     behind it).  ``n_splits`` > 1 (:func:`attn_chunk_tc_splits`) with scratch of :func:`attn_chunk_tc_scratch`
     floats: the key tiles of every block are cut into that many ranges, merged in ascending order by a second
     kernel.  ``keep_first`` (with a window): a request's first tokens stay in sight; ``sink``: one more term of score 0
-    in the softmax's denominator."""
+    in the softmax's denominator; ``chunk`` as for :func:`attn_chunk`."""
     _cuda_c(q, "q")
     _cuda_c(out, "out")
     _cuda_c(pool, "pool")
@@ -778,7 +829,7 @@ def attn_chunk_tc(q: torch.Tensor, pool: torch.Tensor, out: torch.Tensor, *, seg
     code = _lib("attention_tc").locus_attn_chunk_tc(
         _p(q), LL(q.shape[0]), _p(pool), LL(pool.shape[0]), _p(out), _p(seg_q0), _p(seg_qn), _p(seg_ctx),
         _p(block_table), I(block_table.shape[1]), _p(items), I(n_items), I(n_heads), I(n_kv_heads), I(head_dim),
-        I(page_tokens), I(window), F(scale), I(n_splits), _p(part_o if n_splits > 1 else None),
+        I(page_tokens), I(window), I(chunk), F(scale), I(n_splits), _p(part_o if n_splits > 1 else None),
         _p(part_ml if n_splits > 1 else None), I(keep_first if window > 0 else 0), *_sink_args(sink, n_heads), _stream()
     )
     if n_splits > 1 and code == 0:
@@ -884,8 +935,8 @@ def attn_decode(q: torch.Tensor, pool: torch.Tensor, out: torch.Tensor, *, seg_q
                 items: torch.Tensor, n_items: int, n_heads: int, n_kv_heads: int, head_dim: int,
                 page_tokens: int, window: int, scale: float, part_o: torch.Tensor,
                 part_ml: torch.Tensor, counters: torch.Tensor, max_splits: int, keep_first: int = 0,
-                sink=False) -> None:
-    """Attention of single new tokens: ``items`` [n_items] = segments with one new token.  ``keep_first``, ``sink``
+                sink=False, chunk: int = 0) -> None:
+    """Attention of single new tokens: ``items`` [n_items] = segments with one new token.  ``keep_first``, ``sink``, ``chunk``
     as for :func:`attn_chunk` (the streaming kernels, per head and per group of query heads, walk the kept tokens in front
     of the window as one more range of the request and want scratch for two ranges per request and head, the kernel whose
     ranges are fixed for ``max_splits``: :func:`decode_units` with ``fixed_ranges``).
@@ -911,7 +962,7 @@ def attn_decode(q: torch.Tensor, pool: torch.Tensor, out: torch.Tensor, *, seg_q
         # several query heads per key/value head: the kernel that reads every cache row once for its whole group
         code = _lib("attention_gqa").locus_attn_decode_gqa(
             _p(q), _p(pool), _p(out), _p(seg_q0), _p(seg_ctx), _p(block_table), I(block_table.shape[1]), _p(items),
-            I(n_items), I(n_heads), I(n_kv_heads), I(head_dim), I(page_tokens), I(window), F(scale), _p(part_o),
+            I(n_items), I(n_heads), I(n_kv_heads), I(head_dim), I(page_tokens), I(window), I(chunk), F(scale), _p(part_o),
             _p(part_ml), _p(counters), ctypes.c_longlong(max_units), I(GQA_COST_RANGE),
             I(GQA_COST_MERGE_PER_HEAD * (n_heads // n_kv_heads)), I(keep_first if window > 0 else 0), *_sink_args(sink, n_heads),
             _stream()
@@ -921,7 +972,7 @@ def attn_decode(q: torch.Tensor, pool: torch.Tensor, out: torch.Tensor, *, seg_q
     code = _lib("attention").locus_attn_decode(
         _p(q), I(dtype_code(q.dtype)), _p(pool), _p(out), _p(seg_q0), _p(seg_qn), _p(seg_ctx),
         _p(block_table), I(block_table.shape[1]), _p(items), I(n_items), I(n_heads), I(n_kv_heads),
-        I(head_dim), I(page_tokens), I(window), F(scale), _p(part_o), _p(part_ml), _p(counters), I(max_splits),
+        I(head_dim), I(page_tokens), I(window), I(chunk), F(scale), _p(part_o), _p(part_ml), _p(counters), I(max_splits),
         ctypes.c_longlong(max_units), I(keep_first if window > 0 else 0), *_sink_args(sink, n_heads), _stream()
     )
     _check(code, "attn_decode", f"(heads {n_heads}/{n_kv_heads}, head_dim {head_dim})")
@@ -1677,7 +1728,7 @@ def ssm_out(y: torch.Tensor, act: torch.Tensor, proj: torch.Tensor, off_z: int, 
 
 PREP_MAX_TAPS = 16
 PREP_MAX_DIM = 256
-HEAD_NORMS = {None: 0, "rms": 1, "unit": 2}
+HEAD_NORMS = {None: 0, "rms": 1, "unit": 2, "head": 3}
 
 
 def head_prep(proj: torch.Tensor, *, offsets, heads, dims, laid, state_slots: torch.Tensor, seg_q0: torch.Tensor,
@@ -1687,7 +1738,7 @@ def head_prep(proj: torch.Tensor, *, offsets, heads, dims, laid, state_slots: to
               write_kv: bool = True, conv: Optional[torch.Tensor] = None, state: Optional[torch.Tensor] = None,
               conv_offset: int = 0, move_state: bool = True, act: bool = False,
               inv_freq: Optional[torch.Tensor] = None, rot: int = 0, norm: Optional[str] = None, eps: float = 0.0,
-              q_scale: float = 1.0, gates=None) -> None:
+              q_scale: float = 1.0, gates=None, interleaved: bool = False, norm_weights=None) -> None:
     """From the float32 rows ``proj`` of a stacked projection to q in rows and k, v in rows or cache pages, in one
     launch.  ``offsets``, ``heads``, ``dims``, ``laid``: for q, k, v the first column in ``proj``, the number of heads,
     the per-head size and the size a head is laid out at in the output (zeros behind its own elements).  In this
@@ -1696,7 +1747,9 @@ def head_prep(proj: torch.Tensor, *, offsets, heads, dims, laid, state_slots: to
     first token come from the request's slot of ``state`` ([channels, taps - 1] floats from ``conv_offset`` on;
     moved on by the portion's tokens in the same call unless ``move_state`` is off); ``act``: silu; ``inv_freq``
     [rot / 2]: q's and k's pairs (i, i + rot / 2) rotated by position * inv_freq[i]; ``norm`` "rms": q and k divided
-    by sqrt(mean(x^2) + eps) per head, "unit": by sqrt(sum(x^2) + eps); ``q_scale`` on q.  The outputs share one
+    by sqrt(mean(x^2) + eps) per head, "unit": by sqrt(sum(x^2) + eps), "head": by sqrt(mean(x^2) + eps) and multiplied by
+    ``norm_weights`` = (q's, k's) [dim] in FRONT of the rotation; ``interleaved``: the rotation takes the pairs (2i, 2i + 1)
+    instead; ``q_scale`` on q.  The outputs share one
     element type; with ``pool`` (a layer's pages [n_pages, 2, heads_k, page_tokens, laid]) k and v go to ``slots``.
     ``gates`` = (beta, decay, off_b, off_a, a_log, dt_bias): also beta = sigmoid(proj[:, off_b + h]) and decay =
     exp(-exp(a_log[h]) * softplus(proj[:, off_a + h] + dt_bias[h])), [T, heads] float32 each."""
@@ -1728,6 +1781,10 @@ def head_prep(proj: torch.Tensor, *, offsets, heads, dims, laid, state_slots: to
             state_ptr, stride = ctypes.c_void_p(state.data_ptr() + 4 * conv_offset), state.stride(0)
     if inv_freq is not None:
         _need(inv_freq.dtype == torch.float32 and inv_freq.is_cuda and inv_freq.numel() == rot // 2, "head_prep: inv_freq [rot / 2]")
+    q_w, k_w = norm_weights if norm_weights is not None else (None, None)
+    _need((norm == "head") == (q_w is not None), "head_prep: norm_weights go with the norm 'head'")
+    for t, which in ((q_w, 0), (k_w, 1)):
+        _need(t is None or (t.is_cuda and t.is_contiguous() and t.numel() == dims[which] and t.dtype == q_w.dtype), "head_prep: norm_weights [dim]")
     beta = decay = a_log = dt_bias = None
     off_b = off_a = gate_heads = gate_dt = 0
     if gates is not None:
@@ -1740,7 +1797,8 @@ def head_prep(proj: torch.Tensor, *, offsets, heads, dims, laid, state_slots: to
     code = _lib("short_conv").locus_head_prep(
         _p(proj), I(proj.stride(0)), sizes, _p(conv), I(dtype_code(conv.dtype) if conv is not None else 0), I(taps),
         I(1 if act else 0), state_ptr, LL(stride), I(1 if move_state else 0), _p(state_slots), _p(seg_q0), _p(seg_qn),
-        I(n_seg), I(longest_new), _p(positions), _p(inv_freq), I(rot if inv_freq is not None else 0), I(HEAD_NORMS[norm]),
+        I(n_seg), I(longest_new), _p(positions), _p(inv_freq), I(rot if inv_freq is not None else 0),
+        I(1 if interleaved else 0), I(HEAD_NORMS[norm]), _p(q_w), _p(k_w), I(dtype_code(q_w.dtype) if q_w is not None else 0),
         F(eps), F(q_scale), _p(q_out), _p(k_out), _p(v_out), _p(pool), _p(slots), I(page_tokens), I(1 if write_kv else 0),
         I(dtype_code(out_dt)), _p(beta), _p(decay), I(off_b), I(off_a), I(gate_heads), _p(a_log), _p(dt_bias), I(gate_dt),
         _stream())

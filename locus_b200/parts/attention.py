@@ -25,7 +25,9 @@ and v directly behind the projection (``conv_taps``; the last taps - 1 projected
 and k divided by their root mean square per head behind the rotation (``qk_norm`` "rms"), or an RMS norm with weights over
 the whole q and the whole k projection, all heads at once, in front of the rotation (``qk_norm`` "whole"); the heads' outputs multiplied by
 sigmoid(W_g h) in front of the output projection (``out_gate``); a layer without keys and values of its own
-(``has_kv`` off: it reads the cache of the layer call that the run order names).  With any of these (or ``shaped``)
+(``has_kv`` off: it reads the cache of the layer call that the run order names); an RMS norm per head with a weight that
+the heads share, in front of the rotation (``qk_norm`` "head"); a mask of chunks in the place of a window (``chunk``: a query
+sees the keys of its own chunk of that many positions, counted from position 0, up to itself).  With any of these (or ``shaped``)
 the projections are one product into float32 rows [q | k | v | gate] at the stored sizes, and one kernel
 (``kernels.head_prep``) convolves, rotates, norms and writes q and the cache pages at the kernels' head size in
 float32 arithmetic, so that padded heads take a rotation there too.
@@ -86,6 +88,7 @@ NAMES = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": 
          "q_bias": "q_proj.bias", "k_bias": "k_proj.bias", "v_bias": "v_proj.bias", "o_bias": "o_proj.bias",
          "q_conv": "q_proj.conv", "k_conv": "k_proj.conv", "v_conv": "v_proj.conv", "gate": "g_proj.weight",
          "sink": "sink", "q_norm": "q_norm.weight", "k_norm": "k_norm.weight"}
+QK_NORMS = (None, "rms", "unit", "whole", "head")
 
 
 class Attention(Mixer):
@@ -97,11 +100,11 @@ class Attention(Mixer):
                  v_dim: Optional[int] = None, out_scale: float = 1.0, names: Optional[dict] = None,
                  keep_first: int = 0, sink: bool = False, conv_taps: int = 0, qk_norm: Optional[str] = None,
                  qk_norm_eps: float = 0.0, out_gate: bool = False, has_kv: bool = True, shaped: bool = False,
-                 cache_window: Optional[int] = None, cache_keep: Optional[int] = None) -> None:
+                 cache_window: Optional[int] = None, cache_keep: Optional[int] = None, chunk: int = 0) -> None:
         """``v_dim``: the values' size per head where it is not ``head_dim``.  ``out_scale``: a factor on the mixer's
         output (a mixer that runs beside another one).  ``names``: tensor names below the prefix where they differ
-        from ``NAMES``.  ``keep_first``, ``sink``, ``conv_taps``, ``qk_norm`` ("rms"), ``out_gate``, ``has_kv``,
-        ``shaped``: see the head of the file.  ``cache_window`` / ``cache_keep``: what the layer's pages must hold
+        from ``NAMES``.  ``keep_first``, ``sink``, ``conv_taps``, ``qk_norm``, ``out_gate``, ``has_kv``,
+        ``shaped``, ``chunk``: see the head of the file.  ``cache_window`` / ``cache_keep``: what the layer's pages must hold
         where that is more than its own window and kept tokens (another layer call reads them with a wider mask)."""
         super().__init__(prefix)
         self.keep_first, self.sink = (int(keep_first) if window else 0), bool(sink)
@@ -115,8 +118,11 @@ class Attention(Mixer):
             raise ValueError("attention: a norm over the whole projections does not go with a convolution behind them")
         if self.conv_taps > K.PREP_MAX_TAPS:
             raise ValueError(f"attention: a convolution over {conv_taps} tokens (at most {K.PREP_MAX_TAPS})")
-        if qk_norm not in (None, "rms", "unit", "whole"):
-            raise ValueError(f"attention: qk_norm {qk_norm!r} (known: rms, unit, whole)")
+        if qk_norm not in QK_NORMS:
+            raise ValueError(f"attention: qk_norm {qk_norm!r} (known: {', '.join(QK_NORMS[1:])})")
+        self.chunk = int(chunk)
+        if self.chunk < 0 or (self.chunk and (window or cache_window)):
+            raise ValueError(f"attention: a window of {window or cache_window} beside chunks of {chunk} (one or the other)")
         self.cache_window = int(window if cache_window is None else cache_window)
         self.cache_keep = int(self.keep_first if cache_keep is None else cache_keep) if self.cache_window else 0
         if n_heads % n_kv_heads:
@@ -189,14 +195,15 @@ class Attention(Mixer):
         return shapes
 
     def _extra_shapes(self):
-        """A learned sink per query head; the weights of a norm over the whole q and k projections."""
+        """A learned sink per query head; the weights of a norm over the whole q and k projections or over their heads."""
         s = {}
         if self.sink_learned:
             s["sink"] = (self.n_heads,)
-        if self.qk_norm == "whole":
-            s["q_norm"] = (self.n_heads * self.qk_dim,)
+        if self.qk_norm in ("whole", "head"):
+            shared = self.qk_norm == "head"   # one head's weight for all of them
+            s["q_norm"] = (self.qk_dim * (1 if shared else self.n_heads),)
             if self.has_kv:
-                s["k_norm"] = (self.n_kv_heads * self.qk_dim,)
+                s["k_norm"] = (self.qk_dim * (1 if shared else self.n_kv_heads),)
         return s
 
     def _extra_sources(self):
@@ -286,7 +293,7 @@ class Attention(Mixer):
         state = None
         if self.conv_taps > 1:
             state = StateSpec((self.channels * (self.conv_taps - 1),), torch.float32)
-        return PagedKvSpec(self.n_kv_heads, self.head_dim, self.cache_window, keep_first=self.cache_keep), state
+        return PagedKvSpec(self.n_kv_heads, self.head_dim, self.cache_window, keep_first=self.cache_keep, chunk=self.chunk), state
 
     def step_plans(self):
         return [AttentionTiles()]
@@ -298,8 +305,8 @@ class Attention(Mixer):
         proj = rt.rows(f"attention.proj{self.in_width}", self.in_width, torch.float32, T)
         K.linear(h, self.params["w_in"], proj, bias=self.params.get("b_in"))
         table = self.position.rotary_table()
-        if table is not None and (table.magnitude != 1.0 or table.interleaved):
-            raise ValueError("attention: the shaped form rotates half-split pairs without a factor on cosine and sine")
+        if table is not None and table.magnitude != 1.0:
+            raise ValueError("attention: the shaped form rotates without a factor on cosine and sine")
         if self.conv_taps > 1 and not cache.writes:
             raise ValueError("attention: a layer call that reads another call's cache has no convolution state of its own")
         q = rt.rows("attention.q", self.q_dim, rt.dtype, T)
@@ -317,8 +324,9 @@ class Attention(Mixer):
                     pool=cache.pool if kv else None, slots=gb.slots if kv else None, page_tokens=gb.page_tokens,
                     write_kv=cache.writes, conv=self.params.get("conv"), state=cache.state if self.conv_taps > 1 else None,
                     inv_freq=table.inv_freq if table else None, rot=table.rot_dim if table else 0,
-                    norm=None if self.qk_norm == "whole" else self.qk_norm,
-                    eps=self.qk_norm_eps)
+                    interleaved=table.interleaved if table else False,
+                    norm=None if self.qk_norm == "whole" else self.qk_norm, eps=self.qk_norm_eps,
+                    norm_weights=(self.params["q_norm"], self.params.get("k_norm")) if self.qk_norm == "head" else None)
         o = rt.rows("attention.o", self.q_dim, rt.dtype, T)
         self._attend(q, o, batch, cache, gb, rt)
         if self.out_gate:
@@ -355,6 +363,8 @@ class Attention(Mixer):
         T = batch.T
         special = bool(self.keep_first or self.sink)
         extra = dict(keep_first=self.keep_first, sink=self._sink_arg) if special else {}
+        if self.chunk:
+            extra["chunk"] = self.chunk
         common = dict(seg_q0=batch.seg_q0, seg_qn=batch.seg_qn, seg_ctx=batch.seg_ctx,
                       block_table=gb.block_table, n_heads=self.n_heads, n_kv_heads=self.n_kv_heads,
                       head_dim=self.head_dim, page_tokens=gb.page_tokens, window=self.window,
@@ -367,8 +377,8 @@ class Attention(Mixer):
         if tiles["n_chunk_items"]:
             # few query tiles behind a long context: the keys of every tile are cut into ranges
             keys = max_splits * K.DECODE_SPLIT
-            if self.window > 0:
-                keys = min(keys, self.window + self.keep_first + K.TC_ATTN_QUERY_BLOCK)
+            if self.window > 0 or self.chunk > 0:
+                keys = min(keys, (self.window or self.chunk) + self.keep_first + K.TC_ATTN_QUERY_BLOCK)
             if K.attn_chunk_tc_takes(q, self.head_dim, gb.page_tokens, T, keys):
                 n_splits = K.attn_chunk_tc_splits(tiles["n_chunk_items64"], self.n_heads, keys)
                 part_o = part_ml = None

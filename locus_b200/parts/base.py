@@ -103,7 +103,9 @@ class PagedKvSpec:
     and ``extra_width`` further elements per token in a tensor of their own (per-token fields beside the
     rows, as the reference appends them to its cache row, src/locus/model/arch.cpp:539-542).  ``window`` > 0:
     only the last ``window`` tokens are kept; pages behind the window go back while the request lives, except
-    those that hold the request's first ``keep_first`` tokens, which such a window keeps in sight."""
+    those that hold the request's first ``keep_first`` tokens, which such a window keeps in sight.  ``chunk`` > 0
+    (without a window): a query sees the keys of its own chunk of that many positions, counted from position 0, and
+    pages behind the chunk go back."""
 
     n_kv_heads: int
     head_dim: int
@@ -111,6 +113,7 @@ class PagedKvSpec:
     has_v: bool = True
     extra_width: int = 0
     keep_first: int = 0
+    chunk: int = 0
 
     @property
     def planes(self) -> int:
@@ -156,10 +159,17 @@ class Part:
         return []
 
 
-class PendingAdd:
-    """An addition to the residual stream that a feed-forward left undone so that the next norm can
-    fold it into its own pass over the rows: x[t] += sum over slots of pair_out[pair_pos[t * k + slot]].
-    Whoever takes it from the runtime must either hand it to a norm that folds it or ``apply`` it."""
+class Pending:
+    """An addition to the residual stream that was left undone so that the next norm can fold it into its own pass over
+    the rows.  Whoever takes it from the runtime must either hand it to a norm (which folds it when it knows its kind) or
+    ``apply`` it."""
+
+    def apply(self, x: torch.Tensor) -> None:
+        raise NotImplementedError
+
+
+class PendingAdd(Pending):
+    """What a routed feed-forward leaves: x[t] += sum over slots of pair_out[pair_pos[t * k + slot]]."""
 
     def __init__(self, pair_out: torch.Tensor, pair_pos: torch.Tensor, top_k: int) -> None:
         self.pair_out, self.pair_pos, self.top_k = pair_out, pair_pos, top_k
@@ -170,18 +180,28 @@ class PendingAdd:
         K.moe_combine(x, self.pair_out, self.pair_pos, self.top_k)
 
 
+class PendingNorm(Pending):
+    """What an arrangement with norms behind its sublayers leaves: x += scale * norm(y) (``scale`` [width] or None)."""
+
+    def __init__(self, y: torch.Tensor, norm: "Norm", scale: Optional[torch.Tensor]) -> None:
+        self.y, self.norm, self.scale = y, norm, scale
+
+    def apply(self, x: torch.Tensor) -> None:
+        self.norm.forward_add(self.y, x, self.scale)
+
+
 class Norm(Part):
     def forward(self, x: torch.Tensor, out: torch.Tensor, rows: Optional[torch.Tensor] = None,
-                add: Optional[PendingAdd] = None) -> None:
+                add: Optional[Pending] = None) -> None:
         """out = norm(x) (rows: gather of x rows); statistics in float32.  ``add``: a pending
         addition to x that must be done (in x) before the norm: fold it in or call ``add.apply(x)``.
         A caller that gives ``rows`` as well reads x no more afterwards, so the addition then only
         has to show in ``out``."""
         raise NotImplementedError
 
-    def forward_add(self, y: torch.Tensor, x: torch.Tensor) -> None:
+    def forward_add(self, y: torch.Tensor, x: torch.Tensor, scale: Optional[torch.Tensor] = None) -> None:
         """x += norm(y) for float32 rows y of a sublayer's output (arrangements that norm what a sublayer
-        gives instead of what it reads)."""
+        gives instead of what it reads); ``scale`` [width]: x += scale * norm(y)."""
         raise NotImplementedError
 
 

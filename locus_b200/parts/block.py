@@ -13,6 +13,9 @@ and mixed among themselves at every write-back (below).
 ``PostNorm``: x <- norm1(alpha x + mixer(x)); x <- norm2(alpha x + feed_forward(x)): the sublayers read x itself and the
 norm sits on the sum.
 
+``SandwichNorm``: x += s1 * norm1b(mixer(norm1(x))); x += s2 * norm2b(feed_forward(norm2(x))): norms on both sides of a
+sublayer and optional layer scales.
+
 ``Embedding``: x = table[token] (llama.cpp:450); optionally plus a row of a second table addressed by a hash of the
 previous and the current token.  ``LmHead``: logits = W . h in float32,
 W being the embedding table when the head is tied (llama.cpp:292-297, 512-513): the head then
@@ -25,8 +28,9 @@ from typing import Optional
 import torch
 
 from .. import kernels as K
-from .base import (Arrangement, Part, PartSpec, StateSpec, TensorSource, make_part, register_arrangement,
+from .base import (Arrangement, Part, PartSpec, PendingNorm, StateSpec, TensorSource, make_part, register_arrangement,
                    register_embedding, register_head)
+from .norm import DynamicTanh
 
 
 class PreNorm(Arrangement):
@@ -175,6 +179,74 @@ class PostNorm(Arrangement):
             rt._post_norm_rows = x   # block.h holds x's rounding for the block behind this one
 
 
+class SandwichNorm(Arrangement):
+    """Norms in front of and behind every sublayer: x += s1 * norm1b(mixer(norm1(x))); x += s2 * norm2b(ff(norm2(x))).
+    s1, s2 [hidden] are the layer scales (``scale_names``; empty: none).  The sublayers write float32 rows.  The addition
+    behind a sublayer is handed to the norm in front of the next one (:class:`PendingNorm`: the second norm of the block,
+    the first of the next block, the final norm), which folds it into its own pass where it can.  ``feed_forward`` may be
+    absent (kind "none"): the layer is then its mixer alone, with its two norms and one scale."""
+
+    takes_pending_add = True
+
+    def __init__(self, prefix: str, *, hidden: int, norm: PartSpec, mixer: PartSpec, feed_forward: PartSpec,
+                 mixer_prefix: str = "mix", ff_prefix: str = "mlp", norm_names: tuple = ("norm1", "norm1b", "norm2", "norm2b"),
+                 scale_names: tuple = (), tensor_suffixes: Optional[dict] = None) -> None:
+        """``norm_names``: in front of and behind the mixer, in front of and behind the feed-forward.
+        ``tensor_suffixes``: the norm's arguments that name its tensors -> what stands behind ``<prefix>.<norm name>`` in
+        them (default: the plain name as ``tensor``)."""
+        super().__init__(prefix)
+        self.hidden = int(hidden)
+        suffixes = {"tensor": ""} if tensor_suffixes is None else tensor_suffixes
+
+        def norm_part(name):
+            named = {arg: f"{prefix}.{name}{suffix}" for arg, suffix in suffixes.items()}
+            return make_part("norm", PartSpec(norm.kind, {**norm.args, **named}), f"{prefix}.{name}")
+
+        self.norm1, self.norm1b = norm_part(norm_names[0]), norm_part(norm_names[1])
+        self.mixer = make_part("mixer", mixer, f"{prefix}.{mixer_prefix}")
+        self.ff = None if feed_forward.kind == "none" else make_part("feed_forward", feed_forward, f"{prefix}.{ff_prefix}")
+        self.norm2, self.norm2b = (norm_part(norm_names[2]), norm_part(norm_names[3])) if self.ff is not None else (None, None)
+        self.scale_names = tuple(scale_names)[: 2 if self.ff is not None else 1]
+
+    def sub_parts(self):
+        return [self.norm1, self.mixer, self.norm1b] + ([self.norm2, self.ff, self.norm2b] if self.ff is not None else [])
+
+    def param_shapes(self):
+        return {n: (self.hidden,) for n in self.scale_names}
+
+    def sources(self):
+        return [TensorSource(f"{self.prefix}.{n}", (self.hidden,), n, 0, "norm") for n in self.scale_names]
+
+    def _scale(self, i):
+        return self.params[self.scale_names[i]] if i < len(self.scale_names) else None
+
+    def forward(self, x, batch, cache, rt) -> None:
+        T = batch.T
+        defer, rt.defer_add = rt.defer_add, False   # (the sublayers write whole rows: nothing of theirs may be left pending)
+        h = rt.rows("block.h", self.hidden, rt.dtype, T)
+        y = rt.rows("block.y", self.hidden, torch.float32, T)
+        self.norm1.forward(x, h, add=rt.take_pending())
+        if self.mixer.can_overwrite:
+            self.mixer.forward(h, batch, cache, y, rt, accumulate=False)
+        else:
+            y.zero_()
+            self.mixer.forward(h, batch, cache, y, rt)
+        left = PendingNorm(y, self.norm1b, self._scale(0))
+        if self.ff is not None:
+            self.norm2.forward(x, h, add=left)
+            if self.ff.can_overwrite:
+                self.ff.forward(h, batch, y, rt, accumulate=False)
+            else:
+                y.zero_()
+                self.ff.forward(h, batch, y, rt)
+            left = PendingNorm(y, self.norm2b, self._scale(1))
+        rt.defer_add = defer
+        if defer:
+            rt.leave_pending(left)
+        else:
+            left.apply(x)
+
+
 class StreamedPreNorm(Arrangement):
     """Pre-norm sublayers over ``streams`` copies x_1 .. x_S of the residual stream (a row of x holds them one behind
     the other).  For sublayer q (1: the mixer, 2: the feed-forward) with its own read weights a [S], write weights b
@@ -273,14 +345,18 @@ class StreamedPreNorm(Arrangement):
 
 class Embedding(Part):
     def __init__(self, prefix: str, *, vocab: int, hidden: int, tensor: str = "", copies: int = 1,
-                 scale: float = 1.0, pair: Optional[dict] = None) -> None:
+                 scale: float = 1.0, pair: Optional[dict] = None, norm: Optional[PartSpec] = None) -> None:
         """``tensor``: the checkpoint tensor's name where it is not ``<prefix>.weight``.  ``copies`` > 1: a row of the
         output holds the embedding that many times (a model with several copies of the residual stream).  ``scale``:
         a factor on the embedding, applied in float32.  ``pair`` = {tensor, buckets, mul_prev, mul_cur}: a second table
         of buckets + 1 rows whose row (previous token * mul_prev + token * mul_cur) mod buckets is added (its last row for
         a request's first token).  The token that a request's last step ended on is kept in the request's state slot
-        (``state_needs``), so that a prompt may be cut anywhere."""
+        (``state_needs``), so that a prompt may be cut anywhere.  ``norm``: a norm over the row behind all of this (the
+        residual stream then starts from its float32 result)."""
         super().__init__(prefix)
+        self.norm = make_part("norm", norm, prefix + ".norm") if norm is not None else None
+        if self.norm is not None and int(copies) != 1:
+            raise ValueError("embedding: a norm behind the embedding goes with one copy")
         self.vocab, self.hidden, self.copies, self.scale = int(vocab), int(hidden), int(copies), float(scale)
         self.tensor = str(tensor or prefix + ".weight")
         self.pair = dict(pair) if pair else None
@@ -305,6 +381,9 @@ class Embedding(Part):
     def kernel_modules(self, dtype):
         return ["elementwise"]
 
+    def sub_parts(self):
+        return [self.norm] if self.norm is not None else []
+
     def state_needs(self) -> Optional[StateSpec]:
         """What the embedding keeps per request: the last token it saw, when it has a pair table."""
         return StateSpec((1,), torch.int32) if self.pair is not None else None
@@ -317,19 +396,30 @@ class Embedding(Part):
                          seg_qn=batch.seg_qn, state_slots=batch.state_slots, last=cache.state, n_seg=batch.n_seg,
                          longest_new=max(batch.host_seg_qn) if batch.host_seg_qn else batch.T,
                          mul_prev=int(self.pair["mul_prev"]), mul_cur=int(self.pair["mul_cur"]))
+            if self.norm is not None:
+                self.norm.forward(out, out)
+            return
+        if isinstance(self.norm, DynamicTanh):
+            K.embed_rows(tokens, self.params["table"], out, scale=self.scale, dyt_norm=self.norm.tensors())
             return
         if self.copies > 1 or self.scale != 1.0:
             K.embed_rows(tokens, self.params["table"], out, copies=self.copies, scale=self.scale)
         else:
             K.embed_rows(tokens, self.params["table"], out)
+        if self.norm is not None:
+            self.norm.forward(out, out)
 
 
 class LmHead(Part):
     """``tied_to``: the checkpoint tensor that is the head's weight when the head has none of its own
-    (the embedding table of a tied model); two parts that name the same tensor share one device copy."""
+    (the embedding table of a tied model); two parts that name the same tensor share one device copy.  ``scale``: a factor
+    on the logits; ``softcap`` > 0: logits <- softcap * tanh(logits / softcap) behind it, both in the product's epilogue."""
 
-    def __init__(self, prefix: str, *, vocab: int, hidden: int, tied_to: str = "", tensor: str = "") -> None:
+    def __init__(self, prefix: str, *, vocab: int, hidden: int, tied_to: str = "", tensor: str = "", scale: float = 1.0,
+                 softcap: float = 0.0) -> None:
         super().__init__(prefix)
+        self.scale, self.softcap = float(scale), float(softcap)
+        self._row_scale = None
         self.vocab, self.hidden, self.tied_to = int(vocab), int(hidden), str(tied_to or "")
         self.tensor = str(tensor or prefix + ".weight")   # the head's own tensor, when it is not tied
 
@@ -342,13 +432,21 @@ class LmHead(Part):
     def kernel_modules(self, dtype):
         return ["gemm_simt", "gemv"] + (["gemm_skinny", "gemm_tc"] if dtype == torch.bfloat16 else [])
 
+    def bind(self, rt) -> None:
+        if self.scale != 1.0 and not self.softcap > 0:
+            self._row_scale = torch.full((rt.max_wanted,), self.scale, dtype=torch.float32, device=rt.device)
+
     def forward(self, h: torch.Tensor, logits: torch.Tensor) -> None:
-        K.linear(h, self.params["weight"], logits)
+        if self.softcap > 0:
+            K.linear(h, self.params["weight"], logits, act="softcap", act_limit=self.softcap, act_scale=self.scale)
+        else:
+            K.linear(h, self.params["weight"], logits, row_scale=self._row_scale)
 
 
 register_arrangement("pre_norm", PreNorm)
 register_arrangement("output_norm", OutputNorm)
 register_arrangement("streamed_pre_norm", StreamedPreNorm)
 register_arrangement("post_norm", PostNorm)
+register_arrangement("sandwich_norm", SandwichNorm)
 register_embedding("embedding", Embedding)
 register_head("linear", LmHead)

@@ -15,7 +15,12 @@ index i: with turns(t) = rot_dim * ln(original / (2 pi t)) / (2 ln theta) (the i
 makes t turns over the original length), lo = max(floor(turns(fast)), 0), hi = min(ceil(turns(slow)),
 rot_dim - 1) and ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), the frequency of pair i becomes
 f_i / factor * ramp_i + f_i * (1 - ramp_i), and cosine and sine are both multiplied by
-0.1 * ln(factor) + 1 (the table's ``magnitude``).  The table also carries the frequencies in float64
+0.1 * ln(factor) + 1 (the table's ``magnitude``).
+
+``scaling`` = {factor, original, high, low} does it by wavelength instead, without a factor on cosine and sine: with
+t_i = original * f_i / (2 pi), the turns that pair i makes over the original length, f_i stays where t_i > high, becomes
+f_i / factor where t_i < low, and (1 - s) f_i / factor + s f_i with s = (t_i - low) / (high - low) between them (the
+frequency scaling of Llama 3.1).  The table also carries the frequencies in float64
 for kernels that form their angles in float64.
 """
 from __future__ import annotations
@@ -39,8 +44,10 @@ class Rotary(PositionEncoding):
         if self.rot_dim % 2 or not (0 < self.rot_dim <= self.head_dim):
             raise ValueError(f"rotary: rot_dim {self.rot_dim} must be even and within head_dim {self.head_dim}")
         self.scaling = dict(scaling) if scaling else None
+        self.by_wavelength = self.scaling is not None and "high" in self.scaling
         if self.scaling is not None:
-            missing = [k for k in ("factor", "original", "fast", "slow") if not float(self.scaling.get(k, 0)) > 0]
+            keys = ("factor", "original", "high", "low") if self.by_wavelength else ("factor", "original", "fast", "slow")
+            missing = [k for k in keys if not float(self.scaling.get(k, 0)) > 0]
             if missing:
                 raise ValueError(f"rotary: scaling needs positive {', '.join(missing)}")
         self._table: Optional[RotaryTable] = None
@@ -53,6 +60,12 @@ class Rotary(PositionEncoding):
         if self.scaling is None:
             return f
         sc = self.scaling
+        if self.by_wavelength:
+            high, low = float(sc["high"]), float(sc["low"])
+            made = f * (float(sc["original"]) / (2.0 * math.pi))
+            s = (made - low) / (high - low) if high != low else torch.ones_like(f)
+            slow = f / float(sc["factor"])
+            return torch.where(made > high, f, torch.where(made < low, slow, (1.0 - s) * slow + s * f))
 
         def turns(t: float) -> float:
             return n * math.log(float(sc["original"]) / (2.0 * math.pi * t)) / (2.0 * math.log(self.theta))
@@ -64,7 +77,7 @@ class Rotary(PositionEncoding):
 
     def magnitude(self) -> float:
         """What cosine and sine are multiplied by (1 without scaling)."""
-        return 1.0 if self.scaling is None else 0.1 * math.log(float(self.scaling["factor"])) + 1.0
+        return 1.0 if self.scaling is None or self.by_wavelength else 0.1 * math.log(float(self.scaling["factor"])) + 1.0
 
     def inv_freq_host(self) -> torch.Tensor:
         return self.frequencies().to(torch.float32)

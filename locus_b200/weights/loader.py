@@ -109,9 +109,9 @@ def load_weights(model, source) -> None:
                                                  device=model.device)
             filled.add(key)
         dest = part.params[src.param]
-        flat = dest.view(-1, dest.shape[-1]) if dest.dim() >= 2 else dest
+        flat = dest.view(-1, dest.shape[-1]) if dest.dim() >= 2 else dest.view(-1)
         t = source.tensor(src.name)
-        n0 = src.shape[0]
+        n0 = src.shape[0] if src.shape else 1   # (a scalar is one element)
         flat[src.row0 : src.row0 + n0].copy_(t.reshape(flat[src.row0 : src.row0 + n0].shape)
                                              .to(device=model.device, dtype=dest.dtype))
         if whole(part, src):

@@ -20,8 +20,29 @@ def _f(t: torch.Tensor) -> torch.Tensor:
     return t.to(torch.float64 if PRECISE else torch.float32)
 
 
-def embed_rows(tokens, table, out, copies=1, scale=1.0):
-    out.copy_((_f(table[tokens.long()]) * scale).to(out.dtype).repeat(1, copies))
+def embed_rows(tokens, table, out, copies=1, scale=1.0, dyt_norm=None):
+    rows = _f(table[tokens.long()]) * scale
+    if dyt_norm is not None:
+        rows = _dyt(rows, dyt_norm)
+    out.copy_(rows.to(out.dtype).repeat(1, copies))
+
+
+def _dyt(z, norm):
+    alpha, w, b = norm
+    return torch.tanh(_f(alpha) * z) * _f(w) + _f(b)
+
+
+def dyt(x, norm=None, out=None, rows=None, add=None):
+    n = x.shape[0] if out is None else out.shape[0]
+    pick = slice(0, n) if rows is None else rows.long()
+    u = _f(x[pick])
+    if add is not None:
+        y, y_norm, scale = add
+        u = u + (1.0 if scale is None else _f(scale)) * _dyt(_f(y[pick]), y_norm)
+        if rows is None:
+            x[:n] = u.to(x.dtype)
+    if out is not None:
+        out.copy_(_dyt(u, norm).to(out.dtype))
 
 
 def attn_chunk_tc_takes(q, head_dim, page_tokens, n_tokens, max_ctx=0):
@@ -49,9 +70,10 @@ class ExpertLayout(K.ExpertLayout):
 
 def linear(x, w, out, *, w2=None, bias=None, accumulate=False, row_scale=None, scale_rows=None, x_rows=None, lists_ready=False,
            second_tiles=False,
-           x_row_div=1, layout=None, n_rows=None, act=None, act_limit=0.0):
-    assert act in (None, "relu2", "glu_clamp") and not (act == "relu2" and w2 is not None)
+           x_row_div=1, layout=None, n_rows=None, act=None, act_limit=0.0, act_scale=1.0):
+    assert act in (None, "relu2", "glu_clamp", "softcap") and not (act == "relu2" and w2 is not None)
     assert act != "glu_clamp" or (w2 is not None and act_limit > 0)
+    assert act != "softcap" or (w2 is None and act_limit > 0)
     M = out.shape[0] if n_rows is None else n_rows
     if M == 0:
         return
@@ -92,6 +114,8 @@ def linear(x, w, out, *, w2=None, bias=None, accumulate=False, row_scale=None, s
         y = torch.clamp(y, min=0.0) ** 2
     if rs_all is not None and act != "glu_clamp":
         y = y * rs_all
+    if act == "softcap":
+        y = act_limit * torch.tanh(y * act_scale / act_limit)
     if layout is not None:
         M = min(M, int(layout.offsets[w.shape[0]]))   # a grouped product writes the rows of its experts only
         y = y[:M]
@@ -127,8 +151,8 @@ def rope_kv_write(qkv, positions, inv_freq, q_out, pool, slots, *, n_heads, n_kv
         pool[page, 1, :, off, :] = x[t, n_heads + n_kv_heads :].to(pool.dtype)
 
 
-def _attend_one(q, pool, table, p, kvh, page_tokens, window, scale, keep_first=0, sink=False, head=0):
-    lo = max(0, p - window + 1) if window > 0 else 0
+def _attend_one(q, pool, table, p, kvh, page_tokens, window, scale, keep_first=0, sink=False, head=0, chunk=0):
+    lo = max(0, p - window + 1) if window > 0 else (p - p % chunk if chunk > 0 else 0)
     ts = list(range(0, min(keep_first, lo))) + list(range(lo, p + 1))
     pages = [int(table[t // page_tokens]) for t in ts]
     assert all(pg >= 0 for pg in pages), "attention reads a page that was given back"
@@ -146,23 +170,24 @@ def _attend_one(q, pool, table, p, kvh, page_tokens, window, scale, keep_first=0
 
 
 def _attn(q, pool, out, seg_list, *, seg_q0, seg_qn, seg_ctx, block_table, n_heads, n_kv_heads, head_dim,
-          page_tokens, window, scale, keep_first=0, sink=False):
+          page_tokens, window, scale, keep_first=0, sink=False, chunk=0):
     group = n_heads // n_kv_heads
     for seg in seg_list:
         q0, qn, ctx = int(seg_q0[seg]), int(seg_qn[seg]), int(seg_ctx[seg])
         for i in range(qn):
             for h in range(n_heads):
                 qv = q[q0 + i].view(n_heads, head_dim)[h]
-                o = _attend_one(qv, pool, block_table[seg], ctx + i, h // group, page_tokens, window, scale, keep_first, sink, head=h)
+                o = _attend_one(qv, pool, block_table[seg], ctx + i, h // group, page_tokens, window, scale, keep_first, sink, head=h,
+                                chunk=chunk)
                 out[q0 + i].view(n_heads, head_dim)[h] = o.to(out.dtype)
 
 
 def attn_chunk(q, pool, out, *, seg_q0, seg_qn, seg_ctx, block_table, items, n_items, n_heads, n_kv_heads,
-               head_dim, page_tokens, window, scale, keep_first=0, sink=False):
+               head_dim, page_tokens, window, scale, keep_first=0, sink=False, chunk=0):
     segs = sorted({int(items[i, 0]) for i in range(n_items)})
     _attn(q, pool, out, segs, seg_q0=seg_q0, seg_qn=seg_qn, seg_ctx=seg_ctx, block_table=block_table,
           n_heads=n_heads, n_kv_heads=n_kv_heads, head_dim=head_dim, page_tokens=page_tokens, window=window,
-          scale=scale, keep_first=keep_first, sink=sink)
+          scale=scale, keep_first=keep_first, sink=sink, chunk=chunk)
 
 
 def attn_chunk_mma_splits(n_items, n_heads, max_ctx):
@@ -170,20 +195,20 @@ def attn_chunk_mma_splits(n_items, n_heads, max_ctx):
 
 
 def attn_chunk_mma(q, pool, out, *, seg_q0, seg_qn, seg_ctx, block_table, items, n_items, n_heads, n_kv_heads,
-                   head_dim, page_tokens, window, scale, n_splits=1, part_o=None, part_ml=None, keep_first=0, sink=False):
+                   head_dim, page_tokens, window, scale, n_splits=1, part_o=None, part_ml=None, keep_first=0, sink=False, chunk=0):
     attn_chunk(q, pool, out, seg_q0=seg_q0, seg_qn=seg_qn, seg_ctx=seg_ctx, block_table=block_table, items=items,
                n_items=n_items, n_heads=n_heads, n_kv_heads=n_kv_heads, head_dim=head_dim, page_tokens=page_tokens,
-               window=window, scale=scale, keep_first=keep_first, sink=sink)
+               window=window, scale=scale, keep_first=keep_first, sink=sink, chunk=chunk)
 
 
 def attn_decode(q, pool, out, *, seg_q0, seg_qn, seg_ctx, block_table, items, n_items, n_heads, n_kv_heads,
-                head_dim, page_tokens, window, scale, part_o, part_ml, counters, max_splits, keep_first=0, sink=False):
+                head_dim, page_tokens, window, scale, part_o, part_ml, counters, max_splits, keep_first=0, sink=False, chunk=0):
     segs = [int(items[i]) for i in range(n_items)]
     for s in segs:
         assert int(seg_ctx[s]) // K.DECODE_SPLIT + 1 <= max_splits
     _attn(q, pool, out, segs, seg_q0=seg_q0, seg_qn=seg_qn, seg_ctx=seg_ctx, block_table=block_table,
           n_heads=n_heads, n_kv_heads=n_kv_heads, head_dim=head_dim, page_tokens=page_tokens, window=window,
-          scale=scale, keep_first=keep_first, sink=sink)
+          scale=scale, keep_first=keep_first, sink=sink, chunk=chunk)
 
 
 def _select(logits_row, top_k, renorm, scale, score_fn, sel_bias, n_group, n_group_used, group_score="top2"):
@@ -617,7 +642,8 @@ def mlstm_out(o_raw, m_t, proj, off_g, w, eps, out, *, n_heads, v_dim):
 
 def head_prep(proj, *, offsets, heads, dims, laid, state_slots, seg_q0, seg_qn, n_seg, longest_new, positions, q_out,
               k_out=None, v_out=None, pool=None, slots=None, page_tokens=0, write_kv=True, conv=None, state=None,
-              conv_offset=0, move_state=True, act=False, inv_freq=None, rot=0, norm=None, eps=0.0, q_scale=1.0, gates=None):
+              conv_offset=0, move_state=True, act=False, inv_freq=None, rot=0, norm=None, eps=0.0, q_scale=1.0, gates=None,
+              interleaved=False, norm_weights=None):
     widths = [h * d for h, d in zip(heads, dims)]
     C = sum(widths)
     taps = conv.shape[1] if conv is not None else 1
@@ -649,13 +675,16 @@ def head_prep(proj, *, offsets, heads, dims, laid, state_slots, seg_q0, seg_qn, 
             at += H * d
             if H == 0 or (which > 0 and not write_kv):
                 continue
+            if which < 2 and norm == "head":
+                x = x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps) * _f(norm_weights[which])
             if which < 2 and inv_freq is not None and rot > 0:
                 ang = positions[rows].to(torch.float32)[:, None] * inv_freq[None, :].to(torch.float32)
                 c, s = _f(torch.cos(ang))[:, None, :], _f(torch.sin(ang))[:, None, :]
                 half = rot // 2
-                u, v = x[..., :half].clone(), x[..., half:rot].clone()
-                x[..., :half] = u * c - v * s
-                x[..., half:rot] = v * c + u * s
+                a, b = (slice(0, rot, 2), slice(1, rot, 2)) if interleaved else (slice(0, half), slice(half, rot))
+                u, v = x[..., a].clone(), x[..., b].clone()
+                x[..., a] = u * c - v * s
+                x[..., b] = v * c + u * s
             if which < 2 and norm == "rms":
                 x = x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps)
             elif which < 2 and norm == "unit":
@@ -753,7 +782,7 @@ _NAMES = ["embed_rows", "rmsnorm", "rmsnorm_adds", "attn_chunk_tc_takes", "linea
           "cast_rows", "rmsnorm_add", "latent_prep", "latent_q_split", "latent_attn", "heads_to_rows", "retention_scan",
           "retention_gate_norm", "head_tile", "latent_attn_mma_takes", "layernorm", "stream_update", "moe_identity",
           "gated_recurrence", "mlstm_gates", "mlstm_out", "ssm_conv", "ssm_out", "head_prep", "gate_rows", "delta_rule", "delta_out",
-          "embed_pair", "layernorm_post", "span_rmsnorm", "gla_decay", "gla_scan"]
+          "embed_pair", "layernorm_post", "dyt", "span_rmsnorm", "gla_decay", "gla_scan"]
 
 
 def install(monkeypatch) -> None:
