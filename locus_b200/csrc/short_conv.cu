@@ -13,6 +13,9 @@
 //                    v's rows or cache pages, laid out at `laid` elements per head (zeros behind the head's own).
 //                    With gates (a gated delta rule's), one more warp per token forms beta = sigmoid(b) and
 //                    decay = exp(-exp(A_log) * softplus(a + dt_bias)) for every head.
+//   head_rows        the same without a convolution, an activation and gates, for channels that lie in 16-byte pieces: a
+//                    block per token, whose angles' sines and cosines are formed once for all heads, four channels to
+//                    a lane and a head to 8, 16 or 32 lanes.
 //   conv_state_move  afterwards: the slot's last taps - 1 inputs move on by the portion's tokens.
 #include "common.cuh"
 
@@ -147,6 +150,149 @@ __global__ void __launch_bounds__(128) head_prep_kernel(const PrepArgs a) {
     for (int i = lane; i < laid; i += 32) dst[i] = from_f<T>(i < d ? buf[i] * r : 0.f);
 }
 
+// LANES lanes to a head (4 channels each, SLOTS times), 32 / LANES heads to a warp.  Rows 0 .. gridDim.x - 1.
+template <typename T, int LANES, int SLOTS>
+__global__ void __launch_bounds__(256) head_rows_kernel(const PrepArgs a) {
+    __shared__ float cs[PREP_MAX_DIM / 2], sn[PREP_MAX_DIM / 2];
+    __shared__ __align__(16) float xch[8][PREP_MAX_DIM];   // half-split pairs: a warp's rows, read at the partner's place
+    const size_t row = blockIdx.x;
+    const int half = a.inv_freq != nullptr ? a.rot / 2 : 0;
+    // (positions, slots and frequencies were on the device before the step's first kernel)
+    const float pos = static_cast<float>(a.positions[row]);
+    for (int i = threadIdx.x; i < half; i += 256) sincosf(pos * a.inv_freq[i], &sn[i], &cs[i]);
+    const int slot = a.pool != nullptr ? a.slots[row] : 0;
+    const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5, sub = lane & (LANES - 1);
+    const int nq = a.heads[0], nk = a.heads[1], n_units = nq + nk + a.heads[2];
+    constexpr int PER_WARP = 32 / LANES;
+    pdl_entry();
+    pdl_trigger();
+    const float* pr = a.proj + row * a.ld;
+    auto fetch = [&](int base, float4* t) {   // this lane's channels of a unit (zeros past the head's end)
+        const int unit = base + lane / LANES;
+        const int which = unit < nq ? 0 : (unit < nq + nk ? 1 : 2);
+        const int head = unit - (which == 0 ? 0 : (which == 1 ? nq : nq + nk));
+#pragma unroll
+        for (int s = 0; s < SLOTS; ++s) {
+            const int c = (s * LANES + sub) * 4;
+            t[s] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (unit < n_units && (which == 0 || a.write_kv) && c < a.dim[which])
+                t[s] = *reinterpret_cast<const float4*>(pr + a.off[which] + head * a.dim[which] + c);
+        }
+    };
+    const int step = gridDim.y * 8 * PER_WARP;
+    float4 next[SLOTS];
+    fetch((blockIdx.y * 8 + wid) * PER_WARP, next);   // (under way while the first warps form the angles' sines and cosines)
+    __syncthreads();
+    for (int base = (blockIdx.y * 8 + wid) * PER_WARP; base < n_units; base += step) {
+        const int unit = base + lane / LANES;
+        const int which = unit < nq ? 0 : (unit < nq + nk ? 1 : 2);
+        const bool live = unit < n_units && (which == 0 || a.write_kv);
+        const int head = unit - (which == 0 ? 0 : (which == 1 ? nq : nq + nk));
+        const int d = a.dim[which], laid = a.laid[which];
+        float v[SLOTS][4];
+#pragma unroll
+        for (int s = 0; s < SLOTS; ++s) {
+            v[s][0] = next[s].x; v[s][1] = next[s].y; v[s][2] = next[s].z; v[s][3] = next[s].w;
+        }
+        fetch(base + step, next);
+        auto sum_sq = [&]() -> float {   // over the head's channels (every lane of the warp takes part)
+            float ss = 0.f;
+#pragma unroll
+            for (int s = 0; s < SLOTS; ++s)
+#pragma unroll
+                for (int k = 0; k < 4; ++k) ss = fmaf(v[s][k], v[s][k], ss);
+#pragma unroll
+            for (int o = LANES / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+            return ss;
+        };
+        if (a.norm == 3) {
+            const float rms = 1.0f / sqrtf(sum_sq() / static_cast<float>(d) + a.eps);
+            if (live && which < 2) {
+#pragma unroll
+                for (int s = 0; s < SLOTS; ++s)
+#pragma unroll
+                    for (int k = 0; k < 4; ++k) {
+                        const int c = (s * LANES + sub) * 4 + k;
+                        if (c < d) v[s][k] *= rms * ld_dyn(a.norm_w[which], a.norm_w_dt, c);
+                    }
+            }
+        }
+        if (half > 0 && a.adjacent) {
+            if (which < 2) {
+#pragma unroll
+                for (int s = 0; s < SLOTS; ++s)
+#pragma unroll
+                    for (int k = 0; k < 4; k += 2) {
+                        const int i = ((s * LANES + sub) * 4 + k) >> 1;
+                        if (i < half) {
+                            const float x = v[s][k], y = v[s][k + 1];
+                            v[s][k] = x * cs[i] - y * sn[i];
+                            v[s][k + 1] = y * cs[i] + x * sn[i];
+                        }
+                    }
+            }
+        } else if (half > 0) {
+            float* mine = xch[wid] + (lane / LANES) * (PREP_MAX_DIM / PER_WARP);
+            __syncwarp();   // the last round's rows have been read
+#pragma unroll
+            for (int s = 0; s < SLOTS; ++s)
+                *reinterpret_cast<float4*>(mine + (s * LANES + sub) * 4) = make_float4(v[s][0], v[s][1], v[s][2], v[s][3]);
+            __syncwarp();
+            if (which < 2) {
+#pragma unroll
+                for (int s = 0; s < SLOTS; ++s)
+#pragma unroll
+                    for (int k = 0; k < 4; ++k) {
+                        const int c = (s * LANES + sub) * 4 + k;
+                        if (c < half) v[s][k] = v[s][k] * cs[c] - mine[c + half] * sn[c];
+                        else if (c < 2 * half) v[s][k] = v[s][k] * cs[c - half] + mine[c - half] * sn[c - half];
+                    }
+            }
+        }
+        float r = which == 0 ? a.q_scale : 1.0f;
+        if (a.norm == 1 || a.norm == 2) {
+            const float ss = sum_sq();
+            if (which < 2) r *= a.norm == 1 ? 1.0f / sqrtf(ss / static_cast<float>(d) + a.eps) : 1.0f / sqrtf(ss + a.eps);
+        }
+        if (!live) continue;
+        T* dst;
+        if (which == 0) {
+            dst = static_cast<T*>(a.q_out) + (row * nq + head) * laid;
+        } else if (a.pool != nullptr) {
+            const int page = slot / a.page_tokens, o = slot % a.page_tokens;
+            dst = static_cast<T*>(a.pool) + ((static_cast<size_t>(page) * 2 + (which - 1)) * nk + head) * a.page_tokens * laid +
+                  static_cast<size_t>(o) * laid;
+        } else {
+            dst = static_cast<T*>(which == 1 ? a.k_out : a.v_out) + (row * a.heads[which] + head) * laid;
+        }
+#pragma unroll
+        for (int s = 0; s < SLOTS; ++s) {
+            const int c = (s * LANES + sub) * 4;
+            if (c >= laid) continue;
+            if (sizeof(T) == 4) {
+                *reinterpret_cast<float4*>(dst + c) = make_float4(v[s][0] * r, v[s][1] * r, v[s][2] * r, v[s][3] * r);
+            } else {
+                __nv_bfloat162 lo = __floats2bfloat162_rn(v[s][0] * r, v[s][1] * r), hi = __floats2bfloat162_rn(v[s][2] * r, v[s][3] * r);
+                *reinterpret_cast<uint2*>(dst + c) = make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
+            }
+        }
+    }
+}
+
+template <typename T>
+static void launch_head_rows(const PrepArgs& a, int n_rows, cudaStream_t stream) {
+    const int lanes = a.laid[0] <= 32 ? 8 : (a.laid[0] <= 64 ? 16 : 32);
+    const int units = a.heads[0] + a.heads[1] + a.heads[2];
+    // a block takes all heads of its token when there are tokens enough to fill the GPU, else its share of them
+    const int rounds = ceil_div(units, 8 * (32 / lanes));
+    const int want = ceil_div(296, n_rows);
+    const dim3 grid(n_rows, want < rounds ? want : rounds);
+    if (lanes == 8) locus_launch(head_rows_kernel<T, 8, 1>, grid, dim3(256), 0, stream, a);
+    else if (lanes == 16) locus_launch(head_rows_kernel<T, 16, 1>, grid, dim3(256), 0, stream, a);
+    else if (a.laid[0] <= 128) locus_launch(head_rows_kernel<T, 32, 1>, grid, dim3(256), 0, stream, a);
+    else locus_launch(head_rows_kernel<T, 32, 2>, grid, dim3(256), 0, stream, a);
+}
+
 __global__ void __launch_bounds__(256) conv_state_move_kernel(const float* __restrict__ proj, int ld, int off0, int n0,
                                                               int off1, int n1, int off2, float* __restrict__ conv_state,
                                                               long long slot_stride, const int* __restrict__ state_slots,
@@ -169,15 +315,23 @@ __global__ void __launch_bounds__(256) conv_state_move_kernel(const float* __res
     for (int j = 0; j < keep_n; ++j) st[j] = nv[j];
 }
 
+// Whether the heads lie in pieces of four channels: what head_rows_kernel takes.
+static bool laid_alike(const PrepArgs& a) {
+    for (int w = 0; w < 3; ++w)
+        if (a.heads[w] > 0 && (a.dim[w] % 4 || a.off[w] % 4 || a.laid[w] % 4 || a.laid[w] != a.laid[0] || a.laid[w] > PREP_MAX_DIM)) return false;
+    return a.heads[0] > 0;
+}
+
 // sizes [12]: off, heads, dim, laid of q, k, v.  conv [channels, taps] (element type conv_dt) or null; conv_state: the
 // address of the convolution's part of slot 0, moved on by the call when move_state is set.  out_dt: the element type
 // of q_out, k_out, v_out and the pool.  pool: the layer's pages (k and v go there, at slots[t]) or null (k_out, v_out).
+// n_rows > 0: the segments' rows are proj's rows 0 .. n_rows - 1 without a gap (head_rows_kernel runs where it can).
 // adjacent: rotate the pairs (2i, 2i + 1) instead of (i, i + rot/2).  norm 3: q_norm_w, k_norm_w [dim] of element type
 // norm_w_dt.  gates: beta, decay [T, gate_heads] float32 from columns off_b, off_a of proj, or beta null.
 extern "C" int locus_head_prep(const float* proj, int ld, const int* sizes, const void* conv, int conv_dt, int taps, int act,
                                float* conv_state, long long slot_stride, int move_state, const int* state_slots,
-                               const int* seg_q0, const int* seg_qn, int n_seg, int longest_new, const int* positions,
-                               const float* inv_freq, int rot, int adjacent, int norm, const void* q_norm_w,
+                               const int* seg_q0, const int* seg_qn, int n_seg, int longest_new, int n_rows,
+                               const int* positions, const float* inv_freq, int rot, int adjacent, int norm, const void* q_norm_w,
                                const void* k_norm_w, int norm_w_dt, float eps, float q_scale, void* q_out, void* k_out,
                                void* v_out, void* pool, const int* slots, int page_tokens, int write_kv, int out_dt,
                                float* beta, float* decay, int off_b, int off_a, int gate_heads, const void* a_log,
@@ -203,6 +357,15 @@ extern "C" int locus_head_prep(const float* proj, int ld, const int* sizes, cons
     a.q_out = q_out; a.k_out = k_out; a.v_out = v_out; a.pool = pool; a.slots = slots; a.page_tokens = page_tokens;
     a.write_kv = write_kv; a.beta = beta; a.decay = decay; a.off_b = off_b; a.off_a = off_a; a.gate_heads = gate_heads;
     a.a_log = a_log; a.dt_bias = dt_bias; a.gate_dt = gate_dt;
+    if (n_rows > 0 && conv == nullptr && !act && beta == nullptr && ld % 4 == 0 && laid_alike(a) &&
+        (reinterpret_cast<uintptr_t>(proj) & 15) == 0 &&
+        ((reinterpret_cast<uintptr_t>(q_out) | reinterpret_cast<uintptr_t>(k_out) | reinterpret_cast<uintptr_t>(v_out) |
+          reinterpret_cast<uintptr_t>(pool)) & 15) == 0) {
+        if (out_dt == LOCUS_DT_F32) launch_head_rows<float>(a, n_rows, stream);
+        else if (out_dt == LOCUS_DT_BF16) launch_head_rows<bf16>(a, n_rows, stream);
+        else return LOCUS_ERR_UNSUPPORTED;
+        return locus_launch_status();
+    }
     const int units = a.heads[0] + a.heads[1] + a.heads[2] + (beta != nullptr ? 1 : 0);
     const dim3 grid((units + 3) / 4, longest_new, n_seg);
     if (out_dt == LOCUS_DT_F32) locus_launch(head_prep_kernel<float>, grid, dim3(128), 0, stream, a);
@@ -231,12 +394,49 @@ __global__ void __launch_bounds__(256) gate_rows_kernel(T* __restrict__ o, const
     *p = from_f<T>(to_f(*p) * sc_sigmoid(proj[t * ld + off + e]));
 }
 
+// The same for heads of whole 16-byte pieces: eight elements to a thread, a token to blockIdx.y.
+template <typename T>
+__global__ void __launch_bounds__(256) gate_rows8_kernel(T* __restrict__ o, const float* __restrict__ proj, int ld, int off,
+                                                         int pieces, int o_ld, int dim, int laid) {
+    pdl_entry();
+    pdl_trigger();
+    const int i = blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= pieces) return;
+    const size_t t = blockIdx.y;
+    const int e = i * 8;
+    const float4* g4 = reinterpret_cast<const float4*>(proj + t * ld + off + e);
+    const float4 ga = g4[0], gb = g4[1];
+    const float g[8] = {ga.x, ga.y, ga.z, ga.w, gb.x, gb.y, gb.z, gb.w};
+    T* p = o + t * o_ld + (e / dim) * laid + e % dim;
+    constexpr int W = sizeof(T) * 8 / 16;   // 16-byte words of eight elements
+    uint4 w[W];
+#pragma unroll
+    for (int k = 0; k < W; ++k) w[k] = reinterpret_cast<const uint4*>(p)[k];
+    T* x = reinterpret_cast<T*>(w);
+#pragma unroll
+    for (int k = 0; k < 8; ++k) x[k] = from_f<T>(to_f(x[k]) * sc_sigmoid(g[k]));
+#pragma unroll
+    for (int k = 0; k < W; ++k) reinterpret_cast<uint4*>(p)[k] = w[k];
+}
+
 // o [T, o_ld] (heads laid out at `laid` elements of which the first `dim` are the head's own), gate columns
 // [off, off + width) of proj [T, ld] float32, width = heads * dim.
 extern "C" int locus_gate_rows(void* o, int o_dt, int o_ld, const float* proj, int ld, int off, int width, int dim, int laid,
                                int T, cudaStream_t stream) {
     if (T <= 0 || width <= 0) return 0;
     if (dim <= 0 || laid < dim || width % dim) return LOCUS_ERR_UNSUPPORTED;
+    if (dim % 8 == 0 && laid % 8 == 0 && o_ld % 8 == 0 && ld % 4 == 0 && off % 4 == 0 && T <= 65535 &&
+        ((reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(proj)) & 15) == 0) {
+        const int pieces = width / 8, threads = pieces >= 256 ? 256 : ceil_div(pieces, 32) * 32;
+        const dim3 grid(ceil_div(pieces, threads), T);
+        if (o_dt == LOCUS_DT_F32)
+            locus_launch(gate_rows8_kernel<float>, grid, dim3(threads), 0, stream, static_cast<float*>(o), proj, ld, off, pieces, o_ld, dim, laid);
+        else if (o_dt == LOCUS_DT_BF16)
+            locus_launch(gate_rows8_kernel<bf16>, grid, dim3(threads), 0, stream, static_cast<bf16*>(o), proj, ld, off, pieces, o_ld, dim, laid);
+        else
+            return LOCUS_ERR_UNSUPPORTED;
+        return locus_launch_status();
+    }
     const long long n = static_cast<long long>(T) * width;
     const unsigned blocks = static_cast<unsigned>((n + 255) / 256);
     if (o_dt == LOCUS_DT_F32)

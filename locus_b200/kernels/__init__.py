@@ -1738,7 +1738,8 @@ def head_prep(proj: torch.Tensor, *, offsets, heads, dims, laid, state_slots: to
               write_kv: bool = True, conv: Optional[torch.Tensor] = None, state: Optional[torch.Tensor] = None,
               conv_offset: int = 0, move_state: bool = True, act: bool = False,
               inv_freq: Optional[torch.Tensor] = None, rot: int = 0, norm: Optional[str] = None, eps: float = 0.0,
-              q_scale: float = 1.0, gates=None, interleaved: bool = False, norm_weights=None) -> None:
+              q_scale: float = 1.0, gates=None, interleaved: bool = False, norm_weights=None,
+              n_rows: int = 0) -> None:
     """From the float32 rows ``proj`` of a stacked projection to q in rows and k, v in rows or cache pages, in one
     launch.  ``offsets``, ``heads``, ``dims``, ``laid``: for q, k, v the first column in ``proj``, the number of heads,
     the per-head size and the size a head is laid out at in the output (zeros behind its own elements).  In this
@@ -1749,7 +1750,8 @@ def head_prep(proj: torch.Tensor, *, offsets, heads, dims, laid, state_slots: to
     [rot / 2]: q's and k's pairs (i, i + rot / 2) rotated by position * inv_freq[i]; ``norm`` "rms": q and k divided
     by sqrt(mean(x^2) + eps) per head, "unit": by sqrt(sum(x^2) + eps), "head": by sqrt(mean(x^2) + eps) and multiplied by
     ``norm_weights`` = (q's, k's) [dim] in FRONT of the rotation; ``interleaved``: the rotation takes the pairs (2i, 2i + 1)
-    instead; ``q_scale`` on q.  The outputs share one
+    instead; ``n_rows`` > 0: the segments' rows are the rows 0 .. n_rows - 1 of ``proj`` without a gap (the kernel of a block
+    per token then runs where it can); ``q_scale`` on q.  The outputs share one
     element type; with ``pool`` (a layer's pages [n_pages, 2, heads_k, page_tokens, laid]) k and v go to ``slots``.
     ``gates`` = (beta, decay, off_b, off_a, a_log, dt_bias): also beta = sigmoid(proj[:, off_b + h]) and decay =
     exp(-exp(a_log[h]) * softplus(proj[:, off_a + h] + dt_bias[h])), [T, heads] float32 each."""
@@ -1758,7 +1760,7 @@ def head_prep(proj: torch.Tensor, *, offsets, heads, dims, laid, state_slots: to
     _i32(positions, "positions")
     sizes = (ctypes.c_int * 12)(*[int(v) for v in (*offsets, *heads, *dims, *laid)])
     out_dt = q_out.dtype
-    _need(q_out.shape[1] == heads[0] * laid[0], "head_prep: q_out width")
+    _need(q_out.shape[1] == heads[0] * laid[0] and q_out.shape[0] >= n_rows and proj.shape[0] >= n_rows, "head_prep: q_out width")
     if pool is not None:
         _cuda_c(pool, "pool")
         _i32(slots, "slots")
@@ -1797,7 +1799,7 @@ def head_prep(proj: torch.Tensor, *, offsets, heads, dims, laid, state_slots: to
     code = _lib("short_conv").locus_head_prep(
         _p(proj), I(proj.stride(0)), sizes, _p(conv), I(dtype_code(conv.dtype) if conv is not None else 0), I(taps),
         I(1 if act else 0), state_ptr, LL(stride), I(1 if move_state else 0), _p(state_slots), _p(seg_q0), _p(seg_qn),
-        I(n_seg), I(longest_new), _p(positions), _p(inv_freq), I(rot if inv_freq is not None else 0),
+        I(n_seg), I(longest_new), I(n_rows), _p(positions), _p(inv_freq), I(rot if inv_freq is not None else 0),
         I(1 if interleaved else 0), I(HEAD_NORMS[norm]), _p(q_w), _p(k_w), I(dtype_code(q_w.dtype) if q_w is not None else 0),
         F(eps), F(q_scale), _p(q_out), _p(k_out), _p(v_out), _p(pool), _p(slots), I(page_tokens), I(1 if write_kv else 0),
         I(dtype_code(out_dt)), _p(beta), _p(decay), I(off_b), I(off_a), I(gate_heads), _p(a_log), _p(dt_bias), I(gate_dt),

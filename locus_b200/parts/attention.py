@@ -324,7 +324,7 @@ class Attention(Mixer):
                     pool=cache.pool if kv else None, slots=gb.slots if kv else None, page_tokens=gb.page_tokens,
                     write_kv=cache.writes, conv=self.params.get("conv"), state=cache.state if self.conv_taps > 1 else None,
                     inv_freq=table.inv_freq if table else None, rot=table.rot_dim if table else 0,
-                    interleaved=table.interleaved if table else False,
+                    interleaved=table.interleaved if table else False, n_rows=T,
                     norm=None if self.qk_norm == "whole" else self.qk_norm, eps=self.qk_norm_eps,
                     norm_weights=(self.params["q_norm"], self.params.get("k_norm")) if self.qk_norm == "head" else None)
         o = rt.rows("attention.o", self.q_dim, rt.dtype, T)

@@ -1,10 +1,11 @@
-"""Prefill and decode throughput of the Lalepel, the Pozozen, the Mekizen or the Gugozen design at layer sizes that
+"""Prefill and decode throughput of the Lalepel, the Pozozen, the Mekizen, the Gugozen or the Bebovik design at layer sizes that
 resemble a real model's, beside the closest architecture at equal sizes (random weights, synthetic token ids, one GPU):
 Qwen2-MoE for Lalepel and Pozozen; for Mekizen both Pozozen (the closest mixers: windowed attention beside a float32
 recurrence) and Qwen2-MoE; for Gugozen both Lalepel (the closest mixers: latent attention and a float32 linear recurrence,
-with routed experts) and Qwen2-MoE.
+with routed experts) and Qwen2-MoE; for Bebovik both Qwen2 with dense layers only (the closest: grouped-query attention and a
+gated feed-forward of the same sizes) and Mekizen (the closest mixers: attention behind ``head_prep`` with an output gate).
 
-    python -m locus_b200.tools.arch_bench [--design lalepel|pozozen|mekizen|gugozen] [--size m|s] [--layers 4] [--prefill 2048]
+    python -m locus_b200.tools.arch_bench [--design lalepel|pozozen|mekizen|gugozen|bebovik] [--size m|s] [--layers 4] [--prefill 2048]
                                           [--batch 8] [--context 4096] [--steps 16] [--warmup 3] [--dtype bf16|fp32]
                                           [--kernels]
 
@@ -16,7 +17,9 @@ in eight (or four) groups of which half stay open; Mekizen's through (convolved 
 windowed attention with kept first tokens and a sink, the same beside a delta rule again, attention on the second
 layer's keys and values), all with a dense squared-ReLU feed-forward of four times the width; Gugozen's through
 (grouped-query attention with a learned sink, gated linear attention, latent attention, latent attention on the third
-layer's rows), all with clamped gated experts weighted on their input and a shared expert.  Timed on the device with CUDA events after warm-up; every step reads its weights (several
+layer's rows), all with clamped gated experts weighted on their input and a shared expert; Bebovik's are all grouped-query
+attention in chunks (heads / 4 key/value heads, as in the dense Qwen2 beside it) and a clamped gated feed-forward of the width
+of the others' shared expert.  Timed on the device with CUDA events after warm-up; every step reads its weights (several
 hundred MB: more than the L2 holds).  ``--kernels`` adds, for one eager prefill step and one eager decode step of
 each model, the time by kernel entry point, and for the mixers' own kernels what their bytes or flops would take
 at the measured peaks.  Prints one JSON line.
@@ -110,6 +113,22 @@ def gugozen_config(z, n_layers):
             "embedding": {"bigram": {"buckets": 65521, "mul_prev": 1000003, "mul_cur": 31}}, "layers": layers}
 
 
+def bebovik_config(z, n_layers):
+    layer = {"type": "attention", "mlp": {"kind": "dense", "ff": z["shared"], "limit": 7.0}, "mixer": {
+        "heads": z["heads"], "kv_heads": max(1, z["heads"] // 4), "dim": z["dim"], "vdim": z["vdim"], "scale": z["dim"] ** -0.5,
+        "mask": {"size": z["window"]}, "rot": {"base": 500000.0, "dims": z["dim"], "scaling": {
+            "factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}}
+    return {"architecture": "Bebovik", "width": z["width"], "vocab": z["vocab"], "norm": {"eps": 1e-5},
+            "embedding": {"scale": 8.0}, "logit_scale": 0.5, "logit_softcap": 25.0, "layers": [layer] * n_layers}
+
+
+def qwen_dense_config(z, n_layers, max_pos):
+    """Qwen2 with dense layers only: grouped-query attention and a SwiGLU of the sizes of ``bebovik_config``."""
+    raw = qwen_config(z, n_layers, max_pos)
+    raw.update({"num_key_value_heads": max(1, z["heads"] // 4), "mlp_only_layers": list(range(n_layers))})
+    return raw
+
+
 def qwen_config(z, n_layers, max_pos):
     hd = z["dim"] + z["rot"] if (z["dim"] + z["rot"]) in (64, 128) else z["dim"]
     return {"architectures": ["Qwen2MoeForCausalLM"], "model_type": "qwen2_moe", "num_hidden_layers": n_layers,
@@ -153,14 +172,19 @@ def run(args) -> dict:
     gen = torch.Generator().manual_seed(5)
     design = args.design
     own = {"lalepel": lalepel_config, "pozozen": pozozen_config, "mekizen": mekizen_config,
-           "gugozen": gugozen_config}[design](z, args.layers)
+           "gugozen": gugozen_config, "bebovik": bebovik_config}[design](z, args.layers)
     raws = {design: own}
     if design == "mekizen":
         raws["pozozen"] = pozozen_config(z, args.layers)
     if design == "gugozen":
         raws["lalepel"] = lalepel_config(z, args.layers)
-    raws["qwen2_moe"] = qwen_config(z, args.layers, max(ctx, T) + 8)
-    raws["qwen2_moe"].pop("_head")
+    if design == "bebovik":
+        raws["mekizen"] = mekizen_config(z, args.layers)
+        raws["qwen2_dense"] = qwen_dense_config(z, args.layers, max(ctx, T) + 8)
+    else:
+        raws["qwen2_moe"] = qwen_config(z, args.layers, max(ctx, T) + 8)
+    for raw in raws.values():
+        raw.pop("_head", None)
     out = {}
     for name, raw in raws.items():
         entry = find_arch(arch_name_of(raw))
@@ -241,6 +265,26 @@ def run(args) -> dict:
     H, R = z["heads"], z["kv_rank"] + z["rot"]
     keys_avg = sum(min(p + 1, z["window"]) for p in range(T)) / T
     fma_tflops = 148 * 128 * 2 * 1.965e9 / 1e12       # float32 FMAs of the CUDA cores at the top clock
+    if design == "bebovik":
+        G, D, Wd, ff = max(1, H // 4), z["dim"], z["width"], z["shared"]
+        in_w = (2 * H + 2 * G) * D                   # q, k, v and the gate
+        row = T / (pk["hbm_gbs"] * 1e9) * 1e6        # us per byte of a row, over the portion's rows
+        bounds = {
+            "attn_prefill_us": 2.0 * T * keys_avg * H * 2 * D / (pk["bf16_tflops"] * 1e12) * 1e6,
+            "attn_decode_us": B * min(ctx, z["window"]) * 2 * G * D * el / (pk["hbm_gbs"] * 1e9) * 1e6,
+            # the addition and both norms in one pass: the stream in and out, the sublayer's row in, the normed row out
+            "dyt_prefill_us": row * Wd * (4 + 4 + 4 + el),
+            # float32 rows of q, k and v in, 16-bit rows and pages out; the gate's rows in, the heads' outputs in and out
+            "head_prep_prefill_us": row * (H + 2 * G) * D * (4 + el),
+            "gate_rows_prefill_us": row * H * D * (4 + 2 * el),
+            "layer_weights_decode_us": (in_w * Wd + H * D * Wd + 3 * Wd * ff) * el / (pk["hbm_gbs"] * 1e9) * 1e6,
+            "layer_products_prefill_us": 2.0 * T * (in_w * Wd + H * D * Wd + 3 * Wd * ff) / (pk["bf16_tflops"] * 1e12) * 1e6,
+        }
+        return {"metric": f"prefill and decode tokens/s, Bebovik beside Mekizen and dense Qwen2 at equal layer sizes "
+                          f"({args.size}, {args.layers} layers, {args.dtype})",
+                "size": z, "layers": args.layers, "dtype": args.dtype, "data": "synthetic", "designs": out,
+                "bounds_per_layer": bounds, "peaks": pk,
+                "l2": "no flush: every step reads its weights, more than the 126 MB L2"}
     if design == "gugozen":
         d, dv, G = z["ret_dim"], z["vdim"], max(1, H // 4)
         bounds = {
@@ -324,7 +368,7 @@ def run(args) -> dict:
 
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(prog="arch_bench", description=__doc__.split("\n\n")[0])
-    ap.add_argument("--design", default="lalepel", choices=["lalepel", "pozozen", "mekizen", "gugozen"])
+    ap.add_argument("--design", default="lalepel", choices=["lalepel", "pozozen", "mekizen", "gugozen", "bebovik"])
     ap.add_argument("--size", default="m", choices=sorted(SIZES))
     ap.add_argument("--layers", type=int, default=4)
     ap.add_argument("--prefill", type=int, default=2048)

@@ -7,6 +7,7 @@
     python -m locus_b200.tools.kernel_bench recurrence --tokens 2048 --batch 1 [--heads 16 --head-dim 128 --v-dim 128]
                                                        [--per-group 1] [--ones] [--retention | --delta | --gla]
     python -m locus_b200.tools.kernel_bench head_prep --tokens 2048 --batch 1 [--window 4096]
+    python -m locus_b200.tools.kernel_bench rows --tokens 2048 [--k 2048 --heads 16 --kv-heads 4 --head-dim 128]
 
 Times with CUDA events after warm-up.  Weights rotate through enough copies that the L2
 cannot hold them (``linear``); attention reads a cache larger than the L2 at the default
@@ -142,6 +143,8 @@ def _paged(args, B: int, ctx: int, new: int):
     i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
     meta = dict(seg_q0=i32([i * new for i in range(B)]), seg_qn=i32([new] * B), seg_ctx=i32([ctx] * B), block_table=table)
     kw = dict(n_heads=nh, n_kv_heads=nkv, head_dim=hd, page_tokens=P, window=args.window, scale=1 / math.sqrt(hd))
+    if args.chunk:
+        kw["chunk"] = args.chunk
     if args.keep_first or args.sink:
         kw.update(keep_first=args.keep_first, sink=args.sink)
     return pool, q, torch.empty_like(q), meta, kw, i32
@@ -162,6 +165,8 @@ def bench_attn_decode(args) -> None:
 
     us = _time(fn, args.iters, args.graph)
     seen = ctx + 1 if not args.window else min(ctx + 1, args.window + args.keep_first)   # the keys a new token sees
+    if args.chunk:
+        seen = ctx % args.chunk + 1
     byts = B * seen * 2 * args.kv_heads * args.head_dim * pool.element_size()
     print(f"attn_decode batch={B} ctx={ctx} heads={args.heads}/{args.kv_heads} head_dim={args.head_dim} window={args.window} "
           f"keep_first={args.keep_first} sink={args.sink} {args.dtype}: "
@@ -195,7 +200,10 @@ def bench_attn_chunk(args) -> None:
         call(q, pool, out, items=items, n_items=items.shape[0], **meta, **kw, **extra)
 
     us = _time(fn, args.iters, args.graph)
-    flops = 4.0 * args.heads * args.head_dim * (T * ctx + T * (T + 1) / 2)
+    seen = T * ctx + T * (T + 1) / 2
+    if args.chunk:
+        seen = sum(p % args.chunk + 1 for p in range(ctx, ctx + T))
+    flops = 4.0 * args.heads * args.head_dim * seen
     print(f"attn_chunk tokens={T} ctx={ctx} heads={args.heads}/{args.kv_heads} head_dim={args.head_dim} window={args.window} "
           f"keep_first={args.keep_first} sink={args.sink} "
           f"{f'tcgen05, {n_splits} key ranges' if tc else (f'mma.sync, {n_splits} key ranges' if mma else 'cuda cores')}: {us:.1f} us/call  {flops / us / 1e6:.1f} TFLOP/s (causal flops)")
@@ -333,6 +341,61 @@ def bench_head_prep(args) -> None:
           f"{us:.1f} us/call, {by / us / 1e3:.0f} GB/s")
 
 
+def bench_rows(args) -> None:
+    """The row kernels between the products of a layer whose attention has weighted head norms in front of an adjacent-pair
+    rotation, an output gate and Dynamic Tanh norms around it, beside the like kernels of other layers (RMSNorm; the rotation
+    and write of bfloat16 projections), on ``--tokens`` rows; every call takes the next of enough copies of its operands
+    that the L2 cannot hold them."""
+    dev = "cuda:0"
+    T, W, H, G, D, P = args.tokens, args.k, args.heads, args.kv_heads, args.head_dim, args.page_tokens
+    dt = torch.bfloat16 if args.dtype == "bfloat16" else torch.float32
+    el = 2 if dt == torch.bfloat16 else 4
+    in_w = (2 * H + 2 * G) * D
+    n = max(2, int(400e6 // (T * W * 4)) + 1)
+    x, y = [torch.randn(T, W, device=dev) for _ in range(n)], [torch.randn(T, W, device=dev) for _ in range(n)]
+    h = [torch.empty(T, W, device=dev, dtype=dt) for _ in range(n)]
+    n2 = max(2, int(400e6 // (T * in_w * 4)) + 1)
+    proj = [torch.randn(T, in_w, device=dev) for _ in range(n2)]
+    low = [t[:, : (H + 2 * G) * D].contiguous().to(dt) for t in proj]
+    q = [torch.empty(T, H * D, device=dev, dtype=dt) for _ in range(n2)]
+    pool = torch.zeros(-(-T // P), 2, G, P, D, device=dev, dtype=dt)
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    pos, where = torch.arange(T, dtype=torch.int32, device=dev), torch.arange(T, dtype=torch.int32, device=dev)
+    inv = (1e4 ** (-torch.arange(0, D, 2, dtype=torch.float32) / D)).to(dev)
+    w = torch.ones(W, device=dev, dtype=torch.bfloat16)
+    norm = (torch.ones(1, device=dev, dtype=torch.bfloat16), w, w)
+    hw = torch.ones(D, device=dev, dtype=torch.bfloat16)
+    turn = [0]
+
+    def each(bufs, fn):
+        def run():
+            turn[0] += 1
+            fn(turn[0] % bufs)
+        return run
+
+    heads = dict(offsets=(0, H * D, (H + G) * D), heads=(H, G, G), dims=(D, D, D), laid=(D, D, D), state_slots=i32([0]),
+                 seg_q0=i32([0]), seg_qn=i32([T]), n_seg=1, longest_new=T, positions=pos, pool=pool, slots=where, page_tokens=P,
+                 inv_freq=inv, rot=D, norm="head", eps=1e-5, norm_weights=(hw, hw))
+    cases = [
+        ("dyt: addition, both norms", each(n, lambda i: K.dyt(x[i], norm, h[i], add=(y[i], norm, w))), T * W * (12 + el)),
+        ("dyt: norm alone", each(n, lambda i: K.dyt(x[i], norm, h[i])), T * W * (4 + el)),
+        ("rmsnorm", each(n, lambda i: K.rmsnorm(x[i], w, 1e-5, h[i])), T * W * (4 + el)),
+        ("rmsnorm_add", each(n, lambda i: K.rmsnorm_add(y[i], w, 1e-5, x[i])), T * W * 12),
+        ("head_prep, a block per token, adjacent pairs", each(n2, lambda i: K.head_prep(
+            proj[i], q_out=q[i], interleaved=True, n_rows=T, **heads)), T * (H + 2 * G) * D * (4 + el)),
+        ("head_prep, a block per token, half-split pairs", each(n2, lambda i: K.head_prep(proj[i], q_out=q[i], n_rows=T, **heads)),
+         T * (H + 2 * G) * D * (4 + el)),
+        ("head_prep, a warp per head", each(n2, lambda i: K.head_prep(proj[i], q_out=q[i], interleaved=True, **heads)),
+         T * (H + 2 * G) * D * (4 + el)),
+        ("rope_kv_write", each(n2, lambda i: K.rope_kv_write(low[i], pos, inv, q[i], pool, where, n_heads=H, n_kv_heads=G, head_dim=D,
+                                                             rot_dim=D, interleaved=False, page_tokens=P)), T * (H + 2 * G) * D * 2 * el),
+        ("gate_rows", each(n2, lambda i: K.gate_rows(q[i], proj[i], (H + 2 * G) * D, n_heads=H, dim=D, laid=D)), T * H * D * (4 + 2 * el)),
+    ]
+    for name, fn, by in cases:
+        us = _time(fn, args.iters, args.graph)
+        print(f"{name}: {T} rows (width {W}, heads {H}/{G} of {D}), {args.dtype}: {us:.1f} us/call, {by / us / 1e3:.0f} GB/s")
+
+
 def bench_sample(args) -> None:
     """The sampling kernel on --rows rows of --vocab random float32 logits: greedy, temperature 0.8 alone, with
     top-k 50, with top-p 0.9, with top-k 50 + top-p 0.9 + min-p 0.05.  --one-block keeps every row on the one-block
@@ -355,7 +418,7 @@ def bench_sample(args) -> None:
 
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(prog="kernel_bench")
-    ap.add_argument("kernel", choices=["linear", "attn_decode", "attn_chunk", "experts", "sample", "recurrence", "head_prep"])
+    ap.add_argument("kernel", choices=["linear", "attn_decode", "attn_chunk", "experts", "sample", "recurrence", "head_prep", "rows"])
     ap.add_argument("--rows", type=int, default=8, help="sample: rows of logits")
     ap.add_argument("--vocab", type=int, default=151936, help="sample: logits of a row")
     ap.add_argument("--one-block", action="store_true", help="sample: never the cluster kernel")
@@ -381,6 +444,7 @@ def main(argv=None) -> int:
     ap.add_argument("--gla", action="store_true", help="recurrence: gated linear attention (a decay per key channel) instead")
     ap.add_argument("--page-tokens", type=int, default=64)
     ap.add_argument("--window", type=int, default=0)
+    ap.add_argument("--chunk", type=int, default=0, help="attention: queries see the keys of their own chunk of this many positions")
     ap.add_argument("--keep-first", type=int, default=0, dest="keep_first",
                     help="attention: with --window, a request's first tokens stay in sight")
     ap.add_argument("--sink", action="store_true", help="attention: one more term of score 0 in the softmax's denominator")
@@ -408,7 +472,7 @@ def main(argv=None) -> int:
         print("kernel_bench: no CUDA device", file=sys.stderr)
         return 1
     {"linear": bench_linear, "attn_decode": bench_attn_decode, "attn_chunk": bench_attn_chunk,
-     "experts": bench_experts, "sample": bench_sample, "recurrence": bench_recurrence, "head_prep": bench_head_prep}[args.kernel](args)
+     "experts": bench_experts, "sample": bench_sample, "recurrence": bench_recurrence, "head_prep": bench_head_prep, "rows": bench_rows}[args.kernel](args)
     return 0
 
 

@@ -170,5 +170,5 @@ def write_safetensors(path: str, specs: Iterable[Tuple[str, Tuple[int, ...], tor
             if tuple(t.shape) != tuple(shape) or t.dtype != dt:
                 raise SafetensorsError(f"write: tensor {name} is {tuple(t.shape)} {t.dtype}, expected {shape} {dt}")
             t = t.detach().contiguous().cpu()
-            f.write(t.view(torch.uint8).numpy().tobytes() if t.numel() else b"")
+            f.write(t.reshape(-1).view(torch.uint8).numpy().tobytes() if t.numel() else b"")
     os.replace(tmp, path)

@@ -643,7 +643,7 @@ def mlstm_out(o_raw, m_t, proj, off_g, w, eps, out, *, n_heads, v_dim):
 def head_prep(proj, *, offsets, heads, dims, laid, state_slots, seg_q0, seg_qn, n_seg, longest_new, positions, q_out,
               k_out=None, v_out=None, pool=None, slots=None, page_tokens=0, write_kv=True, conv=None, state=None,
               conv_offset=0, move_state=True, act=False, inv_freq=None, rot=0, norm=None, eps=0.0, q_scale=1.0, gates=None,
-              interleaved=False, norm_weights=None):
+              interleaved=False, norm_weights=None, n_rows=0):
     widths = [h * d for h, d in zip(heads, dims)]
     C = sum(widths)
     taps = conv.shape[1] if conv is not None else 1
