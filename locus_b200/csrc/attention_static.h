@@ -47,8 +47,9 @@
 extern "C" {
 #endif
 
-// Same arguments and results as locus_attn_decode, without part_o / part_ml (max_splits must
-// cover the longest context: at least longest position / 128 + 1).
+// Arguments and results as of locus_attn_decode, without its scratch (part_o, part_ml, counters, max_units) and
+// without chunks, kept first tokens and a sink (max_splits must cover the longest context: at least longest
+// position / 128 + 1).
 // Returns 0, a cudaError_t, LOCUS_ERR_UNSUPPORTED (10001) or LOCUS_ERR_SCRATCH_TOO_SMALL.
 int locus_attn_decode_static(const void* q, int dt, const void* pool, void* out, const int* seg_q0,
                              const int* seg_qn, const int* seg_ctx, const int* block_table,

@@ -402,9 +402,9 @@ def test_the_command_line_generates_from_a_folder_of_this_design(cases):
     assert "Mekizen" in archs.stdout
 
 
-def _paged_attention_case(dtype, nh, nkv, hd, P, segs, window, keep_first, seed):
+def _paged_attention_case(dtype, nh, nkv, hd, P, segs, window, keep_first, seed, chunk=0):
     """Requests (cached tokens, new tokens) on shuffled pages; a page that lies wholly between the kept first tokens
-    and the window of the request's first new token has gone back (no entry in the table; the pool's unused pages are
+    and the window (or in front of the chunk) of the request's first new token has gone back (no entry in the table; the pool's unused pages are
     NaN), and so is NaN whatever lies in a request's pages behind its last token."""
     g = torch.Generator().manual_seed(seed)
     need = [-(-(c + n) // P) for c, n in segs]
@@ -414,11 +414,11 @@ def _paged_attention_case(dtype, nh, nkv, hd, P, segs, window, keep_first, seed)
     table = torch.full((len(segs), max(need)), -1, dtype=torch.int32)
     used, q0s, T = 0, [], 0
     for s, (c, n) in enumerate(segs):
-        lo = max(0, c - window + 1) if window else 0
+        lo = max(0, c - window + 1) if window else (c // chunk * chunk if chunk else 0)
         for pg in range(need[s]):
             page = perm[used]
             used += 1
-            if window and pg * P >= keep_first and (pg + 1) * P <= lo:
+            if (window or chunk) and pg * P >= keep_first and (pg + 1) * P <= lo:
                 pool[page] = float("nan")
                 continue
             table[s, pg] = page
