@@ -36,6 +36,15 @@ __device__ __forceinline__ float ld_dyn(const void* p, int dt, size_t i) {
                               : __bfloat162float(reinterpret_cast<const bf16*>(p)[i]);
 }
 
+// Elements i .. i + 3 of such an array (i a multiple of 4, the array's start 16-byte aligned) in one load.
+__device__ __forceinline__ float4 ld4_dyn(const void* p, int dt, size_t i) {
+    if (dt == LOCUS_DT_F32) return *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p) + i);
+    const uint2 v = *reinterpret_cast<const uint2*>(reinterpret_cast<const bf16*>(p) + i);
+    const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.x));
+    const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.y));
+    return make_float4(lo.x, lo.y, hi.x, hi.y);
+}
+
 __device__ __forceinline__ void st_dyn(void* p, int dt, size_t i, float v) {
     if (dt == LOCUS_DT_F32) {
         reinterpret_cast<float*>(p)[i] = v;

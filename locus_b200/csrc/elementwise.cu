@@ -827,15 +827,8 @@ __device__ __forceinline__ float dyt_tanh(float x) { return FAST ? dyt_tanh_fast
 template <int V>
 __device__ __forceinline__ void dyt_params(const void* p, int dt, int c, float* o) {
     if (V == 4) {
-        if (dt == LOCUS_DT_F32) {
-            const float4 v = *reinterpret_cast<const float4*>(static_cast<const float*>(p) + c);
-            o[0] = v.x; o[1 % V] = v.y; o[2 % V] = v.z; o[3 % V] = v.w;
-        } else {
-            const uint2 v = *reinterpret_cast<const uint2*>(static_cast<const bf16*>(p) + c);
-            const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.x));
-            const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.y));
-            o[0] = lo.x; o[1 % V] = lo.y; o[2 % V] = hi.x; o[3 % V] = hi.y;
-        }
+        const float4 v = ld4_dyn(p, dt, c);
+        o[0] = v.x; o[1 % V] = v.y; o[2 % V] = v.z; o[3 % V] = v.w;
     } else {
         o[0] = ld_dyn(p, dt, c);
     }

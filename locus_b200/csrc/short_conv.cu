@@ -21,6 +21,7 @@
 
 #define PREP_MAX_TAPS 16
 #define PREP_MAX_DIM 256
+#define ROWS_WARPS 4      // warps of a block of head_rows_kernel
 
 __device__ __forceinline__ float sc_softplus(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 __device__ __forceinline__ float sc_silu(float x) { return x / (1.0f + expf(-x)); }
@@ -42,7 +43,7 @@ struct PrepArgs {
     int rot, adjacent, norm;
     const void* norm_w[2];    // norm 3: q's and k's weights [dim], shared by the heads
     int norm_w_dt;
-    float eps, q_scale;
+    float eps, q_scale, inv_dim[3];   // (inv_dim: 1 / dim)
     void* q_out;              // [T, heads[0] * laid[0]]
     void* k_out;              // rows [T, heads[1] * laid[1]] and v_out alike, or, with pool set, unused
     void* v_out;
@@ -152,14 +153,14 @@ __global__ void __launch_bounds__(128) head_prep_kernel(const PrepArgs a) {
 
 // LANES lanes to a head (4 channels each, SLOTS times), 32 / LANES heads to a warp.  Rows 0 .. gridDim.x - 1.
 template <typename T, int LANES, int SLOTS>
-__global__ void __launch_bounds__(256) head_rows_kernel(const PrepArgs a) {
+__global__ void __launch_bounds__(32 * ROWS_WARPS) head_rows_kernel(const PrepArgs a) {
     __shared__ float cs[PREP_MAX_DIM / 2], sn[PREP_MAX_DIM / 2];
-    __shared__ __align__(16) float xch[8][PREP_MAX_DIM];   // half-split pairs: a warp's rows, read at the partner's place
+    __shared__ __align__(16) float xch[ROWS_WARPS][PREP_MAX_DIM];   // half-split pairs: a warp's rows, read at the partner's place
     const size_t row = blockIdx.x;
     const int half = a.inv_freq != nullptr ? a.rot / 2 : 0;
     // (positions, slots and frequencies were on the device before the step's first kernel)
     const float pos = static_cast<float>(a.positions[row]);
-    for (int i = threadIdx.x; i < half; i += 256) sincosf(pos * a.inv_freq[i], &sn[i], &cs[i]);
+    for (int i = threadIdx.x; i < half; i += 32 * ROWS_WARPS) sincosf(pos * a.inv_freq[i], &sn[i], &cs[i]);
     const int slot = a.pool != nullptr ? a.slots[row] : 0;
     const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5, sub = lane & (LANES - 1);
     const int nq = a.heads[0], nk = a.heads[1], n_units = nq + nk + a.heads[2];
@@ -179,11 +180,11 @@ __global__ void __launch_bounds__(256) head_rows_kernel(const PrepArgs a) {
                 t[s] = *reinterpret_cast<const float4*>(pr + a.off[which] + head * a.dim[which] + c);
         }
     };
-    const int step = gridDim.y * 8 * PER_WARP;
+    const int step = gridDim.y * ROWS_WARPS * PER_WARP;
     float4 next[SLOTS];
-    fetch((blockIdx.y * 8 + wid) * PER_WARP, next);   // (under way while the first warps form the angles' sines and cosines)
+    fetch((blockIdx.y * ROWS_WARPS + wid) * PER_WARP, next);   // (under way while the first warps form the angles' sines and cosines)
     __syncthreads();
-    for (int base = (blockIdx.y * 8 + wid) * PER_WARP; base < n_units; base += step) {
+    for (int base = (blockIdx.y * ROWS_WARPS + wid) * PER_WARP; base < n_units; base += step) {
         const int unit = base + lane / LANES;
         const int which = unit < nq ? 0 : (unit < nq + nk ? 1 : 2);
         const bool live = unit < n_units && (which == 0 || a.write_kv);
@@ -206,15 +207,15 @@ __global__ void __launch_bounds__(256) head_rows_kernel(const PrepArgs a) {
             return ss;
         };
         if (a.norm == 3) {
-            const float rms = 1.0f / sqrtf(sum_sq() / static_cast<float>(d) + a.eps);
+            const float rms = rsqrtf(sum_sq() * a.inv_dim[which] + a.eps);
             if (live && which < 2) {
 #pragma unroll
-                for (int s = 0; s < SLOTS; ++s)
-#pragma unroll
-                    for (int k = 0; k < 4; ++k) {
-                        const int c = (s * LANES + sub) * 4 + k;
-                        if (c < d) v[s][k] *= rms * ld_dyn(a.norm_w[which], a.norm_w_dt, c);
-                    }
+                for (int s = 0; s < SLOTS; ++s) {
+                    const int c = (s * LANES + sub) * 4;
+                    if (c >= d) continue;
+                    const float4 w = ld4_dyn(a.norm_w[which], a.norm_w_dt, c);
+                    v[s][0] *= rms * w.x; v[s][1] *= rms * w.y; v[s][2] *= rms * w.z; v[s][3] *= rms * w.w;
+                }
             }
         }
         if (half > 0 && a.adjacent) {
@@ -284,13 +285,13 @@ static void launch_head_rows(const PrepArgs& a, int n_rows, cudaStream_t stream)
     const int lanes = a.laid[0] <= 32 ? 8 : (a.laid[0] <= 64 ? 16 : 32);
     const int units = a.heads[0] + a.heads[1] + a.heads[2];
     // a block takes all heads of its token when there are tokens enough to fill the GPU, else its share of them
-    const int rounds = ceil_div(units, 8 * (32 / lanes));
-    const int want = ceil_div(296, n_rows);
+    const int rounds = ceil_div(units, ROWS_WARPS * (32 / lanes));
+    const int want = ceil_div(4 * 148, n_rows);
     const dim3 grid(n_rows, want < rounds ? want : rounds);
-    if (lanes == 8) locus_launch(head_rows_kernel<T, 8, 1>, grid, dim3(256), 0, stream, a);
-    else if (lanes == 16) locus_launch(head_rows_kernel<T, 16, 1>, grid, dim3(256), 0, stream, a);
-    else if (a.laid[0] <= 128) locus_launch(head_rows_kernel<T, 32, 1>, grid, dim3(256), 0, stream, a);
-    else locus_launch(head_rows_kernel<T, 32, 2>, grid, dim3(256), 0, stream, a);
+    if (lanes == 8) locus_launch(head_rows_kernel<T, 8, 1>, grid, dim3(32 * ROWS_WARPS), 0, stream, a);
+    else if (lanes == 16) locus_launch(head_rows_kernel<T, 16, 1>, grid, dim3(32 * ROWS_WARPS), 0, stream, a);
+    else if (a.laid[0] <= 128) locus_launch(head_rows_kernel<T, 32, 1>, grid, dim3(32 * ROWS_WARPS), 0, stream, a);
+    else locus_launch(head_rows_kernel<T, 32, 2>, grid, dim3(32 * ROWS_WARPS), 0, stream, a);
 }
 
 __global__ void __launch_bounds__(256) conv_state_move_kernel(const float* __restrict__ proj, int ld, int off0, int n0,
@@ -342,6 +343,7 @@ extern "C" int locus_head_prep(const float* proj, int ld, const int* sizes, cons
     for (int w = 0; w < 3; ++w) {
         a.off[w] = sizes[w]; a.heads[w] = sizes[3 + w]; a.dim[w] = sizes[6 + w]; a.laid[w] = sizes[9 + w];
         if (a.heads[w] < 0 || a.dim[w] <= 0 || a.dim[w] > PREP_MAX_DIM || a.laid[w] < a.dim[w]) return LOCUS_ERR_UNSUPPORTED;
+        a.inv_dim[w] = 1.0f / static_cast<float>(a.dim[w]);
         channels += a.heads[w] * a.dim[w];
     }
     if (taps < 1 || taps > PREP_MAX_TAPS || n_seg > 65535 || longest_new > 65535) return LOCUS_ERR_UNSUPPORTED;
@@ -358,7 +360,7 @@ extern "C" int locus_head_prep(const float* proj, int ld, const int* sizes, cons
     a.write_kv = write_kv; a.beta = beta; a.decay = decay; a.off_b = off_b; a.off_a = off_a; a.gate_heads = gate_heads;
     a.a_log = a_log; a.dt_bias = dt_bias; a.gate_dt = gate_dt;
     if (n_rows > 0 && conv == nullptr && !act && beta == nullptr && ld % 4 == 0 && laid_alike(a) &&
-        (reinterpret_cast<uintptr_t>(proj) & 15) == 0 &&
+        ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(q_norm_w) | reinterpret_cast<uintptr_t>(k_norm_w)) & 15) == 0 &&
         ((reinterpret_cast<uintptr_t>(q_out) | reinterpret_cast<uintptr_t>(k_out) | reinterpret_cast<uintptr_t>(v_out) |
           reinterpret_cast<uintptr_t>(pool)) & 15) == 0) {
         if (out_dt == LOCUS_DT_F32) launch_head_rows<float>(a, n_rows, stream);
