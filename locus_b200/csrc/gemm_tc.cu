@@ -165,7 +165,8 @@ __device__ __forceinline__ void tmem_ld16(uint32_t taddr, uint32_t* v) {
 // The loader runs ahead across tile boundaries, so the pipeline never drains between tiles, and
 // two accumulator buffers in tensor memory let the MMAs of the next tile run while the epilogue
 // warps drain this one.
-template <bool DUAL>
+// (CAP: the tanh of activation 3, an instance of its own so that the other products' unrolled epilogue does not carry it.)
+template <bool DUAL, bool CAP = false>
 __global__ void __launch_bounds__(192, 1)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_w2,
                const __grid_constant__ XMaps maps_x, TcArgs a) {
@@ -455,7 +456,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                         x *= x;
                     }
                     if (a.row_scale) x *= scales[c0 + j];
-                    if (a.act == 3) x = a.act_param * tanhf(x * a.act_scale / a.act_param);
+                    if (CAP) x = a.act_param * tanhf(x * a.act_scale / a.act_param);
                     val[j] = x;
                 }
                 if (wide) {
@@ -693,6 +694,7 @@ extern "C" int locus_gemm_tc(const void* x, long long x_rows_total, long long ld
     static bool attr_set = false;
     if (!attr_set) {
         if (cudaFuncSetAttribute(gemm_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess ||
+            cudaFuncSetAttribute(gemm_tc_kernel<false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess ||
             cudaFuncSetAttribute(gemm_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess)
             return static_cast<int>(cudaGetLastError());
         attr_set = true;
@@ -708,6 +710,7 @@ extern "C" int locus_gemm_tc(const void* x, long long x_rows_total, long long ld
     const long long n_units = n_tiles_all * a.splits;
     const unsigned grid = static_cast<unsigned>(n_units < n_sm ? n_units : n_sm);
     if (dual) gemm_tc_kernel<true><<<grid, 192, smem, stream>>>(map_w, map_w2, maps_x, a);
+    else if (act == 3) gemm_tc_kernel<false, true><<<grid, 192, smem, stream>>>(map_w, map_w2, maps_x, a);
     else gemm_tc_kernel<false><<<grid, 192, smem, stream>>>(map_w, map_w2, maps_x, a);
     if (split) {
         const long long n_threads = static_cast<long long>(M) * (N / 4);
