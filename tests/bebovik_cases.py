@@ -57,10 +57,10 @@ CONFIGS = {
     "attention_only": model(48, 50, [layer(attention(4, 2, 16, 16, chunk=16, rot=8), 0)]),
     "mlp_only": model(40, 45, [layer(attention(1, 1, 8, 8, chunk=1), 48, 1.0)]),
     # larger heads: heads of 128 with values of 96 (the kernels' head size above the values'), four query heads to a
-    # key/value head, chunks of 48 and 130
+    # key/value head, chunks of 48 and 66
     "wide": model(128, 211, [
-        layer(attention(4, 1, 128, 96, chunk=48, rot=96, base=5e5, scaling=(8.0, 1.0, 4.0, 200), scale=0.12), 160, 1.5),
-        layer(attention(4, 2, 64, 64, chunk=130, rot=32, base=1e4, scale=0.2), 96, 2.0),
+        layer(attention(4, 1, 128, 96, chunk=48, rot=96, base=5e5, scaling=(6.0, 1.0, 5.0, 200), scale=0.12), 160, 1.5),
+        layer(attention(4, 2, 64, 64, chunk=66, rot=24, base=1e4, scale=0.2), 96, 2.0),
     ], emb=9.0, logit_scale=2.5, cap=14.0),
 }
 SEEDS = {n: 231 + i for i, n in enumerate(CONFIGS)}

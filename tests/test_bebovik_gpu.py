@@ -94,7 +94,7 @@ def test_other_page_sizes_and_the_cuda_core_products(page_tokens, dtype, cases, 
 def test_heads_of_128_in_long_portions_on_pages_of_64(dtype, tmp_path_factory):
     """Heads of 128 with values of 96 and four query heads on every key/value head, portions of several hundred tokens that
     span several chunks (the kernels that long portions of that head size take), chunks longer than a portion."""
-    raw = model(256, 301, [layer(attention(8, 2, 128, 96, chunk=200, rot=64, base=5e5, scaling=(8.0, 1.0, 4.0, 300), scale=0.1), 192, 1.5),
+    raw = model(256, 301, [layer(attention(8, 2, 128, 96, chunk=200, rot=64, base=5e5, scaling=(6.0, 1.0, 5.0, 300), scale=0.1), 192, 1.5),
                            layer(attention(4, 2, 128, 128, chunk=512, rot=128, scale=0.08), 0),
                            layer(attention(4, 4, 64, 64, scale=0.15), 128, 2.0)], emb=6.0, logit_scale=2.0, cap=12.0)
     case = Case("big", tmp_path_factory.mktemp("big"), torch.bfloat16, raw=raw, requests=(700, 90), tweak=_milder(dtype))
@@ -237,7 +237,7 @@ def test_the_embeddings_norm_against_its_twin(precise):
 
 @pytest.mark.parametrize("odt", DTYPES, ids=IDS)
 @pytest.mark.parametrize("heads,dims,rot,adjacent,norm", [
-    ((6, 3, 3), (64, 64, 64), 32, True, "head"), ((4, 1, 1), (40, 40, 24), 20, True, "head"), ((3, 3, 3), (256, 256, 200), 100, False, "head"),
+    ((6, 2, 2), (64, 64, 64), 24, True, "head"), ((4, 1, 1), (40, 40, 24), 20, True, "head"), ((3, 3, 3), (256, 256, 200), 100, False, "head"),
     ((5, 5, 5), (12, 12, 8), 6, True, "unit"), ((4, 2, 2), (128, 128, 128), 128, False, "rms"), ((2, 2, 2), (24, 24, 32), 24, False, None),
     ((16, 4, 4), (128, 128, 128), 128, True, "head"), ((3, 1, 1), (10, 10, 7), 6, True, "head"), ((2, 1, 1), (200, 200, 16), 0, True, "head")])
 def test_head_prep_with_weighted_norms_and_adjacent_pairs(heads, dims, rot, adjacent, norm, odt, precise):
