@@ -5,3 +5,4 @@ from .lalepel import LalepelConfig  # noqa: F401
 from .pozozen import PozozenConfig  # noqa: F401
 from .gugozen import GugozenConfig  # noqa: F401
 from .bebovik import BebovikConfig  # noqa: F401
+from .megovik import MegovikConfig  # noqa: F401

@@ -107,6 +107,29 @@ def _parallel(m: Dict[str, Any], where: str) -> ParallelConfig:
     return ParallelConfig(left=left, right=right, left_scale=_num(m, "left_scale", where), right_scale=_num(m, "right_scale", where))
 
 
+def _groups(router: Dict[str, Any], rw: str, outputs: int, top: int) -> Tuple[int, int]:
+    """(groups, groups kept) of a router with ``outputs`` scores; without ``groups``: one group."""
+    groups = _sub(router, "groups", rw, optional=True)
+    count = _pos(groups, "count", rw + "groups.") if groups is not None else 1
+    keep = _pos(groups, "keep", rw + "groups.") if groups is not None else 1
+    if outputs % count or keep > count:
+        raise ConfigError(f"config.json: {rw}groups: {count} groups (keep {keep}) do not fit {outputs} router outputs")
+    if keep * (outputs // count) < top:
+        raise ConfigError(f"config.json: {rw}groups: the {keep} groups kept hold fewer than top {top} experts")
+    return count, keep
+
+
+def _loop(raw: Dict[str, Any], n_layers: int) -> Optional[Tuple[int, int, int]]:
+    """``loop`` as (start, stop, times), None without one."""
+    loop = _sub(raw, "loop", "", optional=True)
+    if loop is None:
+        return None
+    a, b, times = take(loop, "start", int), take(loop, "stop", int), _pos(loop, "times", "loop.")
+    if not (0 <= a <= b <= n_layers):
+        raise ConfigError(f"config.json: loop: start {a} and stop {b} must lie within the {n_layers} layers, in order")
+    return a, b, times
+
+
 def _mlp(raw: Optional[Dict[str, Any]], where: str) -> Optional[RoutedFfConfig]:
     if raw is None:
         return None
@@ -121,13 +144,7 @@ def _mlp(raw: Optional[Dict[str, Any]], where: str) -> Optional[RoutedFfConfig]:
         raise ConfigError(f"config.json: {rw}identity must not be negative")
     if top > experts + identity:
         raise ConfigError(f"config.json: {rw}top {top} exceeds the {experts + identity} router outputs")
-    groups = _sub(router, "groups", rw, optional=True)
-    count = _pos(groups, "count", rw + "groups.") if groups is not None else 1
-    keep = _pos(groups, "keep", rw + "groups.") if groups is not None else 1
-    if (experts + identity) % count or keep > count:
-        raise ConfigError(f"config.json: {rw}groups: {count} groups (keep {keep}) do not fit {experts + identity} router outputs")
-    if keep * ((experts + identity) // count) < top:
-        raise ConfigError(f"config.json: {rw}groups: the {keep} groups kept hold fewer than top {top} experts")
+    count, keep = _groups(router, rw, experts + identity, top)
     return RoutedFfConfig(experts=experts, identity=identity, top=top, group_count=count, group_keep=keep,
                           expert_ff=_pos(expert, "ff", where + "expert."),
                           shared_ff=_pos(shared, "ff", where + "shared.") if shared is not None else 0)
@@ -175,15 +192,8 @@ class PozozenConfig:
             if mlp is not None and not isinstance(mlp, dict):
                 raise ConfigError(f"config.json: {where}mlp must be an object or null")
             layers.append(PozozenLayer(mixer=mx, mlp=_mlp(mlp, where + "mlp.")))
-        loop = _sub(raw, "loop", "", optional=True)
-        lp = None
-        if loop is not None:
-            a, b, times = take(loop, "start", int), take(loop, "stop", int), _pos(loop, "times", "loop.")
-            if not (0 <= a <= b <= len(layers)):
-                raise ConfigError(f"config.json: loop: start {a} and stop {b} must lie within the {len(layers)} layers, in order")
-            lp = (a, b, times)
         streams = take(raw, "streams", int, 0)
         if streams < 0:
             raise ConfigError("config.json: streams must not be negative")
         return cls(vocab=_pos(raw, "vocab", ""), width=_pos(raw, "width", ""), eps=_num(norm, "eps", "norm."),
-                   residual_mult=take(raw, "residual_mult", float, 1.0), streams=streams, loop=lp, layers=tuple(layers))
+                   residual_mult=take(raw, "residual_mult", float, 1.0), streams=streams, loop=_loop(raw, len(layers)), layers=tuple(layers))

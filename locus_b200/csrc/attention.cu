@@ -13,9 +13,11 @@
 // A window may keep a request's first tokens in sight (keep_first > 0: keys t < keep_first stay
 // visible to every later query, at their true positions), and the softmax may have a sink (sink != 0:
 // one more term of score 0 and no value in the denominator, p_j = exp(s_j) / (1 + sum exp(s_j))).
+// A score may have a distance bias taken off, a slope per head times p - t (distance.cuh).
 // Cache layout of one layer: [n_pages][2 (K, V)][nkv][page_tokens][hd].
 #include "common.cuh"
 #include "attn_ranges.cuh"
+#include "distance.cuh"
 #include "sink.cuh"
 
 struct AttnArgs {
@@ -32,6 +34,7 @@ struct AttnArgs {
     int nh, nkv, hd, page_tokens, window, chunk;
     int keep_first, sink;     // see the head of the file
     const float* sink_val;    // with sink: a learned score per query head in its place (null: the score 0)
+    const float* slopes;      // distance bias per query head (distance.cuh), or null
     float scale;
     // decode only
     float* part_o;            // [n_items, nh, max_splits, hd]
@@ -104,6 +107,7 @@ __global__ void __launch_bounds__(128) attn_chunk_kernel(AttnArgs a) {
         l_s[tid] = 0.f;
         lo_s[tid] = first_key(a.window, a.chunk, p0 + tid);
     }
+    const float slope = slope_of(a.slopes, h);
     const int t_hi = p0 + nq - 1;
     const int t_lo = first_key(a.window, a.chunk, p0);
     const int nd = hd / 8;
@@ -143,7 +147,7 @@ __global__ void __launch_bounds__(128) attn_chunk_kernel(AttnArgs a) {
                 const float* qr = qs + qi * hd;
                 const float* kr = ks + kj * (hd + 1);
                 for (int d = 0; d < hd; ++d) dot = fmaf(qr[d], kr[d], dot);
-                s = dot * a.scale;
+                s = fmaf(slope, static_cast<float>(t - p), dot * a.scale);
             }
             sc[qi * (CHUNK_TK + 1) + kj] = s;
         }
@@ -275,6 +279,7 @@ __global__ void __launch_bounds__(128) attn_decode_split_kernel(AttnArgs a) {
         krow[j] = static_cast<unsigned int>((kv_row<T>(a, table, t, kvh, 0) - static_cast<const T*>(a.pool)) >> 4);
     }
     const size_t v_off = static_cast<size_t>(a.nkv) * a.page_tokens * hd;  // V row = K row + v_off
+    const float slope = slope_of(a.slopes, h);
     __syncthreads();
     float mx = -INFINITY;
     for (int j = tid; j < nk; j += 128) {
@@ -297,7 +302,7 @@ __global__ void __launch_bounds__(128) attn_decode_split_kernel(AttnArgs a) {
             for (int u = 0; u < VEC; ++u) dot = fmaf(qs[d + u], kv[u], dot);
         }
         // (a split that holds both kept tokens and the window's start: the keys between them count for nothing)
-        const float s = (k0 + j >= t_lo || k0 + j < kept) ? dot * a.scale : -INFINITY;
+        const float s = (k0 + j >= t_lo || k0 + j < kept) ? fmaf(slope, static_cast<float>(k0 + j - p), dot * a.scale) : -INFINITY;
         sc[j] = s;
         mx = fmaxf(mx, s);
     }
@@ -445,7 +450,8 @@ __device__ __forceinline__ uint4 ld_once(const uint4* p) {
 struct true_tag { static constexpr bool value = true; };
 struct false_tag { static constexpr bool value = false; };
 
-template <typename T, int LPK, bool DEEP, bool PADDED>
+// BIAS: a distance bias; an instance of its own, since at large batches the kernel is bound by instruction issue.
+template <typename T, int LPK, bool DEEP, bool PADDED, bool BIAS>
 __global__ void __launch_bounds__(32 * DS_WARPS, DEEP ? 2 : 4) attn_decode_stream_kernel(AttnArgs a, int n_items, int max_units,
                                                                               int cost_range, int cost_merge) {
     pdl_trigger();  // every block of this grid is resident from the start
@@ -507,6 +513,7 @@ __global__ void __launch_bounds__(32 * DS_WARPS, DEEP ? 2 : 4) attn_decode_strea
         const int k_end = kept_range ? kept : min(p + 1, k_begin + len);   // exclusive
         const int keep = a.keep_first;
         const int kvh = h / (a.nh / a.nkv);
+        const float slope = BIAS ? slope_log2(a.slopes, h) : 0.f;   // (the step's descriptors and constants: no wait needed)
         const int* table = a.block_table + static_cast<size_t>(seg) * a.table_stride;
         const T* pool = static_cast<const T*>(a.pool) + static_cast<size_t>(kvh) * P * hd + d0;
 
@@ -569,6 +576,7 @@ __global__ void __launch_bounds__(32 * DS_WARPS, DEEP ? 2 : 4) attn_decode_strea
                     for (int i = 0; i < VEC; ++i) dot = fmaf(q[i], kf[i], dot);
 #pragma unroll
                     for (int o = LPK / 2; o > 0; o >>= 1) dot += __shfl_xor_sync(0xffffffffu, dot, o);
+                    if (BIAS) dot = fmaf(slope, static_cast<float>(k0 + g * KPL + grp - p), dot);
                     sc[g] = t_live(k0, g) ? dot : -INFINITY;
                 }
                 float mx = m;
@@ -650,6 +658,7 @@ __global__ void __launch_bounds__(32 * DS_WARPS, DEEP ? 2 : 4) attn_decode_strea
                     for (int i = 0; i < VEC; ++i) dot = fmaf(q[i], kf[i], dot);
 #pragma unroll
                     for (int o = LPK / 2; o > 0; o >>= 1) dot += __shfl_xor_sync(0xffffffffu, dot, o);
+                    if (BIAS) dot = fmaf(slope, static_cast<float>(k0 + g * KPL + grp - p), dot);
                     sc[g] = (FAST || t_live(k0, g)) ? dot : -INFINITY;
                 }
                 // K of the next chunk, and the block-table entry of the chunk after the next two
@@ -786,8 +795,9 @@ static AttnArgs make_args(const void* q, const void* pool, void* out, const int*
                           const int* seg_qn, const int* seg_ctx, const int* block_table,
                           int table_stride, const int* items, int nh, int nkv, int hd,
                           int page_tokens, int window, int chunk, float scale, int keep_first = 0, int sink = 0,
-                          const float* sink_val = nullptr) {
+                          const float* sink_val = nullptr, const float* slopes = nullptr) {
     AttnArgs a;
+    a.slopes = slopes;
     a.q = q; a.pool = pool; a.out = out; a.seg_q0 = seg_q0; a.seg_qn = seg_qn; a.seg_ctx = seg_ctx;
     a.block_table = block_table; a.table_stride = table_stride; a.items = items; a.nh = nh;
     a.nkv = nkv; a.hd = hd; a.page_tokens = page_tokens; a.window = window; a.chunk = chunk; a.scale = scale;
@@ -800,12 +810,13 @@ extern "C" int locus_attn_chunk(const void* q, int dt, const void* pool, void* o
                                 const int* seg_q0, const int* seg_qn, const int* seg_ctx,
                                 const int* block_table, int table_stride, const int* items,
                                 int n_items, int nh, int nkv, int hd, int page_tokens, int window, int chunk,
-                                float scale, int keep_first, int sink, const float* sink_val, cudaStream_t stream) {
+                                float scale, int keep_first, int sink, const float* sink_val, const float* slopes,
+                                cudaStream_t stream) {
     if (n_items <= 0) return 0;
     if (int e = check_common(nh, nkv, hd, page_tokens, window, chunk, keep_first)) return e;
     if (n_items > 65535) return LOCUS_ERR_UNSUPPORTED;
     AttnArgs a = make_args(q, pool, out, seg_q0, seg_qn, seg_ctx, block_table, table_stride, items,
-                           nh, nkv, hd, page_tokens, window, chunk, scale, keep_first, sink, sink_val);
+                           nh, nkv, hd, page_tokens, window, chunk, scale, keep_first, sink, sink_val, slopes);
     const size_t smem = sizeof(float) * (CHUNK_BQ * hd + CHUNK_TK * (hd + 1) + CHUNK_TK * hd +
                                          CHUNK_BQ * (CHUNK_TK + 1) + 3 * CHUNK_BQ);
     dim3 grid(nh, n_items);
@@ -832,12 +843,12 @@ extern "C" int locus_attn_decode(const void* q, int dt, const void* pool, void* 
                                  int n_items, int nh, int nkv, int hd, int page_tokens, int window, int chunk,
                                  float scale, float* part_o, float* part_ml, int* counters, int max_splits,
                                  long long max_units, int keep_first, int sink, const float* sink_val,
-                                 cudaStream_t stream) {
+                                 const float* slopes, cudaStream_t stream) {
     if (n_items <= 0) return 0;
     if (int e = check_common(nh, nkv, hd, page_tokens, window, chunk, keep_first)) return e;
     if (nh > 65535 || max_splits <= 0 || max_splits > 65535) return LOCUS_ERR_UNSUPPORTED;
     AttnArgs a = make_args(q, pool, out, seg_q0, seg_qn, seg_ctx, block_table, table_stride, items,
-                           nh, nkv, hd, page_tokens, window, chunk, scale, keep_first, sink, sink_val);
+                           nh, nkv, hd, page_tokens, window, chunk, scale, keep_first, sink, sink_val, slopes);
     a.part_o = part_o; a.part_ml = part_ml; a.counters = counters; a.max_splits = max_splits;
     if (counters == nullptr) return LOCUS_ERR_UNSUPPORTED;
     // (one partial result per request and head at least; two where kept first tokens are a range of their own)
@@ -865,9 +876,11 @@ extern "C" int locus_attn_decode(const void* q, int dt, const void* pool, void* 
         const int units = static_cast<int>(max_units < (1 << 30) ? max_units : (1 << 30));
 #define DS_LAUNCH(TT, L)                                                                                               \
         do {                                                                                                           \
-            if (deep) locus_launch(attn_decode_stream_kernel<TT, L, true, true>, sgrid, 32 * DS_WARPS, 0, stream, a, n_items, units, g_ds_cost_range, g_ds_cost_merge); \
-            else if (pieces != L) locus_launch(attn_decode_stream_kernel<TT, L, false, true>, sgrid, 32 * DS_WARPS, 0, stream, a, n_items, units, g_ds_cost_range, g_ds_cost_merge); \
-            else locus_launch(attn_decode_stream_kernel<TT, L, false, false>, sgrid, 32 * DS_WARPS, 0, stream, a, n_items, units, g_ds_cost_range, g_ds_cost_merge); \
+            if (slopes && deep) locus_launch(attn_decode_stream_kernel<TT, L, true, true, true>, sgrid, 32 * DS_WARPS, 0, stream, a, n_items, units, g_ds_cost_range, g_ds_cost_merge); \
+            else if (slopes) locus_launch(attn_decode_stream_kernel<TT, L, false, true, true>, sgrid, 32 * DS_WARPS, 0, stream, a, n_items, units, g_ds_cost_range, g_ds_cost_merge); \
+            else if (deep) locus_launch(attn_decode_stream_kernel<TT, L, true, true, false>, sgrid, 32 * DS_WARPS, 0, stream, a, n_items, units, g_ds_cost_range, g_ds_cost_merge); \
+            else if (pieces != L) locus_launch(attn_decode_stream_kernel<TT, L, false, true, false>, sgrid, 32 * DS_WARPS, 0, stream, a, n_items, units, g_ds_cost_range, g_ds_cost_merge); \
+            else locus_launch(attn_decode_stream_kernel<TT, L, false, false, false>, sgrid, 32 * DS_WARPS, 0, stream, a, n_items, units, g_ds_cost_range, g_ds_cost_merge); \
         } while (0)
         if (dt == LOCUS_DT_F32) {
             if (lpk == 8) DS_LAUNCH(float, 8);
@@ -952,5 +965,5 @@ extern "C" int locus_attn_decode_static(const void* q, int dt, const void* pool,
     // and the counters are zero between calls.
     return locus_attn_decode(q, dt, pool, out, seg_q0, seg_qn, seg_ctx, block_table, table_stride,
                              items, n_items, nh, nkv, hd, page_tokens, window, 0, scale, part_o, part_ml,
-                             g_attn_static_cnt_ptr[dev], max_splits, cap, 0, 0, nullptr, stream);
+                             g_attn_static_cnt_ptr[dev], max_splits, cap, 0, 0, nullptr, nullptr, stream);
 }

@@ -31,6 +31,7 @@
 // Takes bfloat16, head sizes 64 and 128, groups of 2 to 16 query heads, pages of a multiple of 16 tokens.
 #include "common.cuh"
 #include "attn_ranges.cuh"
+#include "distance.cuh"
 #include "sink.cuh"
 
 struct GqaArgs {
@@ -45,6 +46,7 @@ struct GqaArgs {
     int nh, nkv, page_tokens, window, chunk;  // (mask.cuh)
     const float* sink_val;    // with sink: a learned score per query head in its place (null: the score 0)
     int keep_first, sink;     // with a window: a request's first tokens stay in sight; one more term of score 0 in the denominator
+    const float* slopes;      // distance bias per query head (distance.cuh), or null
     float scale;
     float* part_o;            // [units * G][hd]
     float* part_ml;           // [units * G][2]
@@ -147,8 +149,9 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
 }
 
 // HD: head size (64 or 128).  WIDE: groups of more than 8 heads (a second tile of heads).
+// BIAS: a distance bias (an instance of its own).
 // GQW warps of a block, GQS chunks of 16 keys in flight per warp (10 x 2 for many pairs, 6 x 4 for few: see above).
-template <int HD, bool WIDE, int GQW, int GQS>
+template <int HD, bool WIDE, int GQW, int GQS, bool BIAS>
 __global__ void __launch_bounds__(32 * GQW, 1) attn_decode_gqa_kernel(GqaArgs a, int n_items, long long max_units,
                                                                            int cost_range, int cost_merge) {
     pdl_trigger();  // every block of this grid is resident from the start
@@ -224,13 +227,18 @@ __global__ void __launch_bounds__(32 * GQW, 1) attn_decode_gqa_kernel(GqaArgs a,
         // gq + 8; columns are heads 2 t4 + {0, 1} of the head tile.  m, l: of this lane's two heads per tile
         // (l: this lane's share of the keys).
         float o[HT][MT][4];
-        float m[HT][2], l[HT][2];
+        float m[HT][2], l[HT][2], slope[HT][2];
 #pragma unroll
         for (int ht = 0; ht < HT; ++ht) {
 #pragma unroll
             for (int j = 0; j < MT; ++j) o[ht][j][0] = o[ht][j][1] = o[ht][j][2] = o[ht][j][3] = 0.f;
             m[ht][0] = m[ht][1] = -INFINITY;
             l[ht][0] = l[ht][1] = 0.f;
+#pragma unroll
+            for (int c = 0; c < 2; ++c) {
+                const int g = 8 * ht + 2 * t4 + c;
+                slope[ht][c] = BIAS && g < G ? slope_log2(a.slopes, kvh * G + g) : 0.f;
+            }
         }
 
         // A stage of the warp's ring: the K tile [16 keys][hd], then the V tile, rows as they lie in the page.
@@ -308,10 +316,12 @@ __global__ void __launch_bounds__(32 * GQW, 1) attn_decode_gqa_kernel(GqaArgs a,
                 }
                 // s[0], s[1]: key k0 + gq, heads 2 t4 + {0, 1};  s[2], s[3]: key k0 + 8 + gq, the same heads
                 float sc[4];
-                sc[0] = live_lo ? (s0[0] + s1[0]) * qscale : -INFINITY;
-                sc[1] = live_lo ? (s0[1] + s1[1]) * qscale : -INFINITY;
-                sc[2] = live_hi ? (s0[2] + s1[2]) * qscale : -INFINITY;
-                sc[3] = live_hi ? (s0[3] + s1[3]) * qscale : -INFINITY;
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    sc[i] = (s0[i] + s1[i]) * qscale;
+                    if (BIAS) sc[i] = fmaf(slope[ht][i & 1], static_cast<float>(k0 + gq + 8 * (i >> 1) - p), sc[i]);
+                    if (!(i < 2 ? live_lo : live_hi)) sc[i] = -INFINITY;
+                }
                 float mx[2] = {fmaxf(sc[0], sc[2]), fmaxf(sc[1], sc[3])};
 #pragma unroll
                 for (int c = 0; c < 2; ++c) {
@@ -464,7 +474,7 @@ extern "C" int locus_attn_decode_gqa(const void* q, const void* pool, void* out,
                                      int nkv, int hd, int page_tokens, int window, int chunk, float scale, float* part_o,
                                      float* part_ml, int* counters, long long max_units, int cost_range,
                                      int cost_merge, int keep_first, int sink, const float* sink_val,
-                                     cudaStream_t stream) {
+                                     const float* slopes, cudaStream_t stream) {
     if (n_items <= 0) return 0;
     if (!locus_attn_decode_gqa_takes(LOCUS_DT_BF16, nh, nkv, hd, page_tokens, n_items) || !mask_ok(window, chunk, keep_first) || counters == nullptr)
         return LOCUS_ERR_UNSUPPORTED;
@@ -487,7 +497,7 @@ extern "C" int locus_attn_decode_gqa(const void* q, const void* pool, void* out,
     a.seg_q0 = seg_q0; a.seg_ctx = seg_ctx; a.block_table = block_table; a.table_stride = table_stride; a.items = items;
     a.nh = nh; a.nkv = nkv; a.page_tokens = page_tokens; a.window = window; a.chunk = chunk; a.scale = scale;
     a.keep_first = keep_first; a.sink = sink; a.sink_val = sink ? sink_val : nullptr;
-    a.part_o = part_o; a.part_ml = part_ml; a.counters = counters;
+    a.part_o = part_o; a.part_ml = part_ml; a.counters = counters; a.slopes = slopes;
     const dim3 grid(n_sm);
     const bool wide = nh / nkv > 8;
     // few (request, key/value head) pairs: fewer warps with a deeper ring (a warp's chain of chunks sets the time);
@@ -495,18 +505,23 @@ extern "C" int locus_attn_decode_gqa(const void* q, const void* pool, void* out,
     // 54.5 us, 16 requests (64 pairs) 66.7 against 65.8, 64 requests 230 against 184; 16 heads on 2 at 4,000 tokens:
     // 16 requests (32 pairs) 35.7 against 42.6 us, 32 requests (64 pairs) 44.6 against 45.0
     const bool few = g_gqa_deep >= 0 ? g_gqa_deep != 0 : static_cast<long long>(n_items) * nkv <= GQ_DEEP_PAIRS;
-#define GQA_LAUNCH_WS(HD_, WIDE_, W_, S_)                                                                              \
+#define GQA_LAUNCH_WSB(HD_, WIDE_, W_, S_, B_)                                                                             \
     do {                                                                                                               \
         const size_t smem = static_cast<size_t>(W_) * S_ * 2 * 16 * hd * 2;                                            \
         static bool attr_set = false;                                                                                  \
         if (!attr_set) {                                                                                               \
-            if (cudaFuncSetAttribute(attn_decode_gqa_kernel<HD_, WIDE_, W_, S_>,                                       \
+            if (cudaFuncSetAttribute(attn_decode_gqa_kernel<HD_, WIDE_, W_, S_, B_>,                                       \
                                      cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)) != cudaSuccess) \
                 return static_cast<int>(cudaGetLastError());                                                           \
             attr_set = true;                                                                                           \
         }                                                                                                              \
-        locus_launch(attn_decode_gqa_kernel<HD_, WIDE_, W_, S_>, grid, 32 * W_, smem, stream, a, n_items, max_units,   \
+        locus_launch(attn_decode_gqa_kernel<HD_, WIDE_, W_, S_, B_>, grid, 32 * W_, smem, stream, a, n_items, max_units,   \
                      cost_range, cost_merge);                                                                          \
+    } while (0)
+#define GQA_LAUNCH_WS(HD_, WIDE_, W_, S_)                                                                              \
+    do {                                                                                                               \
+        if (slopes) GQA_LAUNCH_WSB(HD_, WIDE_, W_, S_, true);                                                          \
+        else GQA_LAUNCH_WSB(HD_, WIDE_, W_, S_, false);                                                                \
     } while (0)
 #define GQA_LAUNCH(HD_, WIDE_)                                                                                         \
     do {                                                                                                               \
@@ -520,6 +535,7 @@ extern "C" int locus_attn_decode_gqa(const void* q, const void* pool, void* out,
         if (wide) GQA_LAUNCH(64, true);
         else GQA_LAUNCH(64, false);
     }
+#undef GQA_LAUNCH_WSB
 #undef GQA_LAUNCH_WS
 #undef GQA_LAUNCH
     return locus_launch_status();

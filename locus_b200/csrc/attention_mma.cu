@@ -20,6 +20,7 @@
 // caller uses the CUDA-core kernel.  Rows in shared memory are
 // padded by 16 bytes so that ldmatrix reads no bank twice.
 #include "common.cuh"
+#include "distance.cuh"
 #include "mask.cuh"
 #include "sink.cuh"
 
@@ -39,6 +40,7 @@ struct MmaAttnArgs {
     int nh, nkv, page_tokens, window, chunk;  // (mask.cuh)
     const float* sink_val;  // with sink: a learned score per query head in its place (null: the score 0)
     int keep_first, sink;   // a window that keeps a request's first tokens in sight; one more term of score 0 in the denominator
+    const float* slopes;    // distance bias per query head (distance.cuh), or null
     float scale;
     int n_splits;     // ranges of key tiles per item (1: the block writes out itself)
     float* part_o;    // [item][head][split][MQ][hd] unnormalised sums
@@ -116,6 +118,7 @@ __global__ void __launch_bounds__(128) attn_chunk_mma_kernel(MmaAttnArgs a) {
     const int P = a.page_tokens;
     const int pshift = (P & (P - 1)) == 0 ? __ffs(P) - 1 : -1;  // pages of 2^k tokens: shifts instead of divisions
     const float scale_log2 = a.scale * 1.4426950408889634f;
+    const float slope = slope_log2(a.slopes, h);
 
     // this block's range of the item's key tiles
     int first_tile, n_tiles_all, kept_tiles;
@@ -217,6 +220,15 @@ __global__ void __launch_bounds__(128) attn_chunk_mma_kernel(MmaAttnArgs a) {
         // ---- scale, mask, online softmax (rows g and g + 8 of the warp's 16), in the base-2 domain:
         // exp(x * scale - m) = exp2(x * scale * log2(e) - m').  The mask test runs only on tiles that
         // can hold a masked key for one of this warp's rows (the diagonal, the window's edge, the start).
+        float mult = scale_log2;
+        if (a.slopes != nullptr) {   // (the scores are scaled here already, then)
+            mult = 1.0f;
+#pragma unroll
+            for (int j = 0; j < MK / 8; ++j)
+#pragma unroll
+                for (int i = 0; i < 4; ++i)
+                    s[j][i] = fmaf(slope, static_cast<float>(tile0 + j * 8 + qd * 2 + (i & 1) - pq[i >> 1]), s[j][i] * scale_log2);
+        }
         float mx[2] = {m_run[0], m_run[1]};
         const bool need_mask = tile0 + MK - 1 > p_first || tile0 < lo_last;
         if (need_mask) {
@@ -227,7 +239,7 @@ __global__ void __launch_bounds__(128) attn_chunk_mma_kernel(MmaAttnArgs a) {
                     const int rr = i >> 1;
                     const int t = tile0 + j * 8 + qd * 2 + (i & 1);
                     const bool ok = t <= pq[rr] && (t >= lo_q[rr] || t < a.keep_first);
-                    const float v = ok ? s[j][i] * scale_log2 : -INFINITY;
+                    const float v = ok ? s[j][i] * mult : -INFINITY;
                     s[j][i] = v;
                     mx[rr] = fmaxf(mx[rr], v);
                 }
@@ -237,7 +249,7 @@ __global__ void __launch_bounds__(128) attn_chunk_mma_kernel(MmaAttnArgs a) {
             for (int j = 0; j < MK / 8; ++j) {
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
-                    const float v = s[j][i] * scale_log2;
+                    const float v = s[j][i] * mult;
                     s[j][i] = v;
                     mx[i >> 1] = fmaxf(mx[i >> 1], v);
                 }
@@ -393,7 +405,7 @@ extern "C" int locus_attn_chunk_mma(const void* q, const void* pool, void* out, 
                                     const int* seg_ctx, const int* block_table, int table_stride, const int* items,
                                     int n_items, int nh, int nkv, int hd, int page_tokens, int window, int chunk, float scale,
                                     int n_splits, float* part_o, float* part_ml, int keep_first, int sink, const float* sink_val,
-                                    cudaStream_t stream) {
+                                    const float* slopes, cudaStream_t stream) {
     if (n_items <= 0) return 0;
     if (nh <= 0 || nkv <= 0 || nh % nkv != 0 || nh > 65535 || page_tokens <= 0 || !mask_ok(window, chunk, keep_first))
         return LOCUS_ERR_UNSUPPORTED;
@@ -405,7 +417,7 @@ extern "C" int locus_attn_chunk_mma(const void* q, const void* pool, void* out, 
     a.seg_q0 = seg_q0; a.seg_qn = seg_qn; a.seg_ctx = seg_ctx; a.block_table = block_table;
     a.table_stride = table_stride; a.items = items; a.nh = nh; a.nkv = nkv; a.page_tokens = page_tokens;
     a.window = window; a.chunk = chunk; a.scale = scale; a.keep_first = window > 0 ? keep_first : 0; a.sink = sink; a.sink_val = sink ? sink_val : nullptr;
-    a.n_splits = n_splits; a.part_o = part_o; a.part_ml = part_ml;
+    a.n_splits = n_splits; a.part_o = part_o; a.part_ml = part_ml; a.slopes = slopes;
     switch (hd) {
         case 16: return launch<16>(a, n_items, stream);
         case 32: return launch<32>(a, n_items, stream);

@@ -28,6 +28,7 @@
 #include <string.h>
 
 #include "common.cuh"
+#include "distance.cuh"
 #include "mask.cuh"
 #include "sink.cuh"
 
@@ -51,6 +52,7 @@ struct TcAttnArgs {
     int nh, nkv, page_tokens, window, chunk;  // (mask.cuh)
     const float* sink_val;  // with sink: a learned score per query head in its place (null: the score 0)
     int keep_first, sink;   // with a window: a request's first tokens stay in sight; one more term of score 0 in the denominator
+    const float* slopes;    // distance bias per query head (distance.cuh), or null
     float scale;
     // Ranges of key tiles per block of queries (1: a block writes the result itself).  With more, a block takes
     // one range (blockIdx.z) and leaves, per query row of the step and head, its unnormalised sum, its running
@@ -223,6 +225,8 @@ __device__ __forceinline__ void at_st32(uint32_t taddr, const uint32_t* v) {
 // sum / denominator is the same number whatever reference it was formed with.
 #define AT_LAG_LOG2 8.0f
 
+// BIAS: a distance bias; an instance of its own (the softmax warps are bound by instruction issue).
+template <bool BIAS>
 __global__ void __launch_bounds__(320, 1)
 attn_chunk_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv, TcAttnArgs a) {
     extern __shared__ __align__(1024) uint8_t at_raw[];
@@ -374,7 +378,10 @@ attn_chunk_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
         const int pq = p0 + r;              // its position
         const uint32_t lane_bits = static_cast<uint32_t>(quarter * 32) << 16;
         const float scale_log2 = a.scale * 1.4426950408889634f;
-        const unsigned long long scale2 = at_pair(scale_log2, scale_log2);
+        // what a score is multiplied by behind its maximum: with a bias it is scaled when the bias is taken off
+        const float mult = BIAS ? 1.0f : scale_log2;
+        const unsigned long long scale2 = at_pair(mult, mult);
+        const float slope = BIAS ? slope_log2(a.slopes, h) : 0.f;
         float m_run = -INFINITY, l_run = 0.f;  // the row's reference maximum (base 2, scaled); this thread's part of the denominator
         uint8_t* at_generic = at_raw + (base - at_smem(at_raw));
         uint8_t* gP0 = at_generic + (sP - base) + half * AT_HALF_BYTES + r * 128;
@@ -408,6 +415,24 @@ attn_chunk_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
             // at an edge need the test (a tile of kept tokens lies in front of t_lo, so it is always tested)
             const bool need_mask = tile_first + AT_MK - 1 > p0 || tile_first < lo_last;
             float mx = -INFINITY;
+            if constexpr (BIAS) {
+                // s <- s scale - slope (pq - t), two keys at a time (t - pq is an exact float32)
+                const unsigned long long k2 = at_pair(scale_log2, scale_log2), sl2 = at_pair(slope, slope);
+                const float d0 = static_cast<float>(tile0 - pq);
+                const unsigned long long d2 = at_pair(d0, d0);
+#pragma unroll
+                for (int i = 0; i < 32; i += 2) {
+                    float x, y;
+                    const unsigned long long off0 = at_mul2(sl2, at_add2(d2, at_pair(static_cast<float>(i), static_cast<float>(i + 1))));
+                    at_unpair(at_fma2(at_pair(__uint_as_float(s0[i]), __uint_as_float(s0[i + 1])), k2, off0), x, y);
+                    s0[i] = __float_as_uint(x);
+                    s0[i + 1] = __float_as_uint(y);
+                    const unsigned long long off1 = at_mul2(sl2, at_add2(d2, at_pair(static_cast<float>(i + 32), static_cast<float>(i + 33))));
+                    at_unpair(at_fma2(at_pair(__uint_as_float(s1[i]), __uint_as_float(s1[i + 1])), k2, off1), x, y);
+                    s1[i] = __float_as_uint(x);
+                    s1[i + 1] = __float_as_uint(y);
+                }
+            }
             if (need_mask) {
 #pragma unroll
                 for (int i = 0; i < 32; ++i) {
@@ -418,7 +443,7 @@ attn_chunk_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
             }
 #pragma unroll
             for (int i = 0; i < 32; ++i) mx = at_max3(mx, __uint_as_float(s0[i]), __uint_as_float(s1[i]));
-            mx = fmaxf(mx, with_partner(b, mx)) * scale_log2;  // the scale is positive: the maximum can be scaled last
+            mx = fmaxf(mx, with_partner(b, mx)) * mult;  // the scale is positive: the maximum can be scaled last
             const float m_new = fmaxf(mx, m_run);               // the same in both threads of the row
             // The buffer of P_{j-2} is free when its product is finished (the same barrier frees the stage's V).
             if (j > 1 && !at_wait(pv_done + 8 * b, ((j >> 1) & 1) ^ 1, 9)) ok = false;
@@ -637,7 +662,7 @@ extern "C" int locus_attn_chunk_tc(const void* q, long long T, const void* pool,
                                    int table_stride, const int* items, int n_items, int nh, int nkv, int hd,
                                    int page_tokens, int window, int chunk, float scale, int n_splits, float* part_o,
                                    float* part_ml, int keep_first, int sink, const float* sink_val,
-                                   cudaStream_t stream) {
+                                   const float* slopes, cudaStream_t stream) {
     if (n_items <= 0) return 0;
     if (n_splits < 1 || n_splits > AT_MAX_SPLITS) return LOCUS_ERR_UNSUPPORTED;
     if (n_splits > 1 && (part_o == nullptr || part_ml == nullptr ||
@@ -658,17 +683,19 @@ extern "C" int locus_attn_chunk_tc(const void* q, long long T, const void* pool,
     a.block_table = block_table; a.table_stride = table_stride; a.items = items; a.nh = nh; a.nkv = nkv;
     a.page_tokens = page_tokens; a.window = window; a.chunk = chunk; a.scale = scale;
     a.keep_first = window > 0 ? keep_first : 0; a.sink = sink ? 1 : 0; a.sink_val = sink ? sink_val : nullptr;
-    a.n_splits = n_splits; a.part_o = part_o; a.part_ml = part_ml;
+    a.n_splits = n_splits; a.part_o = part_o; a.part_ml = part_ml; a.slopes = slopes;
     const size_t smem = 7 * AT_TILE_BYTES + 160 + 2 * 2 * 128 * 4;
     static bool set = false;
     if (!set) {
-        if (cudaFuncSetAttribute(attn_chunk_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+        if (cudaFuncSetAttribute(attn_chunk_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess ||
+            cudaFuncSetAttribute(attn_chunk_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
             return static_cast<int>(cudaGetLastError());
         set = true;
     }
     if (n_items > 65535) return LOCUS_ERR_UNSUPPORTED;
     dim3 grid(nh, n_items, n_splits);
-    attn_chunk_tc_kernel<<<grid, 320, smem, stream>>>(map_q, map_kv, a);
+    if (slopes != nullptr) attn_chunk_tc_kernel<true><<<grid, 320, smem, stream>>>(map_q, map_kv, a);
+    else attn_chunk_tc_kernel<false><<<grid, 320, smem, stream>>>(map_q, map_kv, a);
     if (n_splits > 1)
         attn_chunk_tc_merge_kernel<<<dim3(AT_MQ * (AT_HD / 4) / 128, n_items, nh), 128, 0, stream>>>(a);
     return locus_launch_status();

@@ -36,6 +36,9 @@ __device__ __forceinline__ float ld_dyn(const void* p, int dt, size_t i) {
                               : __bfloat162float(reinterpret_cast<const bf16*>(p)[i]);
 }
 
+// The same where the array may be absent (then 0): the biases of two products behind one activation, stored one behind the other.
+__device__ __forceinline__ float pair_bias(const void* p, int dt, size_t i) { return p ? ld_dyn(p, dt, i) : 0.f; }
+
 // Elements i .. i + 3 of such an array (i a multiple of 4, the array's start 16-byte aligned) in one load.
 __device__ __forceinline__ float4 ld4_dyn(const void* p, int dt, size_t i) {
     if (dt == LOCUS_DT_F32) return *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p) + i);

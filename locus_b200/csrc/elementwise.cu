@@ -4,33 +4,42 @@
 #include "common.cuh"
 
 // ---------------------------------------------------------------------------
-// Embedding: out[t, :] = table[tokens[t], :] as float32 (the residual stream is float32), optionally through a Dynamic
-// Tanh (see below): tanh(alpha v) w + b.
+// Embedding: out[t, :] = table[tokens[t], :] as float32 (the residual stream is float32), optionally plus a row of a table
+// of learned position vectors, optionally through a Dynamic Tanh (see below): tanh(alpha v) w + b; optionally written twice,
+// for a model that adds the embedding to the stream again later.
 __global__ void embed_rows_kernel(const int* __restrict__ tokens, const void* __restrict__ table,
                                   int table_dt, float* __restrict__ out, int H, int copies, float scale,
                                   const void* __restrict__ alpha, const void* __restrict__ w, const void* __restrict__ b,
-                                  int norm_dt) {
+                                  int norm_dt, const int* __restrict__ positions, const void* __restrict__ pos_table, int pos_dt,
+                                  float* __restrict__ keep) {
     pdl_entry();
     pdl_trigger();
     const int t = blockIdx.x;
     const size_t row = static_cast<size_t>(tokens[t]) * H;
+    const size_t pos_row = pos_table ? static_cast<size_t>(positions[t]) * H : 0;
     float* o = out + static_cast<size_t>(t) * H * copies;
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
         float v = ld_dyn(table, table_dt, row + i) * scale;
+        if (pos_table) v += ld_dyn(pos_table, pos_dt, pos_row + i);
         if (w) v = fmaf(tanhf(ld_dyn(alpha, norm_dt, 0) * v), ld_dyn(w, norm_dt, i), ld_dyn(b, norm_dt, i));
         for (int c = 0; c < copies; ++c) o[c * H + i] = v;
+        if (keep) keep[static_cast<size_t>(t) * H + i] = v;
     }
 }
 
 // scale: a factor on the row (1: none).  copies > 1: a row of out holds the table's row that many times, one behind the other (a model that keeps
 // several copies of the residual stream starts them all from the embedding).  alpha [1], w [H], b [H] (element type
-// norm_dt) or null: a Dynamic Tanh behind the factor.
+// norm_dt) or null: a Dynamic Tanh behind the factor.  pos_table [positions, H] (element type pos_dt) or null: its row
+// positions[t] is added behind the factor.  keep [T, H] or null: the rows once more.
 extern "C" int locus_embed_rows(const int* tokens, const void* table, int table_dt, float* out,
                                 int T, int H, int copies, float scale, const void* alpha, const void* w, const void* b,
-                                int norm_dt, cudaStream_t stream) {
+                                int norm_dt, const int* positions, const void* pos_table, int pos_dt, float* keep,
+                                cudaStream_t stream) {
     if (T <= 0) return 0;
+    if (pos_table != nullptr && positions == nullptr) return LOCUS_ERR_UNSUPPORTED;
     if (copies < 1 || (w != nullptr && (alpha == nullptr || b == nullptr))) return LOCUS_ERR_UNSUPPORTED;
-    locus_launch(embed_rows_kernel, T, 256, 0, stream, tokens, table, table_dt, out, H, copies, scale, alpha, w, b, norm_dt);
+    locus_launch(embed_rows_kernel, T, 256, 0, stream, tokens, table, table_dt, out, H, copies, scale, alpha, w, b, norm_dt,
+                 positions, pos_table, pos_dt, keep);
     return locus_launch_status();
 }
 
@@ -73,7 +82,8 @@ __global__ void rmsnorm_kernel(const void* __restrict__ x, int x_dt, const void*
 //
 // With add_src: first x[i] += sum over slots s < add_k (in slot order) of add_src[add_pos[i * add_k + s]]
 // (the outputs of a row's experts, the sum that moe_combine_kernel forms, in the same order), written
-// back to x, then the norm of the new row.  With rows the sum goes into the norm only and x stays as
+// back to x, then the norm of the new row.  With add_rows: x[i] += add_rows[i] as well (float32 rows, behind the sum).
+// With rows the sum goes into the norm only and x stays as
 // it was (a row may be named twice, and nobody reads the other rows' sums).
 __device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
 __device__ __forceinline__ float4 load4(const bf16* p) {
@@ -111,7 +121,8 @@ __global__ void __launch_bounds__(256) rmsnorm_f32_kernel(float* __restrict__ x,
                                                           float eps, TO* __restrict__ out,
                                                           const int* __restrict__ rows, int H,
                                                           const void* __restrict__ add_src, int add_bf16,
-                                                          const int* __restrict__ add_pos, int add_k, int vec_io) {
+                                                          const int* __restrict__ add_pos, int add_k,
+                                                          const float* __restrict__ add_rows, int vec_io) {
     __shared__ float warp_part[8];
     __shared__ float scale_s;
     const int i = blockIdx.x;
@@ -129,7 +140,7 @@ __global__ void __launch_bounds__(256) rmsnorm_f32_kernel(float* __restrict__ x,
     pdl_trigger();
     const int r = rows ? rows[i] : i;
     float4* src = reinterpret_cast<float4*>(x + static_cast<size_t>(r) * H);
-    const bool write_back = rows == nullptr;
+    const bool write_back = rows == nullptr, adds = add_src != nullptr || add_rows != nullptr;
     auto fetch = [&](int j) -> float4 {
         float4 t = src[j];
         if (add_src != nullptr) {
@@ -148,8 +159,12 @@ __global__ void __launch_bounds__(256) rmsnorm_f32_kernel(float* __restrict__ x,
                 acc.x += p.x; acc.y += p.y; acc.z += p.z; acc.w += p.w;
             }
             t.x += acc.x; t.y += acc.y; t.z += acc.z; t.w += acc.w;
-            if (write_back) src[j] = t;
         }
+        if (add_rows != nullptr) {
+            const float4 p = reinterpret_cast<const float4*>(add_rows + static_cast<size_t>(r) * H)[j];
+            t.x += p.x; t.y += p.y; t.z += p.z; t.w += p.w;
+        }
+        if (adds && write_back) src[j] = t;
         return t;
     };
     // second reading of a row too wide for the registers: x holds the sum already unless it was left alone
@@ -195,17 +210,18 @@ __global__ void __launch_bounds__(256) rmsnorm_f32_kernel(float* __restrict__ x,
     for (int j = threadIdx.x + 1024; j < n4; j += 256) store4(dst, w, j << 2, fetch_again(j), scale, wide);
 }
 
-// add_src (float32 or bfloat16 rows, add_dt) / add_pos / add_k: see rmsnorm_f32_kernel; only with float32 x, H a
-// multiple of 4, 16-byte aligned x and add_src.
+// add_src (float32 or bfloat16 rows, add_dt) / add_pos / add_k and add_rows: see rmsnorm_f32_kernel; only with float32 x,
+// H a multiple of 4, 16-byte aligned x, add_src and add_rows.
 extern "C" int locus_rmsnorm(void* x, int x_dt, const void* w, int w_dt, float eps, void* out,
                              int out_dt, const int* rows, int n_rows, int H, const void* add_src, int add_dt,
-                             const int* add_pos, int add_k, cudaStream_t stream) {
+                             const int* add_pos, int add_k, const float* add_rows, cudaStream_t stream) {
     if (n_rows <= 0) return 0;
     const bool fast = x_dt == LOCUS_DT_F32 && H % 4 == 0 && (reinterpret_cast<uintptr_t>(x) & 15) == 0;
     if (add_src != nullptr &&
         (!fast || add_pos == nullptr || add_k <= 0 || (reinterpret_cast<uintptr_t>(add_src) & 15) ||
          (add_dt != LOCUS_DT_F32 && add_dt != LOCUS_DT_BF16)))
         return LOCUS_ERR_UNSUPPORTED;
+    if (add_rows != nullptr && (!fast || (reinterpret_cast<uintptr_t>(add_rows) & 15))) return LOCUS_ERR_UNSUPPORTED;
     const int add_bf16 = add_dt == LOCUS_DT_BF16 ? 1 : 0;
     // weights and output rows start on 16-byte boundaries (H % 4 == 0 keeps every row of out aligned for 4 elements)
     const int vec_io = ((reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(out)) & 15) == 0 ? 1 : 0;
@@ -213,7 +229,7 @@ extern "C" int locus_rmsnorm(void* x, int x_dt, const void* w, int w_dt, float e
         float* xf = static_cast<float*>(x);
 #define NORM_LAUNCH(TW, TO)                                                                             \
         locus_launch(rmsnorm_f32_kernel<TW, TO>, n_rows, 256, 0, stream, xf, static_cast<const TW*>(w), eps,      \
-                     static_cast<TO*>(out), rows, H, add_src, add_bf16, add_pos, add_k, vec_io)
+                     static_cast<TO*>(out), rows, H, add_src, add_bf16, add_pos, add_k, add_rows, vec_io)
         if (w_dt == LOCUS_DT_BF16 && out_dt == LOCUS_DT_BF16) NORM_LAUNCH(bf16, bf16);
         else if (w_dt == LOCUS_DT_F32 && out_dt == LOCUS_DT_F32) NORM_LAUNCH(float, float);
         else if (w_dt == LOCUS_DT_F32 && out_dt == LOCUS_DT_BF16) NORM_LAUNCH(float, bf16);
@@ -222,6 +238,27 @@ extern "C" int locus_rmsnorm(void* x, int x_dt, const void* w, int w_dt, float e
         return locus_launch_status();
     }
     rmsnorm_kernel<<<n_rows, 256, 0, stream>>>(x, x_dt, w, w_dt, eps, out, out_dt, rows, H);
+    return locus_launch_status();
+}
+
+// x += y, n float32 elements, four to a thread (one where the tail is shorter).
+__global__ void __launch_bounds__(256) add_rows_kernel(float* __restrict__ x, const float* __restrict__ y, long long n, int wide) {
+    pdl_entry();
+    pdl_trigger();
+    const long long i = (static_cast<long long>(blockIdx.x) * 256 + threadIdx.x) * 4;
+    if (wide && i + 4 <= n) {
+        float4 a = load4(x + i);
+        const float4 b = load4(y + i);
+        put4(x + i, a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w);
+        return;
+    }
+    for (long long j = i; j < n && j < i + 4; ++j) x[j] += y[j];
+}
+
+extern "C" int locus_add_rows(float* x, const float* y, long long n, cudaStream_t stream) {
+    if (n <= 0) return 0;
+    const int wide = ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(y)) & 15) == 0 ? 1 : 0;
+    locus_launch(add_rows_kernel, dim3(static_cast<unsigned>((n + 1023) / 1024)), dim3(256), 0, stream, x, y, n, wide);
     return locus_launch_status();
 }
 

@@ -30,7 +30,8 @@ struct GemmArgs {
     int accumulate;          // out (float32) += result
     int act;                 // 0: none; 1: relu(v)^2 (after the bias, before the row scale); 2 (with w2): the clamped
                              // gated unit g' sigmoid(1.702 g') (u' + 1), g' = min(s g, limit), u' = clamp(s u, +-limit),
-                             // s the row's scale, which then stands for a factor on the input
+                             // s the row's scale, which then stands for a factor on the input; 4 (with w2): relu(v + b) (u + b2),
+                             // then the row scale (`bias` is [2N]: b and behind it b2)
     float act_param;         // the limit of act 2; the cap of act 3 (without w2): cap tanh(act_scale v / cap), behind everything else
     float act_scale;
     const float* row_scale;  // or null: row m is scaled by row_scale[scale_rows ? scale_rows[m] : m]
@@ -144,11 +145,13 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(GemmArgs a) {
                 const float g = fminf(v * rs, a.act_param);
                 const float u = fminf(fmaxf(acc2[i][j] * rs, -a.act_param), a.act_param);
                 v = g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
+            } else if (SWIGLU && a.act == 4) {
+                v = fmaxf(v + pair_bias(a.bias, a.bias_dt, n), 0.f) * (acc2[i][j] + pair_bias(a.bias, a.bias_dt, a.N + n));
             } else if (SWIGLU) {
                 const float g = v;
                 v = g / (1.0f + expf(-g)) * acc2[i][j];
             }
-            if (a.bias) v += ld_dyn(a.bias, a.bias_dt, n);
+            if (a.bias && a.act != 4) v += ld_dyn(a.bias, a.bias_dt, n);
             if (a.act == 1) {
                 v = fmaxf(v, 0.f);
                 v *= v;
@@ -179,8 +182,9 @@ static int launch(const GemmArgs& a, int max_tiles, bool swiglu, cudaStream_t st
 }
 
 // x_dt / w_dt: element types of x and of W (and W2).  flags: bit 0 = add the result into the float32 out,
-// bits 1-2 = the activation: 1 squared ReLU (not with W2), 2 the clamped gated unit with limit act_param (with W2),
-// 3 act_param tanh(act_scale v / act_param) (not with W2).  max_tiles: number of 64-row tiles
+// bits 1-3 = the activation: 1 squared ReLU (not with W2), 2 the clamped gated unit with limit act_param (with W2),
+// 3 act_param tanh(act_scale v / act_param) (not with W2), 4 relu(x . W + b) (x . W2 + b2) (with W2; bias is then [2N], b and
+// behind it b2, or null).  max_tiles: number of 64-row tiles
 // to launch; for a grouped product an upper bound (tiles past *n_tiles return at once).
 extern "C" int locus_gemm_simt(const void* x, int x_dt, const void* w, const void* w2, int w_dt,
                                const void* bias, int bias_dt, void* out, int out_dt,
@@ -191,8 +195,8 @@ extern "C" int locus_gemm_simt(const void* x, int x_dt, const void* w, const voi
                                const int* tile_rows, const int* n_tiles, int max_tiles,
                                long long w_expert_stride, cudaStream_t stream) {
     if (N <= 0 || K <= 0) return LOCUS_ERR_UNSUPPORTED;
-    const int accumulate = flags & 1, act = (flags >> 1) & 3;
-    if ((act == 1 && w2 != nullptr) || (act == 2 && w2 == nullptr) || (act == 3 && (w2 != nullptr || !(act_param > 0.f)))) return LOCUS_ERR_UNSUPPORTED;
+    const int accumulate = flags & 1, act = (flags >> 1) & 7;
+    if ((act == 1 && w2 != nullptr) || ((act == 2 || act == 4) && w2 == nullptr) || act > 4 || (act == 3 && (w2 != nullptr || !(act_param > 0.f)))) return LOCUS_ERR_UNSUPPORTED;
     if (accumulate && out_dt != LOCUS_DT_F32) return LOCUS_ERR_UNSUPPORTED;
     if (x_rows != nullptr && x_row_div <= 0) return LOCUS_ERR_UNSUPPORTED;
     GemmArgs a;

@@ -66,6 +66,7 @@ struct TcArgs {
               // the clamped gated unit g' sigmoid(1.702 g') (u' + 1), g' = min(s g, limit), u' = clamp(s u, +-limit), s the
               // row's scale (then a factor on the input)
     float act_param;  // the limit of act 2; the cap of act 3 (one weight, never split): cap tanh(act_scale v / cap), behind everything else
+    // act 4 (two weights, never split): relu(v + b) (u + b2), then the row's scale; `bias` is then [2N], b and behind it b2
     float act_scale;
     void* out;
     int out_dt;
@@ -165,8 +166,9 @@ __device__ __forceinline__ void tmem_ld16(uint32_t taddr, uint32_t* v) {
 // The loader runs ahead across tile boundaries, so the pipeline never drains between tiles, and
 // two accumulator buffers in tensor memory let the MMAs of the next tile run while the epilogue
 // warps drain this one.
-// (CAP: the tanh of activation 3, an instance of its own so that the other products' unrolled epilogue does not carry it.)
-template <bool DUAL, bool CAP = false>
+// (ALT: an epilogue with an instance of its own, so that the other products' unrolled epilogue does not carry it: the tanh
+// of activation 3 with one weight matrix, the rectified gate of activation 4 with two.)
+template <bool DUAL, bool ALT = false>
 __global__ void __launch_bounds__(192, 1)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_w2,
                const __grid_constant__ XMaps maps_x, TcArgs a) {
@@ -391,6 +393,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
             g1 = g2;
             g2 = g3;
             const float bias = (a.bias && n_ok) ? ld_dyn(a.bias, a.bias_dt, n) : 0.f;
+            const float bias2 = (ALT && DUAL && n_ok) ? pair_bias(a.bias, a.bias_dt, a.N + n) : 0.f;
             // Wide stores: the warp's 32 output columns x 16 token rows go through a small transpose in
             // shared memory so that a lane writes 8 consecutive columns of one token (16 or 32 bytes).
             const long long n_warp = static_cast<long long>(tx) * TILE_W + quarter * 32;
@@ -433,7 +436,13 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                 }
                 asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
                 float val[16];
-                if (DUAL && a.act == 2) {
+                if (DUAL && ALT) {
+#pragma unroll
+                    for (int j = 0; j < 16; ++j) {
+                        val[j] = fmaxf(__uint_as_float(v[j]) + bias, 0.f) * (__uint_as_float(u[j]) + bias2);
+                        if (a.row_scale) val[j] *= scales[c0 + j];
+                    }
+                } else if (DUAL && a.act == 2) {
                     const float lim = a.act_param;
 #pragma unroll
                     for (int j = 0; j < 16; ++j) {
@@ -456,7 +465,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                         x *= x;
                     }
                     if (a.row_scale) x *= scales[c0 + j];
-                    if (CAP) x = a.act_param * tanhf(x * a.act_scale / a.act_param);
+                    if (ALT && !DUAL) x = a.act_param * tanhf(x * a.act_scale / a.act_param);
                     val[j] = x;
                 }
                 if (wide) {
@@ -622,8 +631,8 @@ extern "C" int locus_gemm_tc(const void* x, long long x_rows_total, long long ld
                              const int* tile_rows, const int* n_tiles, int max_tiles, float* split_scratch,
                              int splits, cudaStream_t stream) {
     const int dual = w2 != nullptr ? 1 : 0;
-    const int accumulate = flags & 1, act = (flags >> 1) & 3;  // bit 0: add into out; bits 1-2: the activation
-    if ((act == 1 && (dual || splits > 1)) || (act == 2 && (!dual || splits > 1)) ||
+    const int accumulate = flags & 1, act = (flags >> 1) & 7;  // bit 0: add into out; bits 1-3: the activation
+    if ((act == 1 && (dual || splits > 1)) || ((act == 2 || act == 4) && (!dual || splits > 1)) || act > 4 ||
         (act == 3 && (dual || splits > 1 || !(act_param > 0.f))))
         return LOCUS_ERR_UNSUPPORTED;
     if (N <= 0 || K <= 0 || K % 8 != 0 || ldx % 8 != 0) return LOCUS_ERR_UNSUPPORTED;
@@ -695,6 +704,7 @@ extern "C" int locus_gemm_tc(const void* x, long long x_rows_total, long long ld
     if (!attr_set) {
         if (cudaFuncSetAttribute(gemm_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess ||
             cudaFuncSetAttribute(gemm_tc_kernel<false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess ||
+            cudaFuncSetAttribute(gemm_tc_kernel<true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess ||
             cudaFuncSetAttribute(gemm_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess)
             return static_cast<int>(cudaGetLastError());
         attr_set = true;
@@ -709,7 +719,8 @@ extern "C" int locus_gemm_tc(const void* x, long long x_rows_total, long long ld
     }
     const long long n_units = n_tiles_all * a.splits;
     const unsigned grid = static_cast<unsigned>(n_units < n_sm ? n_units : n_sm);
-    if (dual) gemm_tc_kernel<true><<<grid, 192, smem, stream>>>(map_w, map_w2, maps_x, a);
+    if (dual && act == 4) gemm_tc_kernel<true, true><<<grid, 192, smem, stream>>>(map_w, map_w2, maps_x, a);
+    else if (dual) gemm_tc_kernel<true><<<grid, 192, smem, stream>>>(map_w, map_w2, maps_x, a);
     else if (act == 3) gemm_tc_kernel<false, true><<<grid, 192, smem, stream>>>(map_w, map_w2, maps_x, a);
     else gemm_tc_kernel<false><<<grid, 192, smem, stream>>>(map_w, map_w2, maps_x, a);
     if (split) {

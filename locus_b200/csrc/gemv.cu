@@ -24,6 +24,7 @@ struct GemvArgs {
     int accumulate;
     int act;  // 1: relu(v)^2 after the bias, before the row scale; 2 (two weights): the clamped gated unit of gemm_simt.cu;
               // 3 (one weight): act_param tanh(act_scale v / act_param), behind everything else
+              // 4 (two weights): relu(v + b) (u + b2), then the row scale (`bias` is [2N]: b and behind it b2)
     float act_param, act_scale;
     const float* row_scale;
     const int* scale_rows;
@@ -173,10 +174,12 @@ __global__ void __launch_bounds__(32 * GV_WARPS) rowstream_kernel(GemvArgs a) {
         if (DUAL && a.act == 2) {
             const float g = fminf(v * rs, a.act_param), uc = fminf(fmaxf(u * rs, -a.act_param), a.act_param);
             v = g / (1.0f + expf(-1.702f * g)) * (uc + 1.0f);
+        } else if (DUAL && a.act == 4) {
+            v = fmaxf(v + pair_bias(a.bias, a.bias_dt, n), 0.f) * (u + pair_bias(a.bias, a.bias_dt, a.N + n));
         } else if (DUAL) {
             v = v / (1.0f + expf(-v)) * u;
         }
-        if (a.bias) v += ld_dyn(a.bias, a.bias_dt, n);
+        if (a.bias && a.act != 4) v += ld_dyn(a.bias, a.bias_dt, n);
         if (a.act == 1) {
             v = fmaxf(v, 0.f);
             v *= v;
@@ -215,8 +218,8 @@ extern "C" int locus_gemv(const void* x, int x_dt, const void* w, const void* w2
                           const int* tile_rows, const int* n_tiles, int max_tiles, long long w_expert_stride,
                           cudaStream_t stream) {
     if (N <= 0 || K <= 0 || K % 8 != 0 || ldx % 8 != 0) return LOCUS_ERR_UNSUPPORTED;
-    const int accumulate = flags & 1, act = (flags >> 1) & 3;  // the flags of locus_gemm_simt
-    if ((act == 1 && w2 != nullptr) || (act == 2 && w2 == nullptr) || (act == 3 && (w2 != nullptr || !(act_param > 0.f)))) return LOCUS_ERR_UNSUPPORTED;
+    const int accumulate = flags & 1, act = (flags >> 1) & 7;  // the flags of locus_gemm_simt
+    if ((act == 1 && w2 != nullptr) || ((act == 2 || act == 4) && w2 == nullptr) || act > 4 || (act == 3 && (w2 != nullptr || !(act_param > 0.f)))) return LOCUS_ERR_UNSUPPORTED;
     if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(w2)) & 31)
         return LOCUS_ERR_UNSUPPORTED;
     if (accumulate && out_dt != LOCUS_DT_F32) return LOCUS_ERR_UNSUPPORTED;

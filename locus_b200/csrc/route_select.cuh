@@ -8,7 +8,7 @@
 // selection scores = scores (+ sel_bias, which never enters the weights); with n_group > 1 only the
 // n_group_used groups with the largest group score stay eligible (the others are masked to -1e30); a group's score
 // is the sum of its two best selection scores or, with GROUP_SCORE_BEST among the flags of score_fn, its best one; k rounds of arg-max with strict '>' (ties to the lowest index); weight = score / wsum *
-// scale, wsum = sum of the picked scores when renorm, else 1.
+// scale, wsum = sum of the picked scores when renorm (of sigmoid scores: + 1e-20), else 1.
 #define SCORE_SOFTMAX 0
 #define SCORE_SIGMOID 1
 #define SCORE_FN_MASK 15      // score_fn: the score function in the low bits, flags above them
@@ -140,7 +140,8 @@ __device__ __forceinline__ void select_token(const float* __restrict__ lg, float
         wsum += w;
         __syncwarp();
     }
-    const float div = o.renorm ? wsum : 1.0f;
+    // (sigmoid scores may all be close to 0: the tiny term keeps the quotient a number, and is lost beside any other sum)
+    const float div = o.renorm ? wsum + ((o.score_fn & SCORE_FN_MASK) == SCORE_SIGMOID ? 1e-20f : 0.f) : 1.0f;
     if (in_lanes) {
         if (lane < k) wts[t * k + lane] = my_w / div * o.scale;
     } else if (lane == 0) {

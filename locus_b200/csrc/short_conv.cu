@@ -9,7 +9,8 @@
 //                    the head with a weight per channel (norm 3), the rotation of the pairs (i, i + rot/2), or of the
 //                    adjacent pairs (2i, 2i + 1), of the first `rot` channels of a q or k head by position *
 //                    inv_freq[i], and for q and k the division by sqrt(mean(x^2) + eps) (norm 1) or sqrt(sum(x^2) +
-//                    eps) (norm 2) and q's factor.  The result goes, in the output's element type, to q's rows and to k's and
+//                    eps) (norm 2) and q's factors: a constant one, and one that grows with the logarithm of the position,
+//                    1 + coef ln(floor((p + 1) / every) + 1).  The result goes, in the output's element type, to q's rows and to k's and
 //                    v's rows or cache pages, laid out at `laid` elements per head (zeros behind the head's own).
 //                    With gates (a gated delta rule's), one more warp per token forms beta = sigmoid(b) and
 //                    decay = exp(-exp(A_log) * softplus(a + dt_bias)) for every head.
@@ -44,6 +45,8 @@ struct PrepArgs {
     const void* norm_w[2];    // norm 3: q's and k's weights [dim], shared by the heads
     int norm_w_dt;
     float eps, q_scale, inv_dim[3];   // (inv_dim: 1 / dim)
+    float temp_coef;          // 0: no factor by position
+    double temp_every;
     void* q_out;              // [T, heads[0] * laid[0]]
     void* k_out;              // rows [T, heads[1] * laid[1]] and v_out alike, or, with pool set, unused
     void* v_out;
@@ -58,6 +61,11 @@ struct PrepArgs {
     const void* dt_bias;
     int gate_dt;
 };
+
+// q's factor at position p.  The quotient is floored where it cannot have been rounded across an integer: in float64.
+__device__ __forceinline__ float q_temperature(const PrepArgs& a, int p) {
+    return fmaf(a.temp_coef, logf(static_cast<float>(floor((static_cast<double>(p) + 1.0) / a.temp_every)) + 1.0f), 1.0f);
+}
 
 template <typename T>
 __global__ void __launch_bounds__(128) head_prep_kernel(const PrepArgs a) {
@@ -137,6 +145,7 @@ __global__ void __launch_bounds__(128) head_prep_kernel(const PrepArgs a) {
         r = a.norm == 1 ? 1.0f / sqrtf(ss / static_cast<float>(d) + a.eps) : 1.0f / sqrtf(ss + a.eps);
     }
     if (which == 0) r *= a.q_scale;
+    if (which == 0 && a.temp_coef != 0.f) r *= q_temperature(a, a.positions[row]);
     T* dst;
     if (which == 0) {
         dst = static_cast<T*>(a.q_out) + (row * nq + head) * laid;
@@ -154,13 +163,14 @@ __global__ void __launch_bounds__(128) head_prep_kernel(const PrepArgs a) {
 // LANES lanes to a head (4 channels each, SLOTS times), 32 / LANES heads to a warp.  Rows 0 .. gridDim.x - 1.
 template <typename T, int LANES, int SLOTS>
 __global__ void __launch_bounds__(32 * ROWS_WARPS) head_rows_kernel(const PrepArgs a) {
-    __shared__ float cs[PREP_MAX_DIM / 2], sn[PREP_MAX_DIM / 2];
+    __shared__ float cs[PREP_MAX_DIM / 2], sn[PREP_MAX_DIM / 2], q_factor;
     __shared__ __align__(16) float xch[ROWS_WARPS][PREP_MAX_DIM];   // half-split pairs: a warp's rows, read at the partner's place
     const size_t row = blockIdx.x;
     const int half = a.inv_freq != nullptr ? a.rot / 2 : 0;
     // (positions, slots and frequencies were on the device before the step's first kernel)
     const float pos = static_cast<float>(a.positions[row]);
     for (int i = threadIdx.x; i < half; i += 32 * ROWS_WARPS) sincosf(pos * a.inv_freq[i], &sn[i], &cs[i]);
+    if (threadIdx.x == 0) q_factor = a.temp_coef != 0.f ? a.q_scale * q_temperature(a, a.positions[row]) : a.q_scale;
     const int slot = a.pool != nullptr ? a.slots[row] : 0;
     const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5, sub = lane & (LANES - 1);
     const int nq = a.heads[0], nk = a.heads[1], n_units = nq + nk + a.heads[2];
@@ -250,7 +260,7 @@ __global__ void __launch_bounds__(32 * ROWS_WARPS) head_rows_kernel(const PrepAr
                     }
             }
         }
-        float r = which == 0 ? a.q_scale : 1.0f;
+        float r = which == 0 ? q_factor : 1.0f;
         if (a.norm == 1 || a.norm == 2) {
             const float ss = sum_sq();
             if (which < 2) r *= a.norm == 1 ? 1.0f / sqrtf(ss / static_cast<float>(d) + a.eps) : 1.0f / sqrtf(ss + a.eps);
@@ -328,12 +338,12 @@ static bool laid_alike(const PrepArgs& a) {
 // of q_out, k_out, v_out and the pool.  pool: the layer's pages (k and v go there, at slots[t]) or null (k_out, v_out).
 // n_rows > 0: the segments' rows are proj's rows 0 .. n_rows - 1 without a gap (head_rows_kernel runs where it can).
 // adjacent: rotate the pairs (2i, 2i + 1) instead of (i, i + rot/2).  norm 3: q_norm_w, k_norm_w [dim] of element type
-// norm_w_dt.  gates: beta, decay [T, gate_heads] float32 from columns off_b, off_a of proj, or beta null.
+// norm_w_dt.  temp_coef, temp_every: q's factor by position (0: none).  gates: beta, decay [T, gate_heads] float32 from columns off_b, off_a of proj, or beta null.
 extern "C" int locus_head_prep(const float* proj, int ld, const int* sizes, const void* conv, int conv_dt, int taps, int act,
                                float* conv_state, long long slot_stride, int move_state, const int* state_slots,
                                const int* seg_q0, const int* seg_qn, int n_seg, int longest_new, int n_rows,
                                const int* positions, const float* inv_freq, int rot, int adjacent, int norm, const void* q_norm_w,
-                               const void* k_norm_w, int norm_w_dt, float eps, float q_scale, void* q_out, void* k_out,
+                               const void* k_norm_w, int norm_w_dt, float eps, float q_scale, float temp_coef, double temp_every, void* q_out, void* k_out,
                                void* v_out, void* pool, const int* slots, int page_tokens, int write_kv, int out_dt,
                                float* beta, float* decay, int off_b, int off_a, int gate_heads, const void* a_log,
                                const void* dt_bias, int gate_dt, cudaStream_t stream) {
@@ -348,6 +358,7 @@ extern "C" int locus_head_prep(const float* proj, int ld, const int* sizes, cons
     }
     if (taps < 1 || taps > PREP_MAX_TAPS || n_seg > 65535 || longest_new > 65535) return LOCUS_ERR_UNSUPPORTED;
     if (rot < 0 || rot % 2 || rot > a.dim[0] || rot > a.dim[1] || (rot > 0 && inv_freq == nullptr)) return LOCUS_ERR_UNSUPPORTED;
+    if (temp_coef != 0.f && !(temp_every > 0.0)) return LOCUS_ERR_UNSUPPORTED;
     if (conv != nullptr && taps > 1 && conv_state == nullptr) return LOCUS_ERR_UNSUPPORTED;
     if (norm < 0 || norm > 3 || (norm == 3 && (q_norm_w == nullptr || (k_norm_w == nullptr && a.heads[1] > 0)))) return LOCUS_ERR_UNSUPPORTED;
     if (pool != nullptr && (a.laid[1] != a.laid[2] || page_tokens <= 0 || slots == nullptr)) return LOCUS_ERR_UNSUPPORTED;
@@ -356,6 +367,7 @@ extern "C" int locus_head_prep(const float* proj, int ld, const int* sizes, cons
     a.conv_state = conv_state; a.slot_stride = slot_stride; a.state_slots = state_slots; a.seg_q0 = seg_q0; a.seg_qn = seg_qn;
     a.positions = positions; a.inv_freq = inv_freq; a.rot = rot; a.adjacent = adjacent; a.norm = norm;
     a.norm_w[0] = q_norm_w; a.norm_w[1] = k_norm_w; a.norm_w_dt = norm_w_dt; a.eps = eps; a.q_scale = q_scale;
+    a.temp_coef = temp_coef; a.temp_every = temp_every;
     a.q_out = q_out; a.k_out = k_out; a.v_out = v_out; a.pool = pool; a.slots = slots; a.page_tokens = page_tokens;
     a.write_kv = write_kv; a.beta = beta; a.decay = decay; a.off_b = off_b; a.off_a = off_a; a.gate_heads = gate_heads;
     a.a_log = a_log; a.dt_bias = dt_bias; a.gate_dt = gate_dt;

@@ -200,18 +200,29 @@ F = ctypes.c_float
 
 # ---------------------------------------------------------------------------
 def embed_rows(tokens: torch.Tensor, table: torch.Tensor, out: torch.Tensor, copies: int = 1, scale: float = 1.0,
-               dyt_norm=None) -> None:
+               dyt_norm=None, positions: Optional[torch.Tensor] = None, pos_table: Optional[torch.Tensor] = None,
+               keep: Optional[torch.Tensor] = None) -> None:
     """out[t, :] = table[tokens[t], :] * scale as float32; ``copies`` > 1: the row that many times, one behind the
-    other (``out`` [T, copies * H]).  ``dyt_norm`` = (alpha, weight, bias): the row through :func:`dyt`'s norm."""
+    other (``out`` [T, copies * H]).  ``dyt_norm`` = (alpha, weight, bias): the row through :func:`dyt`'s norm.
+    ``pos_table`` [positions, H] with ``positions`` [T] int32: row positions[t] is added behind the factor.  ``keep`` [T, H]
+    float32: the rows once more."""
     _i32(tokens, "tokens")
     _cuda_c(table, "table")
     _cuda_c(out, "out")
     T, H = out.shape[0], table.shape[1]
     _need(out.dtype == torch.float32, "embed_rows: out must be float32")
     _need(tokens.numel() == T and copies >= 1 and out.shape[1] == H * copies, "embed_rows: shape mismatch")
+    if pos_table is not None:
+        _cuda_c(pos_table, "pos_table")
+        _need(positions is not None and pos_table.shape[1] == H and positions.numel() >= T, "embed_rows: positions and their table")
+        _i32(positions, "positions")
+    if keep is not None:
+        _cuda_c(keep, "keep")
+        _need(keep.dtype == torch.float32 and tuple(keep.shape) == (T, H), "embed_rows: keep must be float32 [T, H]")
     code = _lib("elementwise").locus_embed_rows(
         _p(tokens), _p(table), I(dtype_code(table.dtype)), _p(out), I(T), I(H), I(copies), F(scale),
-        *_dyt_args(dyt_norm, H), _stream()
+        *_dyt_args(dyt_norm, H), _p(positions), _p(pos_table), I(dtype_code(pos_table.dtype) if pos_table is not None else 0),
+        _p(keep), _stream()
     )
     _check(code, "embed_rows")
 
@@ -262,17 +273,18 @@ def dyt(x: torch.Tensor, norm=None, out: Optional[torch.Tensor] = None, rows: Op
 
 
 def rmsnorm_adds(x: torch.Tensor) -> bool:
-    """Whether :func:`rmsnorm` can fold a pending expert sum into rows like ``x``'s."""
+    """Whether :func:`rmsnorm` can fold a pending addition into rows like ``x``'s."""
     return x.dtype == torch.float32 and x.shape[-1] % 4 == 0
 
 
 def rmsnorm(x: torch.Tensor, w: torch.Tensor, eps: float, out: torch.Tensor,
-            rows: Optional[torch.Tensor] = None, add=None) -> None:
+            rows: Optional[torch.Tensor] = None, add=None, add_rows: Optional[torch.Tensor] = None) -> None:
     """out[i] = x[rows[i] if rows else i] * rsqrt(mean(x^2) + eps) * w  (statistics in float32).
 
     ``add`` = (pair_out, pair_pos, top_k): first x[i] += the sum that :func:`moe_combine` forms (same
     order), written back to ``x``; needs :func:`rmsnorm_adds`.  With ``rows`` the sum enters the norm
-    of the gathered rows only and ``x`` stays as it was."""
+    of the gathered rows only and ``x`` stays as it was.  ``add_rows`` (float32 rows like ``x``'s): added in the same way,
+    behind that sum."""
     _cuda_c(x, "x")
     _cuda_c(w, "w")
     _cuda_c(out, "out")
@@ -294,10 +306,13 @@ def rmsnorm(x: torch.Tensor, w: torch.Tensor, eps: float, out: torch.Tensor,
         _need(add_src.dtype in (torch.float32, torch.bfloat16) and add_src.shape[-1] == H
               and add_pos.numel() >= (n if rows is None else x.shape[0]) * add_k,
               "rmsnorm: expert sum of another shape")
+    if add_rows is not None:
+        _cuda_c(add_rows, "add_rows")
+        _need(rmsnorm_adds(x) and add_rows.dtype == torch.float32 and add_rows.shape == x.shape, "rmsnorm: add_rows must be float32 rows like x's")
     code = _lib("elementwise").locus_rmsnorm(
         _p(x), I(dtype_code(x.dtype)), _p(w), I(dtype_code(w.dtype)), F(eps), _p(out),
         I(dtype_code(out.dtype)), _p(rows), I(n), I(H), _p(add_src),
-        I(dtype_code(add_src.dtype) if add_src is not None else 0), _p(add_pos), I(add_k), _stream()
+        I(dtype_code(add_src.dtype) if add_src is not None else 0), _p(add_pos), I(add_k), _p(add_rows), _stream()
     )
     _check(code, "rmsnorm")
 
@@ -479,7 +494,7 @@ def expert_tile(n_pairs: int, n_experts: int) -> int:
 
 
 # activations of a product's epilogue, by their code in the kernels' flags
-ACTIVATIONS = {None: 0, "relu2": 1, "glu_clamp": 2, "softcap": 3}
+ACTIVATIONS = {None: 0, "relu2": 1, "glu_clamp": 2, "softcap": 3, "reglu": 4}
 
 
 def tc_error() -> int:
@@ -500,6 +515,7 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, w2: Optional[
     ``act`` = "glu_clamp" (with ``w2``): the clamped gated unit out = g sigmoid(1.702 g) (u + 1) with g = min(s x . w^T,
     ``act_limit``), u = clamp(s x . w2^T, -act_limit, act_limit), where s is the row's ``row_scale`` (1 without): the
     scale then stands for a factor on the row of x and is not applied once more behind the activation.  ``act`` =
+    "reglu" (with ``w2``): max(x . w^T + b, 0) * (x . w2^T + b2), ``bias`` being [2 N], b and behind it b2.  ``act`` =
     "softcap" (not with ``w2``): ``act_limit`` * tanh(``act_scale`` * v / ``act_limit``) behind everything else.  ``bias`` [N] is added, ``row_scale`` [M]
     multiplies the row (``scale_rows``: row m uses row_scale[scale_rows[m]]), ``accumulate`` adds the result into the float32 ``out``.
     ``x_rows``: logical row m reads x[x_rows[m] // x_row_div].  ``layout``: grouped product,
@@ -526,13 +542,13 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, w2: Optional[
         _need(w2.shape == w.shape and w2.dtype == w.dtype and w2.is_contiguous(), "linear: w2 must match w")
     if accumulate:
         _need(out.dtype == torch.float32, "linear: accumulate needs a float32 out")
-    _need(act in ACTIVATIONS and not (act == "relu2" and w2 is not None) and not (act == "glu_clamp" and (w2 is None or not act_limit > 0))
+    _need(act in ACTIVATIONS and not (act == "relu2" and w2 is not None) and not (act == "reglu" and w2 is None) and not (act == "glu_clamp" and (w2 is None or not act_limit > 0))
           and not (act == "softcap" and (w2 is not None or not act_limit > 0)),
-          f"linear: activation {act!r} (known: relu2 without w2; glu_clamp with w2 and a positive act_limit; softcap without "
+          f"linear: activation {act!r} (known: relu2 without w2; reglu with w2; glu_clamp with w2 and a positive act_limit; softcap without "
           "w2 and with a positive act_limit)")
     flags = I((1 if accumulate else 0) | (ACTIVATIONS[act] << 1))
     if bias is not None:
-        _need(bias.numel() == N and bias.is_contiguous(), "linear: bias size")
+        _need(bias.numel() == (2 * N if act == "reglu" else N) and bias.is_contiguous(), "linear: bias size")
     if row_scale is not None:
         _need(row_scale.dtype == torch.float32 and row_scale.is_contiguous(), "linear: row_scale must be float32")
         if scale_rows is not None:
@@ -671,16 +687,26 @@ def _sink_args(sink, n_heads: int):
     return I(1 if sink else 0), None
 
 
+def _slopes_arg(slopes: Optional[torch.Tensor], n_heads: int):
+    """Pointer of a distance bias's slopes (float32 [n_heads] on the device; None: no bias)."""
+    if slopes is not None:
+        _need(slopes.is_cuda and slopes.dtype == torch.float32 and slopes.is_contiguous() and slopes.numel() == n_heads,
+              "attention: the slopes of a distance bias must be float32 [n_heads] on the device")
+    return _p(slopes)
+
+
 def attn_chunk(q: torch.Tensor, pool: torch.Tensor, out: torch.Tensor, *, seg_q0: torch.Tensor,
                seg_qn: torch.Tensor, seg_ctx: torch.Tensor, block_table: torch.Tensor,
                items: torch.Tensor, n_items: int, n_heads: int, n_kv_heads: int, head_dim: int,
-               page_tokens: int, window: int, scale: float, keep_first: int = 0, sink=False, chunk: int = 0) -> None:
+               page_tokens: int, window: int, scale: float, keep_first: int = 0, sink=False, chunk: int = 0,
+               slopes: Optional[torch.Tensor] = None) -> None:
     """Attention of portions of prompts: ``items`` [n_items, 2] = (segment, first query of a
     16-query tile).  Keys come from the cache through ``block_table`` [n_seg, width].  ``keep_first``: with a
     window, a request's first that many tokens stay in sight of every later query; ``sink``: the softmax has one
     more term in its denominator that has no value: True for the score 0, a float32 tensor [n_heads] for a learned
     score per head (taken as it is, not multiplied by ``scale``).  ``chunk`` > 0 (without a window): a query sees the keys of
-    its own chunk of that many positions, counted from position 0, up to itself."""
+    its own chunk of that many positions, counted from position 0, up to itself.  ``slopes`` [n_heads] float32: a distance
+    bias, slopes[h] * (p - t) is taken off the scaled score of a query at position p with the key at t."""
     _cuda_c(q, "q")
     _cuda_c(out, "out")
     _cuda_c(pool, "pool")
@@ -690,7 +716,8 @@ def attn_chunk(q: torch.Tensor, pool: torch.Tensor, out: torch.Tensor, *, seg_q0
     code = _lib("attention").locus_attn_chunk(
         _p(q), I(dtype_code(q.dtype)), _p(pool), _p(out), _p(seg_q0), _p(seg_qn), _p(seg_ctx),
         _p(block_table), I(block_table.shape[1]), _p(items), I(n_items), I(n_heads), I(n_kv_heads),
-        I(head_dim), I(page_tokens), I(window), I(chunk), F(scale), I(keep_first), *_sink_args(sink, n_heads), _stream()
+        I(head_dim), I(page_tokens), I(window), I(chunk), F(scale), I(keep_first), *_sink_args(sink, n_heads),
+        _slopes_arg(slopes, n_heads), _stream()
     )
     _check(code, "attn_chunk", f"(heads {n_heads}/{n_kv_heads}, head_dim {head_dim})")
 
@@ -733,7 +760,7 @@ def attn_chunk_mma(q: torch.Tensor, pool: torch.Tensor, out: torch.Tensor, *, se
                    items: torch.Tensor, n_items: int, n_heads: int, n_kv_heads: int, head_dim: int,
                    page_tokens: int, window: int, scale: float, n_splits: int = 1,
                    part_o: Optional[torch.Tensor] = None, part_ml: Optional[torch.Tensor] = None,
-                   keep_first: int = 0, sink=False, chunk: int = 0) -> None:
+                   keep_first: int = 0, sink=False, chunk: int = 0, slopes: Optional[torch.Tensor] = None) -> None:
     """Attention of portions of prompts on the tensor cores: ``items`` [n_items, 2] =
     (segment, first query of a 64-query tile); otherwise as :func:`attn_chunk`.  ``n_splits`` > 1
     (:func:`attn_chunk_mma_splits`) with scratch of :func:`attn_chunk_mma_scratch` floats: the keys of
@@ -753,7 +780,7 @@ def attn_chunk_mma(q: torch.Tensor, pool: torch.Tensor, out: torch.Tensor, *, se
         _p(q), _p(pool), _p(out), _p(seg_q0), _p(seg_qn), _p(seg_ctx), _p(block_table), I(block_table.shape[1]),
         _p(items), I(n_items), I(n_heads), I(n_kv_heads), I(head_dim), I(page_tokens), I(window), I(chunk), F(scale),
         I(n_splits), _p(part_o if n_splits > 1 else None), _p(part_ml if n_splits > 1 else None), I(keep_first),
-        *_sink_args(sink, n_heads), _stream()
+        *_sink_args(sink, n_heads), _slopes_arg(slopes, n_heads), _stream()
     )
     if n_splits > 1 and code == 0:
         _count_launches(1)
@@ -806,13 +833,13 @@ def attn_chunk_tc(q: torch.Tensor, pool: torch.Tensor, out: torch.Tensor, *, seg
                   items: torch.Tensor, n_items: int, n_heads: int, n_kv_heads: int, head_dim: int,
                   page_tokens: int, window: int, scale: float, n_splits: int = 1,
                   part_o: Optional[torch.Tensor] = None, part_ml: Optional[torch.Tensor] = None,
-                  keep_first: int = 0, sink=False, chunk: int = 0) -> None:
+                  keep_first: int = 0, sink=False, chunk: int = 0, slopes: Optional[torch.Tensor] = None) -> None:
     """Attention of portions of prompts with tcgen05 tensor cores (scores and sums in tensor memory):
     ``items`` as for :func:`attn_chunk_mma` (tiles of 64 queries; a block takes an even one and the 64 queries
     behind it).  ``n_splits`` > 1 (:func:`attn_chunk_tc_splits`) with scratch of :func:`attn_chunk_tc_scratch`
     floats: the key tiles of every block are cut into that many ranges, merged in ascending order by a second
     kernel.  ``keep_first`` (with a window): a request's first tokens stay in sight; ``sink``: one more term of score 0
-    in the softmax's denominator; ``chunk`` as for :func:`attn_chunk`."""
+    in the softmax's denominator; ``chunk``, ``slopes`` as for :func:`attn_chunk`."""
     _cuda_c(q, "q")
     _cuda_c(out, "out")
     _cuda_c(pool, "pool")
@@ -830,7 +857,8 @@ def attn_chunk_tc(q: torch.Tensor, pool: torch.Tensor, out: torch.Tensor, *, seg
         _p(q), LL(q.shape[0]), _p(pool), LL(pool.shape[0]), _p(out), _p(seg_q0), _p(seg_qn), _p(seg_ctx),
         _p(block_table), I(block_table.shape[1]), _p(items), I(n_items), I(n_heads), I(n_kv_heads), I(head_dim),
         I(page_tokens), I(window), I(chunk), F(scale), I(n_splits), _p(part_o if n_splits > 1 else None),
-        _p(part_ml if n_splits > 1 else None), I(keep_first if window > 0 else 0), *_sink_args(sink, n_heads), _stream()
+        _p(part_ml if n_splits > 1 else None), I(keep_first if window > 0 else 0), *_sink_args(sink, n_heads),
+        _slopes_arg(slopes, n_heads), _stream()
     )
     if n_splits > 1 and code == 0:
         _count_launches(1)
@@ -935,9 +963,9 @@ def attn_decode(q: torch.Tensor, pool: torch.Tensor, out: torch.Tensor, *, seg_q
                 items: torch.Tensor, n_items: int, n_heads: int, n_kv_heads: int, head_dim: int,
                 page_tokens: int, window: int, scale: float, part_o: torch.Tensor,
                 part_ml: torch.Tensor, counters: torch.Tensor, max_splits: int, keep_first: int = 0,
-                sink=False, chunk: int = 0) -> None:
-    """Attention of single new tokens: ``items`` [n_items] = segments with one new token.  ``keep_first``, ``sink``, ``chunk``
-    as for :func:`attn_chunk` (the streaming kernels, per head and per group of query heads, walk the kept tokens in front
+                sink=False, chunk: int = 0, slopes: Optional[torch.Tensor] = None) -> None:
+    """Attention of single new tokens: ``items`` [n_items] = segments with one new token.  ``keep_first``, ``sink``, ``chunk``,
+    ``slopes`` as for :func:`attn_chunk` (the streaming kernels, per head and per group of query heads, walk the kept tokens in front
     of the window as one more range of the request and want scratch for two ranges per request and head, the kernel whose
     ranges are fixed for ``max_splits``: :func:`decode_units` with ``fixed_ranges``).
 
@@ -965,7 +993,7 @@ def attn_decode(q: torch.Tensor, pool: torch.Tensor, out: torch.Tensor, *, seg_q
             I(n_items), I(n_heads), I(n_kv_heads), I(head_dim), I(page_tokens), I(window), I(chunk), F(scale), _p(part_o),
             _p(part_ml), _p(counters), ctypes.c_longlong(max_units), I(GQA_COST_RANGE),
             I(GQA_COST_MERGE_PER_HEAD * (n_heads // n_kv_heads)), I(keep_first if window > 0 else 0), *_sink_args(sink, n_heads),
-            _stream()
+            _slopes_arg(slopes, n_heads), _stream()
         )
         _check(code, "attn_decode", f"(grouped queries; heads {n_heads}/{n_kv_heads}, head_dim {head_dim})")
         return
@@ -973,7 +1001,8 @@ def attn_decode(q: torch.Tensor, pool: torch.Tensor, out: torch.Tensor, *, seg_q
         _p(q), I(dtype_code(q.dtype)), _p(pool), _p(out), _p(seg_q0), _p(seg_qn), _p(seg_ctx),
         _p(block_table), I(block_table.shape[1]), _p(items), I(n_items), I(n_heads), I(n_kv_heads),
         I(head_dim), I(page_tokens), I(window), I(chunk), F(scale), _p(part_o), _p(part_ml), _p(counters), I(max_splits),
-        ctypes.c_longlong(max_units), I(keep_first if window > 0 else 0), *_sink_args(sink, n_heads), _stream()
+        ctypes.c_longlong(max_units), I(keep_first if window > 0 else 0), *_sink_args(sink, n_heads), _slopes_arg(slopes, n_heads),
+        _stream()
     )
     _check(code, "attn_decode", f"(heads {n_heads}/{n_kv_heads}, head_dim {head_dim})")
 
@@ -1210,6 +1239,15 @@ def moe_combine(x: torch.Tensor, pair_out: torch.Tensor, pair_pos: torch.Tensor,
     code = _lib("elementwise").locus_moe_combine(_p(x), _p(pair_out), I(dtype_code(pair_out.dtype)), _p(pair_pos), I(T),
                                                  I(top_k), I(H), _stream())
     _check(code, "moe_combine")
+
+
+def add_rows(x: torch.Tensor, y: torch.Tensor) -> None:
+    """x += y, float32 rows of one shape."""
+    _cuda_c(x, "x")
+    _cuda_c(y, "y")
+    _need(x.dtype == y.dtype == torch.float32 and x.shape == y.shape, "add_rows: float32 rows of one shape")
+    code = _lib("elementwise").locus_add_rows(_p(x), _p(y), LL(x.numel()), _stream())
+    _check(code, "add_rows")
 
 
 def gather_rows(src: torch.Tensor, idx: torch.Tensor, div: int, out: torch.Tensor, n: int) -> None:
@@ -1739,7 +1777,7 @@ def head_prep(proj: torch.Tensor, *, offsets, heads, dims, laid, state_slots: to
               conv_offset: int = 0, move_state: bool = True, act: bool = False,
               inv_freq: Optional[torch.Tensor] = None, rot: int = 0, norm: Optional[str] = None, eps: float = 0.0,
               q_scale: float = 1.0, gates=None, interleaved: bool = False, norm_weights=None,
-              n_rows: int = 0) -> None:
+              n_rows: int = 0, q_temp=None) -> None:
     """From the float32 rows ``proj`` of a stacked projection to q in rows and k, v in rows or cache pages, in one
     launch.  ``offsets``, ``heads``, ``dims``, ``laid``: for q, k, v the first column in ``proj``, the number of heads,
     the per-head size and the size a head is laid out at in the output (zeros behind its own elements).  In this
@@ -1751,7 +1789,9 @@ def head_prep(proj: torch.Tensor, *, offsets, heads, dims, laid, state_slots: to
     by sqrt(mean(x^2) + eps) per head, "unit": by sqrt(sum(x^2) + eps), "head": by sqrt(mean(x^2) + eps) and multiplied by
     ``norm_weights`` = (q's, k's) [dim] in FRONT of the rotation; ``interleaved``: the rotation takes the pairs (2i, 2i + 1)
     instead; ``n_rows`` > 0: the segments' rows are the rows 0 .. n_rows - 1 of ``proj`` without a gap (the kernel of a block
-    per token then runs where it can); ``q_scale`` on q.  The outputs share one
+    per token then runs where it can); ``q_scale`` on q; ``q_temp`` = (coef, every): q also
+    multiplied by 1 + coef * ln(floor((p + 1) / every) + 1) at position p.  ``offsets`` may name one stretch twice (values that
+    are the keys as projected).  The outputs share one
     element type; with ``pool`` (a layer's pages [n_pages, 2, heads_k, page_tokens, laid]) k and v go to ``slots``.
     ``gates`` = (beta, decay, off_b, off_a, a_log, dt_bias): also beta = sigmoid(proj[:, off_b + h]) and decay =
     exp(-exp(a_log[h]) * softplus(proj[:, off_a + h] + dt_bias[h])), [T, heads] float32 each."""
@@ -1785,6 +1825,7 @@ def head_prep(proj: torch.Tensor, *, offsets, heads, dims, laid, state_slots: to
         _need(inv_freq.dtype == torch.float32 and inv_freq.is_cuda and inv_freq.numel() == rot // 2, "head_prep: inv_freq [rot / 2]")
     q_w, k_w = norm_weights if norm_weights is not None else (None, None)
     _need((norm == "head") == (q_w is not None), "head_prep: norm_weights go with the norm 'head'")
+    _need(q_temp is None or q_temp[1] > 0, "head_prep: q_temp (coef, every) needs a positive every")
     for t, which in ((q_w, 0), (k_w, 1)):
         _need(t is None or (t.is_cuda and t.is_contiguous() and t.numel() == dims[which] and t.dtype == q_w.dtype), "head_prep: norm_weights [dim]")
     beta = decay = a_log = dt_bias = None
@@ -1801,7 +1842,7 @@ def head_prep(proj: torch.Tensor, *, offsets, heads, dims, laid, state_slots: to
         I(1 if act else 0), state_ptr, LL(stride), I(1 if move_state else 0), _p(state_slots), _p(seg_q0), _p(seg_qn),
         I(n_seg), I(longest_new), I(n_rows), _p(positions), _p(inv_freq), I(rot if inv_freq is not None else 0),
         I(1 if interleaved else 0), I(HEAD_NORMS[norm]), _p(q_w), _p(k_w), I(dtype_code(q_w.dtype) if q_w is not None else 0),
-        F(eps), F(q_scale), _p(q_out), _p(k_out), _p(v_out), _p(pool), _p(slots), I(page_tokens), I(1 if write_kv else 0),
+        F(eps), F(q_scale), F(q_temp[0] if q_temp else 0.0), D(q_temp[1] if q_temp else 1.0), _p(q_out), _p(k_out), _p(v_out), _p(pool), _p(slots), I(page_tokens), I(1 if write_kv else 0),
         I(dtype_code(out_dt)), _p(beta), _p(decay), I(off_b), I(off_a), I(gate_heads), _p(a_log), _p(dt_bias), I(gate_dt),
         _stream())
     if code == 0 and conv is not None and taps > 1 and move_state and n_seg > 0 and longest_new > 0:

@@ -12,7 +12,7 @@ import torch
 
 from ..config.base import load_config
 from ..engine.batch import LayerCache, Runtime, StepBatch
-from ..parts.base import (ModelPlan, PagedKvSpec, Part, PartSpec, StateSpec, TensorSource,
+from ..parts.base import (ModelPlan, PagedKvSpec, Part, PartSpec, PendingRows, StateSpec, TensorSource,
                           iter_parts, make_part)
 
 
@@ -49,6 +49,9 @@ class Model:
                     raise ValueError(f"run order entry {i}: cache_of must name an earlier entry")
                 if plan.order[call.cache_of].cache_of is not None:
                     raise ValueError(f"run order entry {i}: cache_of must name an entry with a cache of its own")
+        self.adds_embedding = any(call.add_embedding for call in plan.order)
+        if self.adds_embedding and plan.residual_streams != 1:
+            raise ValueError("the embedding is added again to one residual stream only")
         self.rt: Optional[Runtime] = None
         self.loaded = False
 
@@ -113,11 +116,17 @@ class Model:
         T = batch.T
         x = rt.rows("model.x", self.plan.hidden_size * self.plan.residual_streams, torch.float32, T)
         order = self.plan.order
-        if len(caches) > len(order):
-            self.embedding.forward(batch.tokens, x, batch=batch, cache=caches[len(order)])
-        else:
-            self.embedding.forward(batch.tokens, x)
+        e = rt.rows("model.embedding", self.plan.hidden_size, torch.float32, T) if self.adds_embedding else None
+        self.embedding.forward(batch.tokens, x, batch=batch, cache=caches[len(order)] if len(caches) > len(order) else None,
+                               **({"keep": e} if e is not None else {}))
         for i, (call, cache) in enumerate(zip(order, caches)):
+            if call.add_embedding:
+                again = PendingRows(e, rt.take_pending())
+                if self.blocks[call.layer].takes_pending_add:
+                    rt.defer_add = True
+                    rt.leave_pending(again)
+                else:
+                    again.apply(x)
             # a block may leave its last addition to the residual stream to the next block's first norm,
             # the last block to the final norm
             rt.defer_add = i + 1 == len(order) or self.blocks[order[i + 1].layer].takes_pending_add

@@ -27,7 +27,10 @@ the whole q and the whole k projection, all heads at once, in front of the rotat
 sigmoid(W_g h) in front of the output projection (``out_gate``); a layer without keys and values of its own
 (``has_kv`` off: it reads the cache of the layer call that the run order names); an RMS norm per head with a weight that
 the heads share, in front of the rotation (``qk_norm`` "head"); a mask of chunks in the place of a window (``chunk``: a query
-sees the keys of its own chunk of that many positions, counted from position 0, up to itself).  With any of these (or ``shaped``)
+sees the keys of its own chunk of that many positions, counted from position 0, up to itself); values that are the keys as
+projected, in front of their norm and rotation (``values`` "keys": no W_v); a factor on q that grows with the logarithm of
+its position (``q_temp`` = (coef, every): 1 + coef ln(floor((p + 1) / every) + 1)); a linear distance bias on the scores
+(``slopes``, one per query head: slope * (i - j) is taken off).  With any of these (or ``shaped``)
 the projections are one product into float32 rows [q | k | v | gate] at the stored sizes, and one kernel
 (``kernels.head_prep``) convolves, rotates, norms and writes q and the cache pages at the kernels' head size in
 float32 arithmetic, so that padded heads take a rotation there too.
@@ -100,11 +103,12 @@ class Attention(Mixer):
                  v_dim: Optional[int] = None, out_scale: float = 1.0, names: Optional[dict] = None,
                  keep_first: int = 0, sink: bool = False, conv_taps: int = 0, qk_norm: Optional[str] = None,
                  qk_norm_eps: float = 0.0, out_gate: bool = False, has_kv: bool = True, shaped: bool = False,
-                 cache_window: Optional[int] = None, cache_keep: Optional[int] = None, chunk: int = 0) -> None:
+                 cache_window: Optional[int] = None, cache_keep: Optional[int] = None, chunk: int = 0,
+                 values: str = "own", q_temp: Optional[tuple] = None, slopes: Optional[tuple] = None) -> None:
         """``v_dim``: the values' size per head where it is not ``head_dim``.  ``out_scale``: a factor on the mixer's
         output (a mixer that runs beside another one).  ``names``: tensor names below the prefix where they differ
         from ``NAMES``.  ``keep_first``, ``sink``, ``conv_taps``, ``qk_norm``, ``out_gate``, ``has_kv``,
-        ``shaped``, ``chunk``: see the head of the file.  ``cache_window`` / ``cache_keep``: what the layer's pages must hold
+        ``shaped``, ``chunk``, ``values``, ``q_temp``, ``slopes``: see the head of the file.  ``cache_window`` / ``cache_keep``: what the layer's pages must hold
         where that is more than its own window and kept tokens (another layer call reads them with a wider mask)."""
         super().__init__(prefix)
         self.keep_first, self.sink = (int(keep_first) if window else 0), bool(sink)
@@ -113,7 +117,18 @@ class Attention(Mixer):
         self.sink_learned = sink == "learned"
         self.conv_taps, self.qk_norm, self.qk_norm_eps = int(conv_taps), qk_norm, float(qk_norm_eps)
         self.out_gate, self.has_kv = bool(out_gate), bool(has_kv)
-        self.shaped = bool(shaped or self.conv_taps > 0 or qk_norm or out_gate or not has_kv)
+        if values not in ("own", "keys"):
+            raise ValueError(f"attention: values {values!r} (known: 'own', 'keys')")
+        self.keys_are_values = values == "keys"
+        if self.keys_are_values and (self.conv_taps > 0 or v_dim not in (None, head_dim) or qkv_bias):
+            raise ValueError("attention: values that are the keys have their size, and go with no convolution and no biases")
+        self.q_temp = (float(q_temp[0]), float(q_temp[1])) if q_temp and float(q_temp[0]) != 0.0 else None
+        if self.q_temp and not self.q_temp[1] > 0:
+            raise ValueError(f"attention: q_temp {q_temp} needs a positive second number")
+        self.slopes = tuple(float(s) for s in slopes) if slopes is not None else None
+        if self.slopes is not None and len(self.slopes) != n_heads:
+            raise ValueError(f"attention: {len(self.slopes)} slopes for {n_heads} heads")
+        self.shaped = bool(shaped or self.conv_taps > 0 or qk_norm or out_gate or not has_kv or self.keys_are_values or self.q_temp)
         if qk_norm == "whole" and self.conv_taps > 0:
             raise ValueError("attention: a norm over the whole projections does not go with a convolution behind them")
         if self.conv_taps > K.PREP_MAX_TAPS:
@@ -149,7 +164,7 @@ class Attention(Mixer):
         kv = self.n_kv_heads if self.has_kv else 0
         self.in_rows = [("q", 0, n_heads * self.qk_dim)]
         self.in_rows.append(("k", self.in_rows[-1][1] + self.in_rows[-1][2], kv * self.qk_dim))
-        self.in_rows.append(("v", self.in_rows[-1][1] + self.in_rows[-1][2], kv * self.v_dim))
+        self.in_rows.append(("v", self.in_rows[-1][1] + self.in_rows[-1][2], 0 if self.keys_are_values else kv * self.v_dim))
         self.in_rows.append(("gate", self.in_rows[-1][1] + self.in_rows[-1][2], n_heads * self.v_dim if self.out_gate else 0))
         self.in_used = self.in_rows[-1][1] + self.in_rows[-1][2]
         self.in_width = -(-self.in_used // 8) * 8
@@ -243,6 +258,9 @@ class Attention(Mixer):
 
     def bind(self, rt) -> None:
         self._scale = None
+        self._slopes = None
+        if self.slopes is not None:
+            self._slopes = rt.shared_object(("slopes", self.slopes), lambda: torch.tensor(self.slopes, dtype=torch.float32, device=rt.device))
         # what the kernels get as the sink: a flag, or the learned scores as float32
         self._sink_arg = self.params["sink"].float().contiguous() if self.sink_learned else self.sink
         if self.out_scale != 1.0:
@@ -317,7 +335,11 @@ class Attention(Mixer):
             if kv:
                 spans.append((self.in_rows[1][1], self.in_rows[1][2], self.params["k_norm"]))
             K.span_rmsnorm(proj, spans, self.qk_norm_eps)
-        K.head_prep(proj, offsets=[r[1] for r in self.in_rows[:3]], heads=(self.n_heads, kv, kv),
+        offsets = [r[1] for r in self.in_rows[:3]]
+        if self.keys_are_values:
+            offsets[2] = offsets[1]
+        extra = {"q_temp": self.q_temp} if self.q_temp else {}
+        K.head_prep(proj, offsets=offsets, heads=(self.n_heads, kv, kv),
                     dims=(self.qk_dim, self.qk_dim, self.v_dim), laid=(D, D, D), state_slots=batch.state_slots,
                     seg_q0=batch.seg_q0, seg_qn=batch.seg_qn, n_seg=batch.n_seg,
                     longest_new=max(batch.host_seg_qn) if batch.host_seg_qn else T, positions=batch.positions, q_out=q,
@@ -326,7 +348,7 @@ class Attention(Mixer):
                     inv_freq=table.inv_freq if table else None, rot=table.rot_dim if table else 0,
                     interleaved=table.interleaved if table else False, n_rows=T,
                     norm=None if self.qk_norm == "whole" else self.qk_norm, eps=self.qk_norm_eps,
-                    norm_weights=(self.params["q_norm"], self.params.get("k_norm")) if self.qk_norm == "head" else None)
+                    norm_weights=(self.params["q_norm"], self.params.get("k_norm")) if self.qk_norm == "head" else None, **extra)
         o = rt.rows("attention.o", self.q_dim, rt.dtype, T)
         self._attend(q, o, batch, cache, gb, rt)
         if self.out_gate:
@@ -365,6 +387,8 @@ class Attention(Mixer):
         extra = dict(keep_first=self.keep_first, sink=self._sink_arg) if special else {}
         if self.chunk:
             extra["chunk"] = self.chunk
+        if self._slopes is not None:
+            extra["slopes"] = self._slopes
         common = dict(seg_q0=batch.seg_q0, seg_qn=batch.seg_qn, seg_ctx=batch.seg_ctx,
                       block_table=gb.block_table, n_heads=self.n_heads, n_kv_heads=self.n_kv_heads,
                       head_dim=self.head_dim, page_tokens=gb.page_tokens, window=self.window,

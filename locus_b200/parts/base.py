@@ -43,10 +43,12 @@ class LayerSpec:
 @dataclass(frozen=True)
 class LayerCall:
     """One entry of the run order: run ``layer``; ``cache_of`` names an earlier entry of the
-    order (by its index) whose cache this call reads instead of keeping its own."""
+    order (by its index) whose cache this call reads instead of keeping its own.  ``add_embedding``: what the
+    embedding gave is added to the residual stream once more in front of this call."""
 
     layer: int
     cache_of: Optional[int] = None
+    add_embedding: bool = False
 
 
 @dataclass
@@ -180,6 +182,21 @@ class PendingAdd(Pending):
         K.moe_combine(x, self.pair_out, self.pair_pos, self.top_k)
 
 
+class PendingRows(Pending):
+    """Rows that the model adds to the residual stream between two layer calls: x += y, behind what the call in front
+    left (``before``, if anything)."""
+
+    def __init__(self, y: torch.Tensor, before: Optional[Pending] = None) -> None:
+        self.y, self.before = y, before
+
+    def apply(self, x: torch.Tensor) -> None:
+        from .. import kernels as K
+
+        if self.before is not None:
+            self.before.apply(x)
+        K.add_rows(x, self.y)
+
+
 class PendingNorm(Pending):
     """What an arrangement with norms behind its sublayers leaves: x += scale * norm(y) (``scale`` [width] or None)."""
 
@@ -270,6 +287,11 @@ class Mixer(Part):
 
 class FeedForward(Part):
     can_overwrite = False   # as for Mixer
+
+    def leaves_residual_alone(self, residual: torch.Tensor, rt: "Runtime") -> bool:
+        """Whether ``forward`` would not touch ``residual`` now, but leave its whole sum pending: it may then run beside
+        whatever writes ``residual``."""
+        return False
 
     def forward(self, h: torch.Tensor, batch: "StepBatch", residual: torch.Tensor, rt: "Runtime") -> None:
         """Add the feed-forward output of ``h`` into ``residual`` (float32)."""

@@ -16,7 +16,9 @@ norm sits on the sum.
 ``SandwichNorm``: x += s1 * norm1b(mixer(norm1(x))); x += s2 * norm2b(feed_forward(norm2(x))): norms on both sides of a
 sublayer and optional layer scales.
 
-``Embedding``: x = table[token] (llama.cpp:450); optionally plus a row of a second table addressed by a hash of the
+``ParallelPreNorm``: x += mixer(norm1(x)) + feed_forward(norm1(x)): one norm, both sublayers read its output.
+
+``Embedding``: x = table[token] (llama.cpp:450); optionally plus a learned vector per position; optionally plus a row of a second table addressed by a hash of the
 previous and the current token.  ``LmHead``: logits = W . h in float32,
 W being the embedding table when the head is tied (llama.cpp:292-297, 512-513): the head then
 names the embedding's tensor as the source of its weight.
@@ -66,6 +68,54 @@ class PreNorm(Arrangement):
             return
         self.norm2.forward(x, h)
         self.ff.forward(h, batch, x, rt)
+
+
+# Up to this many tokens in a step the feed-forward of a parallel block runs beside the mixer on the side stream: kernels of
+# a decode step leave most of the GPU idle, and neither sublayer waits for the other.
+PARALLEL_OVERLAP_TOKENS = 64
+
+
+class ParallelPreNorm(Arrangement):
+    """Both sublayers on one norm's output: h = norm1(x); x += mixer(h) + feed_forward(h).  ``feed_forward`` may be absent
+    (kind "none").  In steps of few tokens the feed-forward runs on the runtime's side stream while the mixer runs, up to what
+    writes the residual stream: a dense one's last product follows the mixer's, a routed one's sum is left pending."""
+
+    takes_pending_add = True
+
+    def __init__(self, prefix: str, *, hidden: int, norm: PartSpec, mixer: PartSpec, feed_forward: PartSpec,
+                 mixer_prefix: str = "mix", ff_prefix: str = "mlp", norm_name: str = "norm1") -> None:
+        super().__init__(prefix)
+        self.hidden = int(hidden)
+        # the norm's tensor carries the plain name of the norm (no ".weight" behind it)
+        name = f"{prefix}.{norm_name}"
+        self.norm1 = make_part("norm", PartSpec(norm.kind, {**norm.args, "tensor": name}), name)
+        self.mixer = make_part("mixer", mixer, f"{prefix}.{mixer_prefix}")
+        self.ff = None if feed_forward.kind == "none" else make_part("feed_forward", feed_forward, f"{prefix}.{ff_prefix}")
+
+    def sub_parts(self):
+        return [self.norm1, self.mixer] + ([self.ff] if self.ff is not None else [])
+
+    def forward(self, x, batch, cache, rt) -> None:
+        T = batch.T
+        h = rt.rows("block.h", self.hidden, rt.dtype, T)
+        self.norm1.forward(x, h, add=rt.take_pending())
+        ff = self.ff
+        beside = ff is not None and T <= PARALLEL_OVERLAP_TOKENS
+        if beside and hasattr(ff, "forward_down"):
+            with rt.side():
+                act = ff.forward_up(h, rt)
+            self.mixer.forward(h, batch, cache, x, rt)
+            rt.join()
+            ff.forward_down(act, x, rt)
+        elif beside and ff.leaves_residual_alone(x, rt):
+            with rt.side():
+                ff.forward(h, batch, x, rt)
+            self.mixer.forward(h, batch, cache, x, rt)
+            rt.join()
+        else:
+            self.mixer.forward(h, batch, cache, x, rt)
+            if ff is not None:
+                ff.forward(h, batch, x, rt)
 
 
 class OutputNorm(Arrangement):
@@ -345,14 +395,16 @@ class StreamedPreNorm(Arrangement):
 
 class Embedding(Part):
     def __init__(self, prefix: str, *, vocab: int, hidden: int, tensor: str = "", copies: int = 1,
-                 scale: float = 1.0, pair: Optional[dict] = None, norm: Optional[PartSpec] = None) -> None:
+                 scale: float = 1.0, pair: Optional[dict] = None, norm: Optional[PartSpec] = None,
+                 positions: Optional[dict] = None) -> None:
         """``tensor``: the checkpoint tensor's name where it is not ``<prefix>.weight``.  ``copies`` > 1: a row of the
         output holds the embedding that many times (a model with several copies of the residual stream).  ``scale``:
         a factor on the embedding, applied in float32.  ``pair`` = {tensor, buckets, mul_prev, mul_cur}: a second table
         of buckets + 1 rows whose row (previous token * mul_prev + token * mul_cur) mod buckets is added (its last row for
         a request's first token).  The token that a request's last step ended on is kept in the request's state slot
         (``state_needs``), so that a prompt may be cut anywhere.  ``norm``: a norm over the row behind all of this (the
-        residual stream then starts from its float32 result)."""
+        residual stream then starts from its float32 result).  ``positions`` = {tensor, count}: a table of learned position
+        vectors [count, hidden] whose row of the token's position is added behind the factor."""
         super().__init__(prefix)
         self.norm = make_part("norm", norm, prefix + ".norm") if norm is not None else None
         if self.norm is not None and int(copies) != 1:
@@ -360,9 +412,10 @@ class Embedding(Part):
         self.vocab, self.hidden, self.copies, self.scale = int(vocab), int(hidden), int(copies), float(scale)
         self.tensor = str(tensor or prefix + ".weight")
         self.pair = dict(pair) if pair else None
+        self.positions = dict(positions) if positions else None
         if self.pair is not None:
-            if self.copies != 1 or self.scale != 1.0:
-                raise ValueError("embedding: the pair table goes with one copy and no factor")
+            if self.copies != 1 or self.scale != 1.0 or self.positions is not None:
+                raise ValueError("embedding: the pair table goes with one copy, no factor and no position vectors")
             if int(self.pair["buckets"]) <= 0 or int(self.pair["mul_prev"]) < 0 or int(self.pair["mul_cur"]) < 0:
                 raise ValueError("embedding: the pair table needs positive buckets and multipliers that are not negative")
 
@@ -370,12 +423,16 @@ class Embedding(Part):
         s = {"table": (self.vocab, self.hidden)}
         if self.pair is not None:
             s["pair"] = (int(self.pair["buckets"]) + 1, self.hidden)
+        if self.positions is not None:
+            s["positions"] = (int(self.positions["count"]), self.hidden)
         return s
 
     def sources(self):
         out = [TensorSource(self.tensor, (self.vocab, self.hidden), "table")]
         if self.pair is not None:
             out.append(TensorSource(str(self.pair["tensor"]), (int(self.pair["buckets"]) + 1, self.hidden), "pair"))
+        if self.positions is not None:
+            out.append(TensorSource(str(self.positions["tensor"]), (int(self.positions["count"]), self.hidden), "positions"))
         return out
 
     def kernel_modules(self, dtype):
@@ -388,7 +445,17 @@ class Embedding(Part):
         """What the embedding keeps per request: the last token it saw, when it has a pair table."""
         return StateSpec((1,), torch.int32) if self.pair is not None else None
 
-    def forward(self, tokens: torch.Tensor, out: torch.Tensor, batch=None, cache=None) -> None:
+    def forward(self, tokens: torch.Tensor, out: torch.Tensor, batch=None, cache=None, keep: Optional[torch.Tensor] = None) -> None:
+        """``keep``: float32 rows that receive what ``out`` starts as (a model that adds it again later)."""
+        extra = {}
+        if self.positions is not None:
+            if batch is None:
+                raise ValueError("embedding: learned position vectors need the step's positions")
+            extra = {"positions": batch.positions, "pos_table": self.params["positions"]}
+        if keep is not None:
+            if self.pair is not None or self.norm is not None or self.copies != 1:
+                raise ValueError("embedding: the rows can be kept where one copy leaves the lookup's kernel as it is")
+            extra["keep"] = keep
         if self.pair is not None:
             if batch is None or cache is None or cache.state is None:
                 raise ValueError("embedding: a pair table needs the step's segments and the requests' state slots")
@@ -400,10 +467,10 @@ class Embedding(Part):
                 self.norm.forward(out, out)
             return
         if isinstance(self.norm, DynamicTanh):
-            K.embed_rows(tokens, self.params["table"], out, scale=self.scale, dyt_norm=self.norm.tensors())
+            K.embed_rows(tokens, self.params["table"], out, scale=self.scale, dyt_norm=self.norm.tensors(), **extra)
             return
-        if self.copies > 1 or self.scale != 1.0:
-            K.embed_rows(tokens, self.params["table"], out, copies=self.copies, scale=self.scale)
+        if self.copies > 1 or self.scale != 1.0 or extra:
+            K.embed_rows(tokens, self.params["table"], out, copies=self.copies, scale=self.scale, **extra)
         else:
             K.embed_rows(tokens, self.params["table"], out)
         if self.norm is not None:
@@ -445,6 +512,7 @@ class LmHead(Part):
 
 register_arrangement("pre_norm", PreNorm)
 register_arrangement("output_norm", OutputNorm)
+register_arrangement("parallel_pre_norm", ParallelPreNorm)
 register_arrangement("streamed_pre_norm", StreamedPreNorm)
 register_arrangement("post_norm", PostNorm)
 register_arrangement("sandwich_norm", SandwichNorm)

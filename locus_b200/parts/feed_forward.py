@@ -15,7 +15,8 @@ Further forms: ``activation`` "relu2" (down(max(up h, 0)^2), no gate matrix) and
 
     g = min(W_gate h, limit),  u = clamp(W_up h, -limit, limit),  out = W_down (g sigmoid(1.702 g) (u + 1)),
 
-which is an epilogue of the product kernels like SwiGLU (two accumulators); and ``weight_on_input``: a picked expert's
+which is an epilogue of the product kernels like SwiGLU (two accumulators); "reglu", a rectified gate, out = W_down
+(max(W_gate h + b, 0) * (W_up h + b')) + b'' with biases where the layer has them (``bias``); and ``weight_on_input``: a picked expert's
 weight multiplies its input, out = sum expert_e(w_e h), not its output (the two first products carry the weight as a
 factor, so the epilogue applies it to both sums in front of the clamps, in float32).
 
@@ -33,39 +34,51 @@ from .. import kernels as K
 from .base import FeedForward, PendingAdd, TensorSource, register_feed_forward
 
 
-ACTIVATIONS = ("swiglu", "relu2", "glu_clamp")
+ACTIVATIONS = ("swiglu", "relu2", "glu_clamp", "reglu")
+GATED = ("swiglu", "glu_clamp", "reglu")   # those with a gate matrix
 # tensor names below a feed-forward's prefix, by role; an architecture with other names passes its own
-DENSE_NAMES = {"gate": "gate_proj.weight", "up": "up_proj.weight", "down": "down_proj.weight"}
+DENSE_NAMES = {"gate": "gate_proj.weight", "up": "up_proj.weight", "down": "down_proj.weight",
+               "gate_bias": "gate_proj.bias", "up_bias": "up_proj.bias", "down_bias": "down_proj.bias"}
 
 
 class DenseMlp(FeedForward):
     """``activation`` "swiglu": down(silu(gate h) * (up h)); "relu2": down(max(up h, 0)^2), no gate matrix; "glu_clamp":
-    the clamped gated unit of the head of the file with its ``limit``."""
+    the clamped gated unit of the head of the file with its ``limit``; "reglu": the rectified gate, with ``bias`` on all three
+    projections."""
 
     can_overwrite = True
 
     def __init__(self, prefix: str, *, hidden: int, intermediate: int, activation: str = "swiglu",
-                 names: Optional[dict] = None, limit: float = 0.0) -> None:
+                 names: Optional[dict] = None, limit: float = 0.0, bias: bool = False) -> None:
         super().__init__(prefix)
         if activation not in ACTIVATIONS:
             raise ValueError(f"dense_mlp: activation {activation!r} (known: {', '.join(ACTIVATIONS)})")
         self.hidden, self.inter, self.activation, self.limit = int(hidden), int(intermediate), activation, float(limit)
         if activation == "glu_clamp" and not self.limit > 0:
             raise ValueError(f"dense_mlp: a clamped gated unit needs a positive limit, got {limit}")
+        if bias and activation != "reglu":
+            raise ValueError(f"dense_mlp: biases go with the rectified gate (reglu), not with {activation}")
+        self.bias = bool(bias)
         self.names = {**DENSE_NAMES, **(names or {})}
 
     def param_shapes(self):
         s = {"w_up": (self.inter, self.hidden), "w_down": (self.hidden, self.inter)}
-        if self.activation in ("swiglu", "glu_clamp"):
+        if self.activation in GATED:
             s["w_gate"] = (self.inter, self.hidden)
+        if self.bias:
+            s.update({"b_in": (2 * self.inter,), "b_down": (self.hidden,)})   # the gate's, behind it the linear part's
         return s
 
     def sources(self):
         p, n = self.prefix, self.names
         out = [TensorSource(f"{p}.{n['up']}", (self.inter, self.hidden), "w_up"),
                TensorSource(f"{p}.{n['down']}", (self.hidden, self.inter), "w_down")]
-        if self.activation in ("swiglu", "glu_clamp"):
+        if self.activation in GATED:
             out.insert(0, TensorSource(f"{p}.{n['gate']}", (self.inter, self.hidden), "w_gate"))
+        if self.bias:
+            out += [TensorSource(f"{p}.{n['gate_bias']}", (self.inter,), "b_in", 0, "bias"),
+                    TensorSource(f"{p}.{n['up_bias']}", (self.inter,), "b_in", self.inter, "bias"),
+                    TensorSource(f"{p}.{n['down_bias']}", (self.hidden,), "b_down", 0, "bias")]
         return out
 
     def kernel_modules(self, dtype):
@@ -82,12 +95,14 @@ class DenseMlp(FeedForward):
             K.linear(h, self.params["w_gate"], act, w2=self.params["w_up"])
         elif self.activation == "glu_clamp":
             K.linear(h, self.params["w_gate"], act, w2=self.params["w_up"], act="glu_clamp", act_limit=self.limit)
+        elif self.activation == "reglu":
+            K.linear(h, self.params["w_gate"], act, w2=self.params["w_up"], act="reglu", bias=self.params.get("b_in"))
         else:
             K.linear(h, self.params["w_up"], act, act="relu2")
         return act
 
     def forward_down(self, act, residual, rt, row_scale=None, accumulate=True) -> None:
-        K.linear(act, self.params["w_down"], residual, accumulate=accumulate, row_scale=row_scale)
+        K.linear(act, self.params["w_down"], residual, bias=self.params.get("b_down"), accumulate=accumulate, row_scale=row_scale)
 
 
 # Up to this many tokens in a step the shared expert's first product starts beside the router instead of behind it
@@ -155,7 +170,7 @@ class SparseMoe(FeedForward):
         self.norm_topk, self.I, self.Is = bool(norm_topk), int(expert_intermediate), int(shared_intermediate)
         self.shared_gate = bool(shared_gate) and self.Is > 0
         self.weight_scale = float(weight_scale)
-        if activation not in ACTIVATIONS:
+        if activation not in ACTIVATIONS or activation == "reglu":
             raise ValueError(f"sparse_moe: activation {activation!r} (known: {', '.join(ACTIVATIONS)})")
         self.activation, self.has_router_bias = activation, bool(router_bias)
         self.names = {**MOE_NAMES, **(names or {})}
@@ -246,6 +261,9 @@ class SparseMoe(FeedForward):
                      row_scale=scale[0] if scale else None, scale_rows=scale[1] if scale else None, **kw)
         else:
             K.linear(x, self.params["up_exps"], act, act="relu2", **kw)
+
+    def leaves_residual_alone(self, residual, rt) -> bool:
+        return self.shared is None and bool(rt.defer_add) and K.rmsnorm_adds(residual)
 
     def forward(self, h, batch, residual, rt, accumulate=True) -> None:
         T = h.shape[0]

@@ -14,7 +14,7 @@ from typing import Optional
 import torch
 
 from .. import kernels as K
-from .base import Norm, PendingAdd, PendingNorm, TensorSource, register_norm
+from .base import Norm, PendingAdd, PendingNorm, PendingRows, TensorSource, register_norm
 
 
 class RMSNorm(Norm):
@@ -42,11 +42,15 @@ class RMSNorm(Norm):
         return ["elementwise"]
 
     def forward(self, x: torch.Tensor, out: torch.Tensor, rows: Optional[torch.Tensor] = None, add=None) -> None:
+        # the experts' sum of the block in front, rows added between two layer calls, or both: folded into the norm's pass
+        extra = {}
+        if isinstance(add, PendingRows) and K.rmsnorm_adds(x) and (add.before is None or isinstance(add.before, PendingAdd)):
+            extra["add_rows"], add = add.y, add.before
         if add is not None and not (isinstance(add, PendingAdd) and K.rmsnorm_adds(x)):
             add.apply(x)
             add = None
         K.rmsnorm(x, self.params["weight"], self.eps, out, rows,
-                  add=None if add is None else (add.pair_out, add.pair_pos, add.top_k))
+                  add=None if add is None else (add.pair_out, add.pair_pos, add.top_k), **extra)
 
     def forward_add(self, y: torch.Tensor, x: torch.Tensor, scale: Optional[torch.Tensor] = None) -> None:
         """x += norm(y): the norm of a sublayer's output (float32 rows) added to the residual stream."""

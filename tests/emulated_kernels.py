@@ -20,11 +20,19 @@ def _f(t: torch.Tensor) -> torch.Tensor:
     return t.to(torch.float64 if PRECISE else torch.float32)
 
 
-def embed_rows(tokens, table, out, copies=1, scale=1.0, dyt_norm=None):
+def embed_rows(tokens, table, out, copies=1, scale=1.0, dyt_norm=None, positions=None, pos_table=None, keep=None):
     rows = _f(table[tokens.long()]) * scale
+    if pos_table is not None:
+        rows = rows + _f(pos_table[positions[: len(tokens)].long()])
     if dyt_norm is not None:
         rows = _dyt(rows, dyt_norm)
     out.copy_(rows.to(out.dtype).repeat(1, copies))
+    if keep is not None:
+        keep.copy_(rows.to(keep.dtype))
+
+
+def add_rows(x, y):
+    x += y.to(x.dtype)
 
 
 def _dyt(z, norm):
@@ -53,12 +61,13 @@ def rmsnorm_adds(x):
     return x.dtype == torch.float32 and x.shape[-1] % 4 == 0
 
 
-def rmsnorm(x, w, eps, out, rows=None, add=None):
-    if add is not None and rows is None:
-        moe_combine(x[: out.shape[0]], add[0], add[1], add[2])
-    elif add is not None:
+def rmsnorm(x, w, eps, out, rows=None, add=None, add_rows=None):
+    if rows is not None and (add is not None or add_rows is not None):
         x = x.clone()
-        moe_combine(x, add[0], add[1], add[2])
+    if add is not None:
+        moe_combine(x if rows is not None else x[: out.shape[0]], add[0], add[1], add[2])
+    if add_rows is not None:
+        x += add_rows.to(x.dtype)
     xs = _f(x if rows is None else x[rows.long()])[: out.shape[0]]
     ss = (xs * xs).sum(-1, keepdim=True)
     out.copy_((xs * (1.0 / torch.sqrt(ss / xs.shape[-1] + eps)) * _f(w)).to(out.dtype))
@@ -71,7 +80,8 @@ class ExpertLayout(K.ExpertLayout):
 def linear(x, w, out, *, w2=None, bias=None, accumulate=False, row_scale=None, scale_rows=None, x_rows=None, lists_ready=False,
            second_tiles=False,
            x_row_div=1, layout=None, n_rows=None, act=None, act_limit=0.0, act_scale=1.0):
-    assert act in (None, "relu2", "glu_clamp", "softcap") and not (act == "relu2" and w2 is not None)
+    assert act in (None, "relu2", "glu_clamp", "softcap", "reglu") and not (act == "relu2" and w2 is not None)
+    assert act != "reglu" or w2 is not None
     assert act != "glu_clamp" or (w2 is not None and act_limit > 0)
     assert act != "softcap" or (w2 is None and act_limit > 0)
     M = out.shape[0] if n_rows is None else n_rows
@@ -82,7 +92,11 @@ def linear(x, w, out, *, w2=None, bias=None, accumulate=False, row_scale=None, s
         rs_all = _f(row_scale[scale_rows[:M].long()] if scale_rows is not None else row_scale[:M])[:, None]
 
     def unit(g, u, rows):
-        """Two products of the same rows into one: SwiGLU, or the clamped gated unit with the rows' scale in front."""
+        """Two products of the same rows into one: SwiGLU, the rectified gate with its two biases, or the clamped gated unit
+        with the rows' scale in front."""
+        if act == "reglu":
+            b, b2 = (_f(bias[: g.shape[1]]), _f(bias[g.shape[1]:])) if bias is not None else (0.0, 0.0)
+            return torch.clamp(g + b, min=0.0) * (u + b2)
         if act != "glu_clamp":
             return g / (1.0 + torch.exp(-g)) * u
         s = rs_all[rows] if rs_all is not None else 1.0
@@ -108,7 +122,7 @@ def linear(x, w, out, *, w2=None, bias=None, accumulate=False, row_scale=None, s
                 if w2 is not None:
                     ye = unit(ye, xin[a:b] @ _f(w2[e]).T, slice(a, b))
                 y[a:b] = ye
-    if bias is not None:
+    if bias is not None and act != "reglu":
         y = y + _f(bias)
     if act == "relu2":
         y = torch.clamp(y, min=0.0) ** 2
@@ -151,7 +165,7 @@ def rope_kv_write(qkv, positions, inv_freq, q_out, pool, slots, *, n_heads, n_kv
         pool[page, 1, :, off, :] = x[t, n_heads + n_kv_heads :].to(pool.dtype)
 
 
-def _attend_one(q, pool, table, p, kvh, page_tokens, window, scale, keep_first=0, sink=False, head=0, chunk=0):
+def _attend_one(q, pool, table, p, kvh, page_tokens, window, scale, keep_first=0, sink=False, head=0, chunk=0, slopes=None):
     lo = max(0, p - window + 1) if window > 0 else (p - p % chunk if chunk > 0 else 0)
     ts = list(range(0, min(keep_first, lo))) + list(range(lo, p + 1))
     pages = [int(table[t // page_tokens]) for t in ts]
@@ -159,6 +173,8 @@ def _attend_one(q, pool, table, p, kvh, page_tokens, window, scale, keep_first=0
     k = torch.stack([_f(pool[pg, 0, kvh, t % page_tokens]) for pg, t in zip(pages, ts)])
     v = torch.stack([_f(pool[pg, 1, kvh, t % page_tokens]) for pg, t in zip(pages, ts)])
     s = (k @ _f(q)) * scale
+    if slopes is not None:
+        s = s - _f(slopes)[head] * (p - torch.tensor(ts, dtype=s.dtype))
     if isinstance(sink, torch.Tensor):     # a learned score per head, as it is
         s = torch.cat([s, _f(sink)[head].view(1)])
         return torch.softmax(s, dim=0)[:-1] @ v
@@ -170,7 +186,7 @@ def _attend_one(q, pool, table, p, kvh, page_tokens, window, scale, keep_first=0
 
 
 def _attn(q, pool, out, seg_list, *, seg_q0, seg_qn, seg_ctx, block_table, n_heads, n_kv_heads, head_dim,
-          page_tokens, window, scale, keep_first=0, sink=False, chunk=0):
+          page_tokens, window, scale, keep_first=0, sink=False, chunk=0, slopes=None):
     group = n_heads // n_kv_heads
     for seg in seg_list:
         q0, qn, ctx = int(seg_q0[seg]), int(seg_qn[seg]), int(seg_ctx[seg])
@@ -178,16 +194,16 @@ def _attn(q, pool, out, seg_list, *, seg_q0, seg_qn, seg_ctx, block_table, n_hea
             for h in range(n_heads):
                 qv = q[q0 + i].view(n_heads, head_dim)[h]
                 o = _attend_one(qv, pool, block_table[seg], ctx + i, h // group, page_tokens, window, scale, keep_first, sink, head=h,
-                                chunk=chunk)
+                                chunk=chunk, slopes=slopes)
                 out[q0 + i].view(n_heads, head_dim)[h] = o.to(out.dtype)
 
 
 def attn_chunk(q, pool, out, *, seg_q0, seg_qn, seg_ctx, block_table, items, n_items, n_heads, n_kv_heads,
-               head_dim, page_tokens, window, scale, keep_first=0, sink=False, chunk=0):
+               head_dim, page_tokens, window, scale, keep_first=0, sink=False, chunk=0, slopes=None):
     segs = sorted({int(items[i, 0]) for i in range(n_items)})
     _attn(q, pool, out, segs, seg_q0=seg_q0, seg_qn=seg_qn, seg_ctx=seg_ctx, block_table=block_table,
           n_heads=n_heads, n_kv_heads=n_kv_heads, head_dim=head_dim, page_tokens=page_tokens, window=window,
-          scale=scale, keep_first=keep_first, sink=sink, chunk=chunk)
+          scale=scale, keep_first=keep_first, sink=sink, chunk=chunk, slopes=slopes)
 
 
 def attn_chunk_mma_splits(n_items, n_heads, max_ctx):
@@ -195,20 +211,22 @@ def attn_chunk_mma_splits(n_items, n_heads, max_ctx):
 
 
 def attn_chunk_mma(q, pool, out, *, seg_q0, seg_qn, seg_ctx, block_table, items, n_items, n_heads, n_kv_heads,
-                   head_dim, page_tokens, window, scale, n_splits=1, part_o=None, part_ml=None, keep_first=0, sink=False, chunk=0):
+                   head_dim, page_tokens, window, scale, n_splits=1, part_o=None, part_ml=None, keep_first=0, sink=False, chunk=0,
+                   slopes=None):
     attn_chunk(q, pool, out, seg_q0=seg_q0, seg_qn=seg_qn, seg_ctx=seg_ctx, block_table=block_table, items=items,
                n_items=n_items, n_heads=n_heads, n_kv_heads=n_kv_heads, head_dim=head_dim, page_tokens=page_tokens,
-               window=window, scale=scale, keep_first=keep_first, sink=sink, chunk=chunk)
+               window=window, scale=scale, keep_first=keep_first, sink=sink, chunk=chunk, slopes=slopes)
 
 
 def attn_decode(q, pool, out, *, seg_q0, seg_qn, seg_ctx, block_table, items, n_items, n_heads, n_kv_heads,
-                head_dim, page_tokens, window, scale, part_o, part_ml, counters, max_splits, keep_first=0, sink=False, chunk=0):
+                head_dim, page_tokens, window, scale, part_o, part_ml, counters, max_splits, keep_first=0, sink=False, chunk=0,
+                slopes=None):
     segs = [int(items[i]) for i in range(n_items)]
     for s in segs:
         assert int(seg_ctx[s]) // K.DECODE_SPLIT + 1 <= max_splits
     _attn(q, pool, out, segs, seg_q0=seg_q0, seg_qn=seg_qn, seg_ctx=seg_ctx, block_table=block_table,
           n_heads=n_heads, n_kv_heads=n_kv_heads, head_dim=head_dim, page_tokens=page_tokens, window=window,
-          scale=scale, keep_first=keep_first, sink=sink, chunk=chunk)
+          scale=scale, keep_first=keep_first, sink=sink, chunk=chunk, slopes=slopes)
 
 
 def _select(logits_row, top_k, renorm, scale, score_fn, sel_bias, n_group, n_group_used, group_score="top2"):
@@ -240,7 +258,7 @@ def _select(logits_row, top_k, renorm, scale, score_fn, sel_bias, n_group, n_gro
     for _ in range(top_k):
         best = max((x for x in range(E) if x not in picked), key=lambda x: (float(sel[x]), -x))
         picked.append(best)
-    wsum = sum(p[x] for x in picked) if renorm else 1.0
+    wsum = sum(p[x] for x in picked) + (1e-20 if score_fn == "sigmoid" else 0.0) if renorm else 1.0
     return picked, [float(p[x] / wsum * scale) for x in picked]
 
 
@@ -643,7 +661,7 @@ def mlstm_out(o_raw, m_t, proj, off_g, w, eps, out, *, n_heads, v_dim):
 def head_prep(proj, *, offsets, heads, dims, laid, state_slots, seg_q0, seg_qn, n_seg, longest_new, positions, q_out,
               k_out=None, v_out=None, pool=None, slots=None, page_tokens=0, write_kv=True, conv=None, state=None,
               conv_offset=0, move_state=True, act=False, inv_freq=None, rot=0, norm=None, eps=0.0, q_scale=1.0, gates=None,
-              interleaved=False, norm_weights=None, n_rows=0):
+              interleaved=False, norm_weights=None, n_rows=0, q_temp=None):
     widths = [h * d for h, d in zip(heads, dims)]
     C = sum(widths)
     taps = conv.shape[1] if conv is not None else 1
@@ -691,6 +709,9 @@ def head_prep(proj, *, offsets, heads, dims, laid, state_slots, seg_q0, seg_qn, 
                 x = x / torch.sqrt((x * x).sum(-1, keepdim=True) + eps)
             if which == 0:
                 x = x * q_scale
+                if q_temp is not None:
+                    turns = torch.floor((positions[rows].double() + 1.0) / q_temp[1]) + 1.0
+                    x = x * (1.0 + q_temp[0] * torch.log(_f(turns)))[:, None, None]
             padded = x.new_zeros(qn, H, L)
             padded[..., :d] = x
             if which == 0:
@@ -778,7 +799,7 @@ def head_tile(n_tokens, dtype, widths_ok):
 
 
 _NAMES = ["embed_rows", "rmsnorm", "rmsnorm_adds", "attn_chunk_tc_takes", "linear", "rope_kv_write", "attn_chunk", "attn_chunk_mma", "attn_decode", "router_topk", "router_logits", "router_select",
-          "moe_sort", "route_small", "route_small_takes", "route_fused_small", "moe_combine", "gather_rows", "apply_penalties", "sample",
+          "moe_sort", "route_small", "route_small_takes", "route_fused_small", "moe_combine", "gather_rows", "add_rows", "apply_penalties", "sample",
           "cast_rows", "rmsnorm_add", "latent_prep", "latent_q_split", "latent_attn", "heads_to_rows", "retention_scan",
           "retention_gate_norm", "head_tile", "latent_attn_mma_takes", "layernorm", "stream_update", "moe_identity",
           "gated_recurrence", "mlstm_gates", "mlstm_out", "ssm_conv", "ssm_out", "head_prep", "gate_rows", "delta_rule", "delta_out",
