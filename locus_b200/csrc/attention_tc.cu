@@ -22,6 +22,10 @@
 // warps 2-9: softmax and output, two threads per query row (64 keys and 64 output dimensions each).  Head size 128 only (other sizes and pages that are not a multiple
 // of 64 tokens go to the mma.sync kernel).
 //
+// Keys and values may also lie in plain rows instead of pages (rows form): two matrices [rows][kv heads * 128] in which a
+// segment's keys are consecutive rows from kv_row0[segment] on (latent attention expands its heads' keys and values of a
+// long portion's context that way); only the coordinates of the loads differ.
+//
 // Every wait on an mbarrier is bounded; when one runs out the kernel sets the module's error word,
 // and every later wait of every role returns at once, so the kernel ends quickly instead of hanging.
 #include <cuda.h>
@@ -48,6 +52,7 @@ struct TcAttnArgs {
     const int* seg_ctx;
     const int* block_table;
     int table_stride;
+    const int* kv_row0;     // rows form: a segment's first row of K and V (block_table unused); null: pages
     const int* items;
     int nh, nkv, page_tokens, window, chunk;  // (mask.cuh)
     const float* sink_val;  // with sink: a learned score per query head in its place (null: the score 0)
@@ -228,7 +233,8 @@ __device__ __forceinline__ void at_st32(uint32_t taddr, const uint32_t* v) {
 // BIAS: a distance bias; an instance of its own (the softmax warps are bound by instruction issue).
 template <bool BIAS>
 __global__ void __launch_bounds__(320, 1)
-attn_chunk_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv, TcAttnArgs a) {
+attn_chunk_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
+                     const __grid_constant__ CUtensorMap map_v, TcAttnArgs a) {
     extern __shared__ __align__(1024) uint8_t at_raw[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     // the late tiles of a prompt see the most keys: the grid takes them first, for all heads (the heads are the
@@ -255,7 +261,7 @@ attn_chunk_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
         const int jj = j0 + j;
         return jj < n_keep ? jj * AT_MK : first_tile + (jj - n_keep) * AT_MK;
     };
-    const int* table = a.block_table + static_cast<size_t>(seg) * a.table_stride;
+    const int* table = a.kv_row0 ? nullptr : a.block_table + static_cast<size_t>(seg) * a.table_stride;
 
     // shared memory: Q, K[2], V[2], P[2] (each a tile of two swizzled halves), then the barriers.  That is
     // all the shared memory a block can have, so the tiles start at the very base, which must be
@@ -304,6 +310,9 @@ attn_chunk_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
             at_tma_2d(sQ, &map_q, h * AT_HD, row0, q_full);
             at_tma_2d(sQ + AT_HALF_BYTES, &map_q, h * AT_HD + 64, row0, q_full);
             const long long rows_per_page = 2LL * a.nkv * P;
+            const int v_shift = a.kv_row0 ? 0 : a.nkv * P;  // V rows of a page lie nkv * P rows behind its K rows
+            const int col0 = a.kv_row0 ? kvh * AT_HD : 0;
+            const int rows0 = a.kv_row0 ? a.kv_row0[seg] : 0;
             for (int j = 0; j < n_tiles; ++j) {
                 const int b = j & 1;
                 const uint32_t par = ((j >> 1) & 1) ^ 1;
@@ -313,22 +322,25 @@ attn_chunk_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
                 int krow[2];
                 for (int hh = 0; hh < 2; ++hh) {
                     const int t = tile0 + 64 * hh;
-                    int page = -1;
-                    if (t <= t_hi && (t + 63 >= t_lo || t < keep)) page = table[t / P];
-                    krow[hh] = page < 0 ? -64 : static_cast<int>(page * rows_per_page + static_cast<long long>(kvh) * P + t % P);
+                    const bool seen = t <= t_hi && (t + 63 >= t_lo || t < keep);
+                    if (a.kv_row0) {
+                        krow[hh] = seen ? rows0 + t : -64;
+                    } else {
+                        const int page = seen ? table[t / P] : -1;
+                        krow[hh] = page < 0 ? -64 : static_cast<int>(page * rows_per_page + static_cast<long long>(kvh) * P + t % P);
+                    }
                 }
-                const int v_shift = a.nkv * P;  // V rows of a page lie nkv * P rows behind its K rows
                 if (!at_wait(k_free + 8 * b, par, 1)) break;
                 at_expect_tx(k_full + 8 * b, AT_TILE_BYTES);
                 for (int hh = 0; hh < 2; ++hh)
                     for (int ch = 0; ch < 2; ++ch)
-                        at_tma_2d(sK + b * AT_TILE_BYTES + ch * AT_HALF_BYTES + hh * (64 * 128), &map_kv, 64 * ch, krow[hh],
+                        at_tma_2d(sK + b * AT_TILE_BYTES + ch * AT_HALF_BYTES + hh * (64 * 128), &map_k, col0 + 64 * ch, krow[hh],
                                   k_full + 8 * b);
                 if (!at_wait(v_free + 8 * b, par, 2)) break;
                 at_expect_tx(v_full + 8 * b, AT_TILE_BYTES);
                 for (int hh = 0; hh < 2; ++hh)
                     for (int ch = 0; ch < 2; ++ch)
-                        at_tma_2d(sV + b * AT_TILE_BYTES + ch * AT_HALF_BYTES + hh * (64 * 128), &map_kv, 64 * ch,
+                        at_tma_2d(sV + b * AT_TILE_BYTES + ch * AT_HALF_BYTES + hh * (64 * 128), &map_v, col0 + 64 * ch,
                                   krow[hh] < 0 ? -64 : krow[hh] + v_shift, v_full + 8 * b);
             }
         }
@@ -652,6 +664,33 @@ static bool at_make_map(CUtensorMap* map, const void* ptr, long long rows, long 
               CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
+// The launch shared by the entry points below: `a` carries everything but the scratch of the ranges.
+static int at_launch(const CUtensorMap& map_q, const CUtensorMap& map_k, const CUtensorMap& map_v, TcAttnArgs a, int n_items,
+                     int n_splits, float* part_o, float* part_ml, cudaStream_t stream) {
+    if (n_items > 65535) return LOCUS_ERR_UNSUPPORTED;
+    a.n_splits = n_splits; a.part_o = part_o; a.part_ml = part_ml;
+    const size_t smem = 7 * AT_TILE_BYTES + 160 + 2 * 2 * 128 * 4;
+    static bool set = false;
+    if (!set) {
+        if (cudaFuncSetAttribute(attn_chunk_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess ||
+            cudaFuncSetAttribute(attn_chunk_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+            return static_cast<int>(cudaGetLastError());
+        set = true;
+    }
+    dim3 grid(a.nh, n_items, n_splits);
+    if (a.slopes != nullptr) attn_chunk_tc_kernel<true><<<grid, 320, smem, stream>>>(map_q, map_k, map_v, a);
+    else attn_chunk_tc_kernel<false><<<grid, 320, smem, stream>>>(map_q, map_k, map_v, a);
+    if (n_splits > 1)
+        attn_chunk_tc_merge_kernel<<<dim3(AT_MQ * (AT_HD / 4) / 128, n_items, a.nh), 128, 0, stream>>>(a);
+    return locus_launch_status();
+}
+
+static bool at_scratch_ok(int n_splits, const float* part_o, const float* part_ml) {
+    return n_splits >= 1 && n_splits <= AT_MAX_SPLITS &&
+           (n_splits == 1 || (part_o != nullptr && part_ml != nullptr &&
+                              ((reinterpret_cast<uintptr_t>(part_o) | reinterpret_cast<uintptr_t>(part_ml)) & 15) == 0));
+}
+
 // q, out [T, nh * 128] bfloat16; pool: one layer's pages [n_pages][2][nkv][page_tokens][128] bfloat16;
 // items: [n_items, 2] = (segment, first query of a 64-query tile), a segment's tiles in ascending order.
 // Head size 128 and pages of a multiple of 64 tokens only (LOCUS_ERR_UNSUPPORTED otherwise).
@@ -664,10 +703,7 @@ extern "C" int locus_attn_chunk_tc(const void* q, long long T, const void* pool,
                                    float* part_ml, int keep_first, int sink, const float* sink_val,
                                    const float* slopes, cudaStream_t stream) {
     if (n_items <= 0) return 0;
-    if (n_splits < 1 || n_splits > AT_MAX_SPLITS) return LOCUS_ERR_UNSUPPORTED;
-    if (n_splits > 1 && (part_o == nullptr || part_ml == nullptr ||
-                         ((reinterpret_cast<uintptr_t>(part_o) | reinterpret_cast<uintptr_t>(part_ml)) & 15)))
-        return LOCUS_ERR_UNSUPPORTED;
+    if (!at_scratch_ok(n_splits, part_o, part_ml)) return LOCUS_ERR_UNSUPPORTED;
     if (hd != AT_HD || page_tokens <= 0 || page_tokens % 64 != 0 || !mask_ok(window, chunk, keep_first)) return LOCUS_ERR_UNSUPPORTED;
     if (nh <= 0 || nkv <= 0 || nh % nkv != 0 || nh > 65535) return LOCUS_ERR_UNSUPPORTED;
     const long long pool_rows = n_pages * 2 * nkv * page_tokens;
@@ -680,25 +716,40 @@ extern "C" int locus_attn_chunk_tc(const void* q, long long T, const void* pool,
     if (!at_make_map(&map_kv, pool, pool_rows, hd, hd, 64)) return LOCUS_ERR_UNSUPPORTED;
     TcAttnArgs a;
     a.out = static_cast<bf16*>(out); a.seg_q0 = seg_q0; a.seg_qn = seg_qn; a.seg_ctx = seg_ctx;
-    a.block_table = block_table; a.table_stride = table_stride; a.items = items; a.nh = nh; a.nkv = nkv;
+    a.block_table = block_table; a.table_stride = table_stride; a.kv_row0 = nullptr; a.items = items; a.nh = nh; a.nkv = nkv;
     a.page_tokens = page_tokens; a.window = window; a.chunk = chunk; a.scale = scale;
     a.keep_first = window > 0 ? keep_first : 0; a.sink = sink ? 1 : 0; a.sink_val = sink ? sink_val : nullptr;
-    a.n_splits = n_splits; a.part_o = part_o; a.part_ml = part_ml; a.slopes = slopes;
-    const size_t smem = 7 * AT_TILE_BYTES + 160 + 2 * 2 * 128 * 4;
-    static bool set = false;
-    if (!set) {
-        if (cudaFuncSetAttribute(attn_chunk_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess ||
-            cudaFuncSetAttribute(attn_chunk_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
-            return static_cast<int>(cudaGetLastError());
-        set = true;
-    }
-    if (n_items > 65535) return LOCUS_ERR_UNSUPPORTED;
-    dim3 grid(nh, n_items, n_splits);
-    if (slopes != nullptr) attn_chunk_tc_kernel<true><<<grid, 320, smem, stream>>>(map_q, map_kv, a);
-    else attn_chunk_tc_kernel<false><<<grid, 320, smem, stream>>>(map_q, map_kv, a);
-    if (n_splits > 1)
-        attn_chunk_tc_merge_kernel<<<dim3(AT_MQ * (AT_HD / 4) / 128, n_items, nh), 128, 0, stream>>>(a);
-    return locus_launch_status();
+    a.slopes = slopes;
+    return at_launch(map_q, map_kv, map_kv, a, n_items, n_splits, part_o, part_ml, stream);
+}
+
+// The rows form: k and v [rows, >= nkv * 128] bfloat16 with row strides ldk, ldv (elements, multiples of 8, 16-byte aligned
+// bases); segment s's key at position t is row kv_row0[s] + t of both.  Otherwise as above.
+extern "C" int locus_attn_chunk_tc_rows(const void* q, long long T, const void* k, long long ldk, const void* v, long long ldv,
+                                        long long rows, void* out, const int* seg_q0, const int* seg_qn, const int* seg_ctx,
+                                        const int* kv_row0, const int* items, int n_items, int nh, int nkv, int hd, int window,
+                                        int chunk, float scale, int n_splits, float* part_o, float* part_ml, int keep_first,
+                                        int sink, const float* sink_val, const float* slopes, cudaStream_t stream) {
+    if (n_items <= 0) return 0;
+    if (!at_scratch_ok(n_splits, part_o, part_ml)) return LOCUS_ERR_UNSUPPORTED;
+    if (hd != AT_HD || kv_row0 == nullptr || !mask_ok(window, chunk, keep_first)) return LOCUS_ERR_UNSUPPORTED;
+    if (nh <= 0 || nkv <= 0 || nh % nkv != 0 || nh > 65535) return LOCUS_ERR_UNSUPPORTED;
+    if (T <= 0 || T >= (1LL << 31) || rows <= 0 || rows >= (1LL << 31)) return LOCUS_ERR_UNSUPPORTED;
+    const long long cols = static_cast<long long>(nkv) * hd;
+    if (ldk < cols || ldv < cols || ldk % 8 != 0 || ldv % 8 != 0) return LOCUS_ERR_UNSUPPORTED;
+    if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v) | reinterpret_cast<uintptr_t>(out)) & 15)
+        return LOCUS_ERR_UNSUPPORTED;
+    CUtensorMap map_q, map_k, map_v;
+    if (!at_make_map(&map_q, q, T, static_cast<long long>(nh) * hd, static_cast<long long>(nh) * hd, AT_MQ) ||
+        !at_make_map(&map_k, k, rows, cols, ldk, 64) || !at_make_map(&map_v, v, rows, cols, ldv, 64))
+        return LOCUS_ERR_UNSUPPORTED;
+    TcAttnArgs a;
+    a.out = static_cast<bf16*>(out); a.seg_q0 = seg_q0; a.seg_qn = seg_qn; a.seg_ctx = seg_ctx;
+    a.block_table = nullptr; a.table_stride = 0; a.kv_row0 = kv_row0; a.items = items; a.nh = nh; a.nkv = nkv;
+    a.page_tokens = 64; a.window = window; a.chunk = chunk; a.scale = scale;
+    a.keep_first = window > 0 ? keep_first : 0; a.sink = sink ? 1 : 0; a.sink_val = sink ? sink_val : nullptr;
+    a.slopes = slopes;
+    return at_launch(map_q, map_k, map_v, a, n_items, n_splits, part_o, part_ml, stream);
 }
 
 // Reads and clears the module's error word (0 = no bounded wait ran out).  Synchronises.

@@ -22,6 +22,7 @@
 //                   sees p - window < j <= p; 0 = all), and a sink per head: exp(sink[h]) joins the softmax's
 //                   denominator, without a key or a value
 //   heads_to_rows   [head][token][d] -> [token][head * d]
+//   latent_gather   cached rows of some requests as plain rows, for portions whose heads' keys and values are expanded
 //
 // Angles: position * frequency and its sine and cosine are formed in float64 from float64 frequencies (the
 // host computes them, ramp of a long-context scaling included) and rounded once; `magnitude` multiplies both.
@@ -213,6 +214,47 @@ extern "C" int locus_heads_to_rows(const void* src, int dt, void* out, int T, in
 }
 
 // ---------------------------------------------------------------------------
+// The cached rows of some segments as plain rows: out[row0[seg] + t, :] = the first `width` elements of the segment's cache row
+// of position t, t < seg_ctx + seg_qn.  A warp per row, 16-byte pieces; grid.y: the listed segments.
+template <typename TA>
+__global__ void __launch_bounds__(256) latent_gather_kernel(const TA* __restrict__ pool, TA* __restrict__ out, const int* __restrict__ segs,
+                                                            const int* __restrict__ row0, const int* __restrict__ seg_qn,
+                                                            const int* __restrict__ seg_ctx, const int* __restrict__ block_table,
+                                                            int table_stride, int page_tokens, int row_width, int width) {
+    pdl_entry();
+    pdl_trigger();
+    const int seg = segs[blockIdx.y];
+    const int t = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (t >= seg_ctx[seg] + seg_qn[seg]) return;
+    const int page = block_table[static_cast<size_t>(seg) * table_stride + t / page_tokens];
+    const size_t slot = static_cast<size_t>(max(page, 0)) * page_tokens + t % page_tokens;
+    const uint4* src = reinterpret_cast<const uint4*>(pool + slot * row_width);
+    uint4* dst = reinterpret_cast<uint4*>(out + static_cast<size_t>(row0[seg] + t) * width);
+    const int pieces = width * static_cast<int>(sizeof(TA)) / 16;
+    // (a page behind a window that has gone back: zeros, which no query sees)
+    for (int i = lane; i < pieces; i += 32) dst[i] = page >= 0 ? src[i] : make_uint4(0, 0, 0, 0);
+}
+
+// longest: the most positions (cached and new) of a listed segment.  Rows of whole 16-byte pieces, aligned bases.
+extern "C" int locus_latent_gather(const void* pool, int dt, void* out, const int* segs, int n_segs, const int* row0,
+                                   const int* seg_qn, const int* seg_ctx, const int* block_table, int table_stride, int page_tokens,
+                                   int row_width, int width, int longest, cudaStream_t stream) {
+    if (n_segs <= 0 || longest <= 0) return 0;
+    const int el = dt == LOCUS_DT_F32 ? 4 : 2;
+    if ((dt != LOCUS_DT_F32 && dt != LOCUS_DT_BF16) || n_segs > 65535 || page_tokens <= 0 || width <= 0 || width > row_width ||
+        width * el % 16 || row_width * el % 16 || ((reinterpret_cast<uintptr_t>(pool) | reinterpret_cast<uintptr_t>(out)) & 15))
+        return LOCUS_ERR_UNSUPPORTED;
+    const dim3 grid((longest + 7) / 8, n_segs);
+    if (dt == LOCUS_DT_BF16)
+        locus_launch(latent_gather_kernel<bf16>, grid, dim3(256), 0, stream, static_cast<const bf16*>(pool), static_cast<bf16*>(out), segs, row0,
+                     seg_qn, seg_ctx, block_table, table_stride, page_tokens, row_width, width);
+    else
+        locus_launch(latent_gather_kernel<float>, grid, dim3(256), 0, stream, static_cast<const float*>(pool), static_cast<float*>(out), segs,
+                     row0, seg_qn, seg_ctx, block_table, table_stride, page_tokens, row_width, width);
+    return locus_launch_status();
+}
+
+// ---------------------------------------------------------------------------
 // Attention over the latent rows on the CUDA cores, float32 arithmetic throughout.
 struct LatentArgs {
     const void* q_abs;       // [H, T, kv_rank] head-major: the unrotated queries carried into the latent space
@@ -399,7 +441,7 @@ extern "C" int locus_latent_attn(const void* q_abs, const void* q_rot, int dt, c
 // dh of the latent's dimensions for O += P C.  Scores go through shared memory once per tile so that both warps
 // of a row group see the whole tile's 32 keys: each forms the rows' running maximum and denominator itself (the
 // same numbers) and multiplies its P, rounded to bfloat16, with its half of the rows' latents.  Key tiles of 32
-// rows arrive by cp.async, two buffers.  kv_rank is a template parameter (32 to 512); rot_dim a multiple of 16.
+// rows arrive by cp.async, two buffers.  kv_rank is a template parameter (multiples of 32, from 256 on of 64, up to 512); rot_dim a multiple of 16.
 #define LM_ROWS 64
 #define LM_KEYS 32
 
@@ -725,7 +767,7 @@ static int launch_latent_mma(const LatentMmaArgs& a, int n_items, size_t smem, c
     return locus_launch_status();
 }
 
-// bfloat16; kv_rank 32, 64, 128, 256 or 512; rot_dim a multiple of 16 (0 allowed); a block's 64 rows are
+// bfloat16; kv_rank a multiple of 32 up to 256 or of 64 up to 512; rot_dim a multiple of 16 (0 allowed); a block's 64 rows are
 // (64 >> hb_shift) queries x (1 << hb_shift) heads, and items lists tiles of 64 >> hb_shift queries.  n_splits > 1
 // (up to 16): the key tiles of every block are cut into that many ranges; part_o holds n_items * head blocks *
 // n_splits * 64 * kv_rank floats and part_ml n_items * head blocks * n_splits * 128.
@@ -754,8 +796,15 @@ extern "C" int locus_latent_attn_mma(const void* q_abs, const void* q_rot, const
     switch (kv_rank) {
         case 32: return launch_latent_mma<32>(a, n_items, smem, stream);
         case 64: return launch_latent_mma<64>(a, n_items, smem, stream);
+        case 96: return launch_latent_mma<96>(a, n_items, smem, stream);
         case 128: return launch_latent_mma<128>(a, n_items, smem, stream);
+        case 160: return launch_latent_mma<160>(a, n_items, smem, stream);
+        case 192: return launch_latent_mma<192>(a, n_items, smem, stream);
+        case 224: return launch_latent_mma<224>(a, n_items, smem, stream);
         case 256: return launch_latent_mma<256>(a, n_items, smem, stream);
+        case 320: return launch_latent_mma<320>(a, n_items, smem, stream);
+        case 384: return launch_latent_mma<384>(a, n_items, smem, stream);
+        case 448: return launch_latent_mma<448>(a, n_items, smem, stream);
         case 512: return launch_latent_mma<512>(a, n_items, smem, stream);
     }
     return LOCUS_ERR_UNSUPPORTED;

@@ -807,17 +807,20 @@ TC_ATTN_MAX_SPLITS = 16
 TC_ATTN_QUERY_BLOCK = 128   # queries of a block of the tcgen05 kernel (two of the 64-query tiles of its item list)
 
 
-def attn_chunk_tc_splits(n_items: int, n_heads: int, max_ctx: int) -> int:
+def attn_chunk_tc_splits(n_items: int, n_heads: int, max_ctx: int, n_rows: int = 0) -> int:
     """Ranges the key tiles of every block of :func:`attn_chunk_tc` are cut into.  A block takes 128 queries of one
     head, a block per SM: a portion of a few hundred tokens behind a long context makes fewer blocks than the GPU
     has SMs, each walking thousands of keys alone.  Then the keys are cut so that about every SM has a block, down
-    to four tiles of 128 keys per range (a block's start and end cost about four tiles' time)."""
+    to four tiles of 128 keys per range (a block's start and end cost about four tiles' time).  ``n_rows``: the step's tokens,
+    those of other kernels' segments among them: a range keeps a partial result for each, and they must fit
+    :func:`attn_chunk_tc_scratch`."""
     blocks = -(-n_items // 2) * n_heads
     n_sm = _sm_count()
     tiles = -(-max_ctx // TC_ATTN_QUERY_BLOCK)
     if 2 * blocks > n_sm or tiles < 8:
         return 1
-    return max(1, min(TC_ATTN_MAX_SPLITS, n_sm // blocks, tiles // 4))
+    fit = TC_ATTN_QUERY_BLOCK * n_sm // max(1, n_rows * n_heads) if n_rows > 0 else TC_ATTN_MAX_SPLITS
+    return max(1, min(TC_ATTN_MAX_SPLITS, n_sm // blocks, tiles // 4, fit))
 
 
 def attn_chunk_tc_scratch() -> Tuple[int, int]:
@@ -864,6 +867,39 @@ def attn_chunk_tc(q: torch.Tensor, pool: torch.Tensor, out: torch.Tensor, *, seg
         _count_launches(1)
     _check(code, "attn_chunk_tc", f"(heads {n_heads}/{n_kv_heads}, head_dim {head_dim}, pages of {page_tokens}, "
                                   f"{n_splits} key ranges)")
+
+
+def attn_chunk_tc_rows(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, out: torch.Tensor, *, seg_q0: torch.Tensor,
+                       seg_qn: torch.Tensor, seg_ctx: torch.Tensor, kv_row0: torch.Tensor, items: torch.Tensor, n_items: int,
+                       n_heads: int, n_kv_heads: int, head_dim: int, window: int, scale: float, n_splits: int = 1,
+                       part_o: Optional[torch.Tensor] = None, part_ml: Optional[torch.Tensor] = None, keep_first: int = 0,
+                       sink=False, chunk: int = 0, slopes: Optional[torch.Tensor] = None) -> None:
+    """:func:`attn_chunk_tc` over keys and values in plain rows instead of pages: ``k`` and ``v`` [rows, n_kv_heads *
+    head_dim] (stretches of columns of wider rows are taken), a segment's key at position t in row ``kv_row0[segment]`` + t
+    of both.  ``items`` lists tiles of 64 queries of the segments that have such rows; the others' entries of ``kv_row0`` are
+    not read."""
+    _cuda_c(q, "q")
+    _cuda_c(out, "out")
+    _i32(items, "items")
+    _i32(kv_row0, "kv_row0")
+    _need(q.dtype == k.dtype == v.dtype == out.dtype == torch.bfloat16, "attn_chunk_tc_rows: bfloat16 only")
+    for t in (k, v):
+        _need(t.is_cuda and t.stride(1) == 1 and t.shape[0] == k.shape[0] and t.shape[1] == n_kv_heads * head_dim,
+              "attn_chunk_tc_rows: k, v rows [rows, n_kv_heads * head_dim]")
+    _need(1 <= n_splits <= TC_ATTN_MAX_SPLITS, f"attn_chunk_tc_rows: 1 to {TC_ATTN_MAX_SPLITS} key ranges")
+    if n_splits > 1:
+        units = q.shape[0] * n_heads * n_splits
+        _need(part_o is not None and part_ml is not None and part_o.dtype == part_ml.dtype == torch.float32
+              and part_o.is_cuda and part_ml.is_cuda and part_o.numel() >= units * TC_ATTN_HEAD_DIM and part_ml.numel() >= units * 2,
+              "attn_chunk_tc_rows: scratch too small for these ranges")
+    code = _lib("attention_tc").locus_attn_chunk_tc_rows(
+        _p(q), LL(q.shape[0]), _p(k), LL(k.stride(0)), _p(v), LL(v.stride(0)), LL(k.shape[0]), _p(out), _p(seg_q0), _p(seg_qn),
+        _p(seg_ctx), _p(kv_row0), _p(items), I(n_items), I(n_heads), I(n_kv_heads), I(head_dim), I(window), I(chunk), F(scale),
+        I(n_splits), _p(part_o if n_splits > 1 else None), _p(part_ml if n_splits > 1 else None),
+        I(keep_first if window > 0 else 0), *_sink_args(sink, n_heads), _slopes_arg(slopes, n_heads), _stream())
+    if n_splits > 1 and code == 0:
+        _count_launches(1)
+    _check(code, "attn_chunk_tc", f"(rows; heads {n_heads}/{n_kv_heads}, head_dim {head_dim}, {n_splits} key ranges)")
 
 
 def attn_tc_error() -> int:
@@ -1383,11 +1419,44 @@ def latent_attn(q_abs_hm: torch.Tensor, q_rot: torch.Tensor, pool: torch.Tensor,
     _check(code, "latent_attn", f"(heads {n_heads}, latent {kv_rank} + {rot_dim})")
 
 
-LATENT_MMA_RANKS = (32, 64, 128, 256, 512)
+# Long portions: the heads' keys and values of a segment's whole context are expanded into plain rows and the portion runs on
+# the tcgen05 attention kernel.  A query-key pair then costs 2 x (key + value size) multiply-adds a head instead of 2 x 2 x rank
+# on the mma.sync kernel (sizes of 128 on a latent of 512: a quarter, on the faster pipe); the expansion costs as much as that
+# of two products per context row and is shared by the portion's queries.
+LATENT_EXPAND_FROM = 128         # new tokens of a segment from which on it is expanded
+LATENT_EXPAND_ROWS = 16384       # most context rows of a step that are expanded ...
+LATENT_EXPAND_BYTES = 512 << 20  # ... and most bytes of their keys and values; segments beyond run over the latents
+
+
+def latent_expand_rows(dtype: torch.dtype, n_heads: int, nope_dim: int, rot_dim: int, v_dim: int, kv_rank: int) -> int:
+    """Context rows of a step that may be expanded for the tcgen05 attention kernel; 0 where it does not take this mixer's sizes
+    (bfloat16, keys without a rotated part and values of the kernel's head size)."""
+    if not (USE_TENSOR_CORES and dtype == torch.bfloat16 and nope_dim == v_dim == TC_ATTN_HEAD_DIM and rot_dim == 0 and kv_rank % 8 == 0):
+        return 0
+    return min(LATENT_EXPAND_ROWS, LATENT_EXPAND_BYTES // (2 * n_heads * (nope_dim + v_dim)))
+
+
+def latent_gather(pool: torch.Tensor, out: torch.Tensor, *, segs: torch.Tensor, n_segs: int, row0: torch.Tensor,
+                  seg_qn: torch.Tensor, seg_ctx: torch.Tensor, block_table: torch.Tensor, page_tokens: int, longest: int) -> None:
+    """out[row0[s] + t, :] = the leading elements of segment s's cache row of position t, for the ``n_segs`` segments that
+    ``segs`` lists and all their positions (cached and new); ``longest``: the most positions of one of them."""
+    _cuda_c(pool, "pool")
+    _cuda_c(out, "out")
+    for t, name in ((segs, "segs"), (row0, "row0"), (block_table, "block_table")):
+        _i32(t, name)
+    _need(pool.dtype == out.dtype and pool.shape[-2] == page_tokens and out.shape[1] <= pool.shape[-1] and pool.shape[1] == pool.shape[2] == 1,
+          "latent_gather: rows of the pool's element type, at most as wide")
+    code = _lib("latent_attention").locus_latent_gather(
+        _p(pool), I(dtype_code(pool.dtype)), _p(out), _p(segs), I(n_segs), _p(row0), _p(seg_qn), _p(seg_ctx), _p(block_table),
+        I(block_table.shape[1]), I(page_tokens), I(pool.shape[-1]), I(out.shape[1]), I(longest), _stream())
+    _check(code, "latent_gather", f"(rows of {out.shape[1]} of {pool.shape[-1]})")
+
+
+LATENT_MMA_RANKS = (32, 64, 96, 128, 160, 192, 224, 256, 320, 384, 448, 512)
 
 
 def latent_attn_mma_takes(dtype: torch.dtype, kv_rank: int, rot_dim: int) -> bool:
-    """Whether :func:`latent_attn_mma` takes this case: bfloat16, a latent of 32, 64, 128, 256 or 512 elements and a
+    """Whether :func:`latent_attn_mma` takes this case: bfloat16, a latent whose size is a multiple of 32 up to 256 or of 64 up to 512, and a
     rotated part that is a multiple of 16 (or none); everything else runs on :func:`latent_attn`."""
     return (USE_TENSOR_CORES and dtype == torch.bfloat16 and kv_rank in LATENT_MMA_RANKS and rot_dim % 16 == 0)
 

@@ -404,7 +404,7 @@ class Attention(Mixer):
             if self.window > 0 or self.chunk > 0:
                 keys = min(keys, (self.window or self.chunk) + self.keep_first + K.TC_ATTN_QUERY_BLOCK)
             if K.attn_chunk_tc_takes(q, self.head_dim, gb.page_tokens, T, keys):
-                n_splits = K.attn_chunk_tc_splits(tiles["n_chunk_items64"], self.n_heads, keys)
+                n_splits = K.attn_chunk_tc_splits(tiles["n_chunk_items64"], self.n_heads, keys, T)
                 part_o = part_ml = None
                 if n_splits > 1:
                     n_o, n_ml = K.attn_chunk_tc_scratch()

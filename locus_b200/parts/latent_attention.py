@@ -21,6 +21,10 @@ cache rows of the layer call that the run order names (that layer's latent and r
 W_uk, W_uv and queries.  The rotated parts' pairs are interleaved, (2i, 2i + 1), or the halves (i, i + dims/2), as the
 position encoding says.
 
+Long portions (kernels.LATENT_EXPAND_FROM tokens of a request on) of sizes that the tcgen05 attention kernel takes go the
+other way: the cached latents of the request's context are gathered into plain rows, expanded into every head's keys and
+values by one product with [W_uk; W_uv], and attended to by that kernel.  The pages hold latents either way.
+
 The softmax's denominator may hold a learned sink per head, exp(sink_h), without a key or a value.  A query at
 position p sees the keys j with p - window < j <= p (window 0: all).  Scores, softmax, the norms' statistics,
 positions and angles are float32 (angles are formed in float64 and rounded once).
@@ -58,6 +62,52 @@ class LatentTiles(StepPlan):
             raise ValueError("latent attention: the step has more query tiles than the plan's capacity holds")
         self._lib.locus_sort_tiles_by_position(n, out.ctypes.data, seg_ctx.ctypes.data)
         return {"items": (0, 2 * n, (-1, 2)), "n_items": n}
+
+
+class SplitTiles(StepPlan):
+    """Work items where long portions have their keys and values expanded: tiles of 64 queries over the segments with at least
+    ``expand_from`` new tokens (as long as the rows of their contexts fit into ``max_rows`` together), with the segments and
+    the first row of each; tiles of ``tile`` queries over all others.  Both ordered as in :class:`LatentTiles`."""
+
+    def __init__(self, tile: int, max_rows: int, expand_from: int) -> None:
+        from ..cache import native
+
+        self._lib = native.lib()
+        self.tile, self.max_rows, self.expand_from = int(tile), int(max_rows), int(expand_from)
+        self.key = ("latent_attention.split", self.tile, self.max_rows, self.expand_from)
+
+    def capacity(self, max_tokens: int, max_segments: int) -> int:
+        return 2 * (max_tokens // self.tile + max_tokens // K.MMA_QUERY_TILE + 2 * max_segments) + 2 * max_segments
+
+    def build(self, seg_q0, seg_qn, seg_ctx, out):
+        n_seg, ctx = len(seg_qn), seg_ctx.ctypes.data
+        rows, longest, long_segs = 0, 0, []
+        row0 = np.full(n_seg, -1, dtype=np.int32)
+        for s in np.nonzero(seg_qn >= self.expand_from)[0]:
+            n = int(seg_ctx[s]) + int(seg_qn[s])
+            if rows + n <= self.max_rows:
+                row0[s] = rows
+                rows += n
+                longest = max(longest, n)
+                long_segs.append(int(s))
+        is_long = row0 >= 0
+        # the segments of the other kind count as having no tokens (the helper lists none of them)
+        short = np.ascontiguousarray(np.where(is_long, 0, seg_qn), dtype=np.int32)
+        long = np.ascontiguousarray(np.where(is_long, seg_qn, 0), dtype=np.int32)
+        at, n = 0, []
+        for qn, tile in ((short, self.tile), (long, K.MMA_QUERY_TILE)):
+            base = out.ctypes.data + 4 * at
+            k = self._lib.locus_plan_query_tiles(n_seg, qn.ctypes.data, tile, 1, base, len(out) - at)
+            if k < 0:
+                raise ValueError("latent attention: the step has more query tiles than the plan's capacity holds")
+            self._lib.locus_sort_tiles_by_position(k, base, ctx)
+            n.append((at, k))
+            at += 2 * k
+        out[at:at + n_seg] = row0
+        out[at + n_seg:at + n_seg + len(long_segs)] = long_segs
+        return {"items": (n[0][0], 2 * n[0][1], (-1, 2)), "n_items": n[0][1], "long_items": (n[1][0], 2 * n[1][1], (-1, 2)),
+                "n_long_items": n[1][1], "row0": (at, n_seg, None), "long_segs": (at + n_seg, len(long_segs), None),
+                "n_long": len(long_segs), "n_rows": rows, "longest": longest}
 
 
 class HeadTiles(StepPlan):
@@ -125,8 +175,8 @@ class LatentAttention(Mixer):
 
     # -- weights ------------------------------------------------------------
     def param_shapes(self):
-        s = {"w_uq": (self.H * (self.dn + self.dr), self.q_rank or self.hidden), "w_uk": (self.H * self.dn, self.kv_rank),
-             "w_uv": (self.H * self.dv, self.kv_rank), "w_o": (self.hidden, self.H * self.dv)}
+        s = {"w_uq": (self.H * (self.dn + self.dr), self.q_rank or self.hidden), "w_ukv": (self.H * (self.dn + self.dv), self.kv_rank),
+             "w_o": (self.hidden, self.H * self.dv)}
         if self.n_down + self.n_gate:
             s["w_down"] = (self.down_width, self.hidden)
         if self.q_rank:
@@ -151,8 +201,8 @@ class LatentAttention(Mixer):
                     TensorSource(f"{p}.{n['dkv_norm']}", (self.kv_rank,), "g_kv", 0, "norm")]
         if self.out_gate:
             out.append(TensorSource(f"{p}.{n['gate']}", (self.n_gate, self.hidden), "w_down", self.n_down))
-        out += [TensorSource(f"{p}.{n['uk']}", (self.H * self.dn, self.kv_rank), "w_uk"),
-               TensorSource(f"{p}.{n['uv']}", (self.H * self.dv, self.kv_rank), "w_uv"),
+        out += [TensorSource(f"{p}.{n['uk']}", (self.H * self.dn, self.kv_rank), "w_ukv"),
+               TensorSource(f"{p}.{n['uv']}", (self.H * self.dv, self.kv_rank), "w_ukv", self.H * self.dn),
                TensorSource(f"{p}.{n['o']}", (self.hidden, self.H * self.dv), "w_o")]
         if self.has_sink:
             out.append(TensorSource(f"{p}.{n['sink']}", (self.H,), "sink", 0, "bias"))
@@ -160,7 +210,10 @@ class LatentAttention(Mixer):
 
     def kernel_modules(self, dtype):
         return ["elementwise", "gemm_simt", "gemv", "latent_attention"] + (["short_conv"] if self.out_gate else []) + (
-            ["gemm_skinny", "gemm_tc"] if dtype == torch.bfloat16 else [])
+            ["gemm_skinny", "gemm_tc"] if dtype == torch.bfloat16 else []) + (["attention_tc"] if self._expand_rows(dtype) else [])
+
+    def _expand_rows(self, dtype) -> int:
+        return K.latent_expand_rows(dtype, self.H, self.dn, self.dr, self.dv, self.kv_rank)
 
     def cache_needs(self):
         return PagedKvSpec(1, self.row, self.window, has_v=False), None
@@ -169,13 +222,15 @@ class LatentAttention(Mixer):
         return [self._query_tiles, self._head_tiles]
 
     @property
-    def _query_tiles(self) -> LatentTiles:
+    def _query_tiles(self) -> StepPlan:
         """Tiles of 16 queries for the CUDA-core kernel, or of 64 / (heads that share a block) for the tensor-core
-        kernel where it takes this mixer's sizes."""
+        kernel where it takes this mixer's sizes; where long portions are expanded, of the short segments alone."""
         dtype = getattr(self, "_dtype", torch.float32)
         self._mma = K.latent_attn_mma_takes(dtype, self.kv_rank, self.dr)
         self._head_shift = K.latent_mma_head_shift(self.H)
-        return LatentTiles(64 >> self._head_shift if self._mma else K.LATENT_QUERY_TILE)
+        tile = 64 >> self._head_shift if self._mma else K.LATENT_QUERY_TILE
+        self._max_rows = self._expand_rows(dtype)
+        return SplitTiles(tile, self._max_rows, K.LATENT_EXPAND_FROM) if self._max_rows else LatentTiles(tile)
 
     @property
     def _head_tiles(self) -> HeadTiles:
@@ -188,8 +243,9 @@ class LatentAttention(Mixer):
         self._dtype = rt.dtype
         # W_uk per head, transposed: the weight [kv_rank, nope_dim] of the product that carries a head's query into
         # the latent space (a layout of the same numbers)
-        self._w_uk_t = self.params["w_uk"].view(self.H, self.dn, self.kv_rank).transpose(1, 2).contiguous()
-        self._w_uv = self.params["w_uv"].view(self.H, self.dv, self.kv_rank)
+        w_uk, w_uv = self.params["w_ukv"].split([self.H * self.dn, self.H * self.dv])
+        self._w_uk_t = w_uk.view(self.H, self.dn, self.kv_rank).transpose(1, 2).contiguous()
+        self._w_uv = w_uv.view(self.H, self.dv, self.kv_rank)
         self._sink = self.params["sink"].float().contiguous() if self.has_sink else None
         self._gq, self._gkv = self.params.get("g_q"), self.params.get("g_kv")
         if "w_down" in self.params:
@@ -219,6 +275,46 @@ class LatentAttention(Mixer):
                           rot_dim=self.dr, rot_pairs=pairs, write=cache.writes and self.has_kv, half_split=half)
         q = rt.rows("latent.q", H * (self.dn + self.dr), rt.dtype, T)
         K.linear(cq if self.q_rank else h, self.params["w_uq"], q)
+        o = rt.rows("latent.o", H * self.dv, rt.dtype, T)
+        tiles = batch.plans[self._tiles_key]
+        if tiles["n_items"]:
+            self._attend_latents(q, o, tiles, batch, cache, gb, rt)
+        if tiles.get("n_long_items"):
+            self._attend_expanded(q, o, tiles, batch, cache, gb, rt)
+        if self.out_gate:
+            K.gate_rows(o, down, self.n_down, n_heads=H, dim=self.dv, laid=self.dv)
+        K.linear(o, self.params["w_o"], residual, accumulate=accumulate)
+
+    def _attend_expanded(self, q, o, tiles, batch, cache, gb, rt) -> None:
+        """The step's long segments: their contexts' keys and values expanded into rows [keys of all heads | values of all heads]."""
+        H, n = self.H, tiles["n_rows"]
+        c = rt.buf(f"latent.c_rows{self.kv_rank}", (self._max_rows, self.kv_rank), rt.dtype)[:n]
+        K.latent_gather(cache.pool, c, segs=tiles["long_segs"], n_segs=tiles["n_long"], row0=tiles["row0"], seg_qn=batch.seg_qn,
+                        seg_ctx=batch.seg_ctx, block_table=gb.block_table, page_tokens=gb.page_tokens, longest=tiles["longest"])
+        kv = rt.buf("latent.kv_rows", (self._max_rows, H * (self.dn + self.dv)), rt.dtype)[:n]
+        K.linear(c, self.params["w_ukv"], kv)
+        keys = tiles["longest"]
+        if self.window > 0:
+            keys = min(keys, self.window + K.TC_ATTN_QUERY_BLOCK)
+        n_splits = K.attn_chunk_tc_splits(tiles["n_long_items"], H, keys, batch.T)
+        part_o = part_ml = None
+        if n_splits > 1:
+            n_o, n_ml = K.attn_chunk_tc_scratch()
+            part_o = rt.buf("attention.chunk_tc_part_o", (n_o,), torch.float32)
+            part_ml = rt.buf("attention.chunk_tc_part_ml", (n_ml,), torch.float32)
+        K.attn_chunk_tc_rows(q, kv[:, : H * self.dn], kv[:, H * self.dn:], o, seg_q0=batch.seg_q0, seg_qn=batch.seg_qn, seg_ctx=batch.seg_ctx,
+                             kv_row0=tiles["row0"], items=tiles["long_items"], n_items=tiles["n_long_items"], n_heads=H, n_kv_heads=H,
+                             head_dim=self.dn, window=self.window, scale=self.scale, n_splits=n_splits, part_o=part_o, part_ml=part_ml,
+                             sink=self._sink if self._sink is not None else False)
+
+    def _attend_latents(self, q, o, tiles, batch, cache, gb, rt) -> None:
+        """The step's short segments over the cached latents themselves (the per-head products run over all rows)."""
+        T, H = batch.T, self.H
+        table = self.position.rotary_table()
+        freq = table.freq64 if table is not None else None
+        pairs = table.rot_dim // 2 if table is not None else 0
+        mag = table.magnitude if table is not None else 1.0
+        half = table is not None and not table.interleaved
         q_nope = rt.rows(f"latent.q_nope{self.dn}", self.dn, rt.dtype, H * T, per_token=H)
         q_rot = rt.rows("latent.q_rot", H * self.dr, rt.dtype, T)
         K.latent_q_split(q, batch.positions, freq, mag, q_nope, q_rot, n_heads=H, nope_dim=self.dn, rot_dim=self.dr,
@@ -229,7 +325,6 @@ class LatentAttention(Mixer):
         q_abs = rt.rows(f"latent.q_abs{self.kv_rank}", self.kv_rank, rt.dtype, H * T, per_token=H)
         K.linear(q_nope, self._w_uk_t, q_abs, layout=lay, n_rows=H * T, lists_ready=True)
         o_lat = rt.rows(f"latent.o_lat{self.kv_rank}", self.kv_rank, rt.dtype, H * T, per_token=H)
-        tiles = batch.plans[self._tiles_key]
         common = dict(seg_q0=batch.seg_q0, seg_qn=batch.seg_qn, seg_ctx=batch.seg_ctx, block_table=gb.block_table,
                       items=tiles["items"], n_items=tiles["n_items"], n_tokens=T, n_heads=H, kv_rank=self.kv_rank,
                       rot_dim=self.dr, page_tokens=gb.page_tokens, window=self.window, scale=self.scale)
@@ -251,11 +346,7 @@ class LatentAttention(Mixer):
             K.latent_attn(q_abs, q_rot, cache.pool, self._sink, o_lat, **common)
         o_hm = rt.rows(f"latent.o_hm{self.dv}", self.dv, rt.dtype, H * T, per_token=H)
         K.linear(o_lat, self._w_uv, o_hm, layout=lay, n_rows=H * T, lists_ready=True)
-        o = rt.rows("latent.o", H * self.dv, rt.dtype, T)
         K.heads_to_rows(o_hm, o, n_tokens=T, n_heads=H)
-        if self.out_gate:
-            K.gate_rows(o, down, self.n_down, n_heads=H, dim=self.dv, laid=self.dv)
-        K.linear(o, self.params["w_o"], residual, accumulate=accumulate)
 
 
 register_mixer("latent_attention", LatentAttention)

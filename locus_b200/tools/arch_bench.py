@@ -1,11 +1,13 @@
-"""Prefill and decode throughput of the Lalepel, the Pozozen, the Mekizen, the Gugozen or the Bebovik design at layer sizes that
+"""Prefill and decode throughput of the Lalepel, the Pozozen, the Mekizen, the Gugozen, the Bebovik or the Megovik design at layer sizes that
 resemble a real model's, beside the closest architecture at equal sizes (random weights, synthetic token ids, one GPU):
 Qwen2-MoE for Lalepel and Pozozen; for Mekizen both Pozozen (the closest mixers: windowed attention beside a float32
 recurrence) and Qwen2-MoE; for Gugozen both Lalepel (the closest mixers: latent attention and a float32 linear recurrence,
 with routed experts) and Qwen2-MoE; for Bebovik both Qwen2 with dense layers only (the closest: grouped-query attention and a
-gated feed-forward of the same sizes) and Mekizen (the closest mixers: attention behind ``head_prep`` with an output gate).
+gated feed-forward of the same sizes) and Mekizen (the closest mixers: attention behind ``head_prep`` with an output gate);
+for Megovik both Gugozen (the closest mixers: grouped-query attention behind ``head_prep`` and latent attention, routed
+experts with sigmoid scores) and Qwen2 with dense layers only (grouped-query attention and a dense gated feed-forward).
 
-    python -m locus_b200.tools.arch_bench [--design lalepel|pozozen|mekizen|gugozen|bebovik] [--size m|s] [--layers 4] [--prefill 2048]
+    python -m locus_b200.tools.arch_bench [--design lalepel|pozozen|mekizen|gugozen|bebovik|megovik] [--size m|s] [--layers 4] [--prefill 2048]
                                           [--batch 8] [--context 4096] [--steps 16] [--warmup 3] [--dtype bf16|fp32]
                                           [--kernels]
 
@@ -19,7 +21,10 @@ layer's keys and values), all with a dense squared-ReLU feed-forward of four tim
 (grouped-query attention with a learned sink, gated linear attention, latent attention, latent attention on the third
 layer's rows), all with clamped gated experts weighted on their input and a shared expert; Bebovik's are all grouped-query
 attention in chunks (heads / 4 key/value heads, as in the dense Qwen2 beside it) and a clamped gated feed-forward of the width
-of the others' shared expert.  Timed on the device with CUDA events after warm-up; every step reads its weights (several
+of the others' shared expert; Megovik's cycle through (latent attention with a dense rectified gate, grouped-query attention
+with routed experts, latent attention behind a query latent with a dense gate, latent attention with routed experts), heads and
+latents as in Gugozen beside it, the dense gates of the width of the shared expert, every layer once (``--loop`` N: all layers N
+times in a row).  Timed on the device with CUDA events after warm-up; every step reads its weights (several
 hundred MB: more than the L2 holds).  ``--kernels`` adds, for one eager prefill step and one eager decode step of
 each model, the time by kernel entry point, and for the mixers' own kernels what their bytes or flops would take
 at the measured peaks.  Prints one JSON line.
@@ -122,6 +127,28 @@ def bebovik_config(z, n_layers):
             "embedding": {"scale": 8.0}, "logit_scale": 0.5, "logit_softcap": 25.0, "layers": [layer] * n_layers}
 
 
+def megovik_config(z, n_layers, max_pos, times=1):
+    moe = {"kind": "moe", "router": {"experts": z["experts"], "top": z["top"], "scale": 2.5, "groups": {"count": 4, "keep": 2}},
+           "expert": {"ff": z["ff"]}}
+    mlp = {"kind": "dense", "ff": z["shared"]}
+
+    def lat(ff, q_latent=False):
+        m = {"heads": z["heads"], "dim": z["dim"], "vdim": z["vdim"], "kv_rank": z["kv_rank"], "scale": z["dim"] ** -0.5}
+        if q_latent:
+            m["q_rank"] = z["q_rank"]
+        return {"type": "latent_attention_2" if q_latent else "latent_attention", "mlp": ff, "mixer": m}
+
+    att = {"type": "attention", "mlp": moe, "mixer": {
+        "heads": z["heads"], "kv_heads": max(1, z["heads"] // 4), "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5,
+        "q_temp": {"coef": 0.1, "every": 2048}}}
+    cycle = (lat(mlp), att, lat(mlp, True), lat(moe))
+    raw = {"architecture": "Megovik", "width": z["width"], "vocab": z["vocab"], "max_positions": max_pos, "norm": {"eps": 1e-6},
+           "embedding": {"scale": 8.0}, "logit_scale": 0.5, "layers": [cycle[i % 4] for i in range(n_layers)]}
+    if times > 1:
+        raw["loop"] = {"start": 0, "stop": n_layers, "times": times}
+    return raw
+
+
 def qwen_dense_config(z, n_layers, max_pos):
     """Qwen2 with dense layers only: grouped-query attention and a SwiGLU of the sizes of ``bebovik_config``."""
     raw = qwen_config(z, n_layers, max_pos)
@@ -172,13 +199,17 @@ def run(args) -> dict:
     gen = torch.Generator().manual_seed(5)
     design = args.design
     own = {"lalepel": lalepel_config, "pozozen": pozozen_config, "mekizen": mekizen_config,
-           "gugozen": gugozen_config, "bebovik": bebovik_config}[design](z, args.layers)
+           "gugozen": gugozen_config, "bebovik": bebovik_config,
+           "megovik": lambda z, n: megovik_config(z, n, max(ctx, T) + 8, args.loop)}[design](z, args.layers)
     raws = {design: own}
     if design == "mekizen":
         raws["pozozen"] = pozozen_config(z, args.layers)
     if design == "gugozen":
         raws["lalepel"] = lalepel_config(z, args.layers)
-    if design == "bebovik":
+    if design == "megovik":
+        raws["gugozen"] = gugozen_config(z, args.layers)
+        raws["qwen2_dense"] = qwen_dense_config(z, args.layers, max(ctx, T) + 8)
+    elif design == "bebovik":
         raws["mekizen"] = mekizen_config(z, args.layers)
         raws["qwen2_dense"] = qwen_dense_config(z, args.layers, max(ctx, T) + 8)
     else:
@@ -265,6 +296,27 @@ def run(args) -> dict:
     H, R = z["heads"], z["kv_rank"] + z["rot"]
     keys_avg = sum(min(p + 1, z["window"]) for p in range(T)) / T
     fma_tflops = 148 * 128 * 2 * 1.965e9 / 1e12       # float32 FMAs of the CUDA cores at the top clock
+    if design == "megovik":
+        G, D, Wd, r = max(1, H // 4), z["dim"], z["width"], z["kv_rank"]
+        causal = T * (T + 1) / 2
+        row = T / (pk["hbm_gbs"] * 1e9) * 1e6        # us per byte of a row, over the portion's rows
+        bounds = {
+            "attn_prefill_us": 2.0 * causal * H * 2 * D / (pk["bf16_tflops"] * 1e12) * 1e6,
+            # the pages hold normed keys and, as values, the keys as projected: two planes
+            "attn_decode_us": B * ctx * 2 * G * D * el / (pk["hbm_gbs"] * 1e9) * 1e6,
+            "latent_attn_prefill_us": 2.0 * causal * H * 2 * r / (pk["bf16_tflops"] * 1e12) * 1e6,
+            "latent_attn_decode_us": B * ctx * r * el / (pk["hbm_gbs"] * 1e9) * 1e6,
+            "gugozen_latent_attn_prefill_us": 2.0 * causal * H * (R + r) / (pk["bf16_tflops"] * 1e12) * 1e6,
+            "gugozen_latent_attn_decode_us": B * ctx * R * el / (pk["hbm_gbs"] * 1e9) * 1e6,
+            "head_prep_prefill_us": row * ((H + G) * D * 4 + (H + 2 * G) * D * el),
+            "dense_ff_prefill_us": 2.0 * T * 3 * Wd * z["shared"] / (pk["bf16_tflops"] * 1e12) * 1e6,
+            "dense_ff_decode_us": 3 * Wd * z["shared"] * el / (pk["hbm_gbs"] * 1e9) * 1e6,
+        }
+        return {"metric": f"prefill and decode tokens/s, Megovik beside Gugozen and dense Qwen2 at equal layer sizes "
+                          f"({args.size}, {args.layers} layers{f' x {args.loop}' if args.loop > 1 else ''}, {args.dtype})",
+                "size": z, "layers": args.layers, "dtype": args.dtype, "data": "synthetic", "designs": out,
+                "bounds_per_layer": bounds, "peaks": pk,
+                "l2": "no flush: every step reads its weights, more than the 126 MB L2"}
     if design == "bebovik":
         G, D, Wd, ff = max(1, H // 4), z["dim"], z["width"], z["shared"]
         in_w = (2 * H + 2 * G) * D                   # q, k, v and the gate
@@ -368,7 +420,7 @@ def run(args) -> dict:
 
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(prog="arch_bench", description=__doc__.split("\n\n")[0])
-    ap.add_argument("--design", default="lalepel", choices=["lalepel", "pozozen", "mekizen", "gugozen", "bebovik"])
+    ap.add_argument("--design", default="lalepel", choices=["lalepel", "pozozen", "mekizen", "gugozen", "bebovik", "megovik"])
     ap.add_argument("--size", default="m", choices=sorted(SIZES))
     ap.add_argument("--layers", type=int, default=4)
     ap.add_argument("--prefill", type=int, default=2048)
@@ -377,6 +429,7 @@ def main(argv=None) -> int:
     ap.add_argument("--steps", type=int, default=16)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--dtype", default="bf16", choices=["bf16", "fp32"])
+    ap.add_argument("--loop", type=int, default=1, help="megovik: all layers that many times in a row")
     ap.add_argument("--kernels", action="store_true")
     args = ap.parse_args(argv)
     print(json.dumps(run(args)))

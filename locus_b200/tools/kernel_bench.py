@@ -6,6 +6,7 @@
     python -m locus_b200.tools.kernel_bench experts --tokens 2048 [--experts 60 --top-k 4 --k 2048 --n 1408] [--part up|down]
     python -m locus_b200.tools.kernel_bench recurrence --tokens 2048 --batch 1 [--heads 16 --head-dim 128 --v-dim 128]
                                                        [--per-group 1] [--ones] [--retention | --delta | --gla]
+    python -m locus_b200.tools.kernel_bench latent --tokens 2048 --batch 1 [--ctx 0] [--rank 512] [--absorbed]
     python -m locus_b200.tools.kernel_bench head_prep --tokens 2048 --batch 1 [--window 4096]
     python -m locus_b200.tools.kernel_bench rows --tokens 2048 [--k 2048 --heads 16 --kv-heads 4 --head-dim 128]
 
@@ -67,15 +68,18 @@ def bench_linear(args) -> None:
     x = torch.randn(M, Kd, device=dev).to(dt)
     out = torch.zeros(M, N, device=dev, dtype=torch.float32 if args.accumulate else dt)
     state = {"i": 0}
+    extra = {}
+    if args.rectified and args.dual:
+        extra = dict(act="reglu", bias=torch.randn(2 * N, device=dev).to(dt))
 
     def fn():
         i = state["i"] % copies
         state["i"] += 1
-        K.linear(x, ws[i], out, w2=w2s[i] if args.dual else None, accumulate=args.accumulate)
+        K.linear(x, ws[i], out, w2=w2s[i] if args.dual else None, accumulate=args.accumulate, **extra)
 
     us = _time(fn, args.iters, args.graph)
     flops = 2.0 * M * N * Kd * (2 if args.dual else 1)
-    print(f"linear M={M} N={N} K={Kd} dual={int(args.dual)} accumulate={int(args.accumulate)} {args.dtype}: "
+    print(f"linear M={M} N={N} K={Kd} dual={int(args.dual)}{' rectified' if extra else ''} accumulate={int(args.accumulate)} {args.dtype}: "
           f"{us:.1f} us/call  {flops / us / 1e6:.1f} TFLOP/s  weights {wbytes / us / 1e3:.1f} GB/s  "
           f"(tensor-core error word {K.tc_error() if dt == torch.bfloat16 else 0})")
 
@@ -147,6 +151,8 @@ def _paged(args, B: int, ctx: int, new: int):
         kw["chunk"] = args.chunk
     if args.keep_first or args.sink:
         kw.update(keep_first=args.keep_first, sink=args.sink)
+    if args.slopes:
+        kw["slopes"] = torch.tensor([2.0 ** (-8.0 * (h + 1) / nh) for h in range(nh)], dtype=torch.float32, device=dev)
     return pool, q, torch.empty_like(q), meta, kw, i32
 
 
@@ -169,7 +175,7 @@ def bench_attn_decode(args) -> None:
         seen = ctx % args.chunk + 1
     byts = B * seen * 2 * args.kv_heads * args.head_dim * pool.element_size()
     print(f"attn_decode batch={B} ctx={ctx} heads={args.heads}/{args.kv_heads} head_dim={args.head_dim} window={args.window} "
-          f"keep_first={args.keep_first} sink={args.sink} {args.dtype}: "
+          f"keep_first={args.keep_first} sink={args.sink} slopes={args.slopes} {args.dtype}: "
           f"{us:.1f} us/call  cache read {byts / us / 1e3:.1f} GB/s")
 
 
@@ -205,7 +211,7 @@ def bench_attn_chunk(args) -> None:
         seen = sum(p % args.chunk + 1 for p in range(ctx, ctx + T))
     flops = 4.0 * args.heads * args.head_dim * seen
     print(f"attn_chunk tokens={T} ctx={ctx} heads={args.heads}/{args.kv_heads} head_dim={args.head_dim} window={args.window} "
-          f"keep_first={args.keep_first} sink={args.sink} "
+          f"keep_first={args.keep_first} sink={args.sink} slopes={args.slopes} "
           f"{f'tcgen05, {n_splits} key ranges' if tc else (f'mma.sync, {n_splits} key ranges' if mma else 'cuda cores')}: {us:.1f} us/call  {flops / us / 1e6:.1f} TFLOP/s (causal flops)")
 
 
@@ -379,6 +385,7 @@ def bench_rows(args) -> None:
     cases = [
         ("dyt: addition, both norms", each(n, lambda i: K.dyt(x[i], norm, h[i], add=(y[i], norm, w))), T * W * (12 + el)),
         ("dyt: norm alone", each(n, lambda i: K.dyt(x[i], norm, h[i])), T * W * (4 + el)),
+        ("rmsnorm, rows added in front", each(n, lambda i: K.rmsnorm(x[i], w, 1e-5, h[i], add_rows=y[i])), T * W * (12 + el)),
         ("rmsnorm", each(n, lambda i: K.rmsnorm(x[i], w, 1e-5, h[i])), T * W * (4 + el)),
         ("rmsnorm_add", each(n, lambda i: K.rmsnorm_add(y[i], w, 1e-5, x[i])), T * W * 12),
         ("head_prep, a block per token, adjacent pairs", each(n2, lambda i: K.head_prep(
@@ -387,6 +394,9 @@ def bench_rows(args) -> None:
          T * (H + 2 * G) * D * (4 + el)),
         ("head_prep, a warp per head", each(n2, lambda i: K.head_prep(proj[i], q_out=q[i], interleaved=True, **heads)),
          T * (H + 2 * G) * D * (4 + el)),
+        ("head_prep, no rotation, q by position, values from k", each(n2, lambda i: K.head_prep(
+            proj[i], q_out=q[i], n_rows=T, q_temp=(0.5, 256), **{**heads, "offsets": (0, H * D, H * D), "inv_freq": None, "rot": 0})),
+         T * ((H + G) * D * 4 + (H + 2 * G) * D * el)),
         ("rope_kv_write", each(n2, lambda i: K.rope_kv_write(low[i], pos, inv, q[i], pool, where, n_heads=H, n_kv_heads=G, head_dim=D,
                                                              rot_dim=D, interleaved=False, page_tokens=P)), T * (H + 2 * G) * D * 2 * el),
         ("gate_rows", each(n2, lambda i: K.gate_rows(q[i], proj[i], (H + 2 * G) * D, n_heads=H, dim=D, laid=D)), T * H * D * (4 + 2 * el)),
@@ -394,6 +404,76 @@ def bench_rows(args) -> None:
     for name, fn, by in cases:
         us = _time(fn, args.iters, args.graph)
         print(f"{name}: {T} rows (width {W}, heads {H}/{G} of {D}), {args.dtype}: {us:.1f} us/call, {by / us / 1e3:.0f} GB/s")
+
+
+def bench_latent(args) -> None:
+    """Latent attention of ``--batch`` requests with ``--tokens`` new tokens each behind ``--ctx`` cached ones, heads of
+    ``--head-dim`` on a latent of ``--rank`` without a rotated part: over the cached latents (single tokens, short portions;
+    ``--absorbed``: any), with the two per-head products around it, or with the heads' keys and values expanded (portions of
+    ``kernels.LATENT_EXPAND_FROM`` tokens on).  One line per kernel and one for all."""
+    dev, dt = "cuda:0", torch.bfloat16
+    B, n, ctx, H, D, r, P = args.batch, args.tokens, args.ctx, args.heads, args.head_dim, args.rank, args.page_tokens
+    T, total = B * n, ctx + n
+    per = -(-total // P)
+    copies = max(1, min(16, int(3e8 // (B * per * P * r * 2))))
+    pools = [torch.randn(B * per, 1, 1, P, r, device=dev).to(dt) for _ in range(copies)]
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    table = torch.arange(B * per, dtype=torch.int32, device=dev).view(B, per).contiguous()
+    meta = dict(seg_q0=i32([i * n for i in range(B)]), seg_qn=i32([n] * B), seg_ctx=i32([ctx] * B))
+    q = torch.randn(T, H * D, device=dev).to(dt)
+    w_ukv = (torch.randn(2 * H * D, r, device=dev) * 0.02).to(dt)
+    o, state = torch.empty(T, H * D, device=dev, dtype=dt), {"i": 0}
+    keys = B * (n * ctx + n * (n + 1) / 2)
+
+    def pool():
+        state["i"] += 1
+        return pools[state["i"] % copies]
+
+    steps = []
+    if n >= K.LATENT_EXPAND_FROM and not args.absorbed:
+        c, kv = torch.empty(B * total, r, device=dev, dtype=dt), torch.empty(B * total, 2 * H * D, device=dev, dtype=dt)
+        row0, segs = i32([i * total for i in range(B)]), i32(list(range(B)))
+        items = i32([[s, a] for a in range(0, n, 64) for s in range(B)])
+        n_splits = K.attn_chunk_tc_splits(len(items), H, total, T)
+        n_o, n_ml = K.attn_chunk_tc_scratch()
+        extra = dict(n_splits=n_splits, part_o=torch.empty(n_o, device=dev), part_ml=torch.empty(n_ml, device=dev)) if n_splits > 1 else {}
+        steps = [("latent_gather", lambda: K.latent_gather(pool(), c, segs=segs, n_segs=B, row0=row0, seg_qn=meta["seg_qn"], seg_ctx=meta["seg_ctx"],
+                                                           block_table=table, page_tokens=P, longest=total), 0, 4.0 * B * total * r),
+                 ("expansion", lambda: K.linear(c, w_ukv, kv), 2.0 * B * total * 2 * H * D * r, 2.0 * (B * total * (r + 2 * H * D) + w_ukv.numel())),
+                 (f"attn_chunk_tc_rows ({n_splits} key ranges)",
+                  lambda: K.attn_chunk_tc_rows(q, kv[:, : H * D], kv[:, H * D:], o, kv_row0=row0, items=items, n_items=len(items), n_heads=H,
+                                               n_kv_heads=H, head_dim=D, window=0, scale=D ** -0.5, **meta, **extra),
+                  4.0 * keys * H * D, 0)]
+    else:
+        shift = K.latent_mma_head_shift(H)
+        items = i32([[s, a] for a in range(0, n, 64 >> shift) for s in range(B)])
+        tile = K.head_tile(T, dt, True)
+        tiles = [(h, h * T + a, min(tile, T - a)) for h in range(H) for a in range(0, T, tile)]
+        lay = K.HeadLayout(H, tile, i32([h * T for h in range(H + 1)]), *[i32([t[j] for t in tiles]) for j in range(3)], i32([len(tiles)]), len(tiles))
+        w_uk_t, w_uv = w_ukv[: H * D].view(H, D, r).transpose(1, 2).contiguous(), w_ukv[H * D:].view(H, D, r)
+        q_hm, q_rot = torch.empty(H * T, D, device=dev, dtype=dt), torch.empty(T, 0, device=dev, dtype=dt)
+        q_abs, o_lat, o_hm = (torch.randn(H * T, w, device=dev).to(dt) for w in (r, r, D))
+        n_splits = K.latent_attn_mma_splits(len(items), H, shift, total)
+        n_o, n_ml = K.latent_attn_mma_scratch(r)
+        extra = dict(n_splits=n_splits, part_o=torch.empty(n_o, device=dev), part_ml=torch.empty(n_ml, device=dev)) if n_splits > 1 else {}
+        pos, fl = torch.zeros(T, dtype=torch.int32, device=dev), 2.0 * T * H * D * r
+        steps = [("latent_q_split", lambda: K.latent_q_split(q, pos, None, 1.0, q_hm, q_rot, n_heads=H, nope_dim=D, rot_dim=0, rot_pairs=0), 0, 4.0 * T * H * D),
+                 ("product into the latent space", lambda: K.linear(q_hm, w_uk_t, q_abs, layout=lay, n_rows=H * T, lists_ready=True), fl, w_uk_t.numel() * 2.0),
+                 (f"latent_attn_mma ({n_splits} key ranges)",
+                  lambda: K.latent_attn_mma(q_abs, q_rot, pool(), None, o_lat, head_shift=shift, items=items, n_items=len(items), n_tokens=T, n_heads=H,
+                                            kv_rank=r, rot_dim=0, page_tokens=P, window=0, scale=D ** -0.5, block_table=table, **meta, **extra),
+                  4.0 * keys * H * r, 2.0 * B * total * r),
+                 ("product out of the latent space", lambda: K.linear(o_lat, w_uv, o_hm, layout=lay, n_rows=H * T, lists_ready=True), fl, w_uv.numel() * 2.0),
+                 ("heads_to_rows", lambda: K.heads_to_rows(o_hm, o, n_tokens=T, n_heads=H), 0, 4.0 * T * H * D)]
+
+    def all_of_it():
+        for _, fn, _, _ in steps:
+            fn()
+    steps.append(("all", all_of_it, 4.0 * keys * H * D, 2.0 * B * total * r))
+    for name, fn, fl, by in steps:
+        us = _time(fn, args.iters, args.graph)
+        print(f"latent {B} x {n} tokens behind {ctx}, {H} heads of {D}, rank {r}: {name}: {us:.1f} us/call"
+              + (f"  {fl / us / 1e6:.1f} TFLOP/s" if fl else "") + (f"  {by / us / 1e3:.0f} GB/s" if by else ""))
 
 
 def bench_sample(args) -> None:
@@ -418,7 +498,7 @@ def bench_sample(args) -> None:
 
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(prog="kernel_bench")
-    ap.add_argument("kernel", choices=["linear", "attn_decode", "attn_chunk", "experts", "sample", "recurrence", "head_prep", "rows"])
+    ap.add_argument("kernel", choices=["linear", "attn_decode", "attn_chunk", "experts", "sample", "recurrence", "head_prep", "rows", "latent"])
     ap.add_argument("--rows", type=int, default=8, help="sample: rows of logits")
     ap.add_argument("--vocab", type=int, default=151936, help="sample: logits of a row")
     ap.add_argument("--one-block", action="store_true", help="sample: never the cluster kernel")
@@ -443,11 +523,15 @@ def main(argv=None) -> int:
     ap.add_argument("--delta", action="store_true", help="recurrence: the gated delta rule instead")
     ap.add_argument("--gla", action="store_true", help="recurrence: gated linear attention (a decay per key channel) instead")
     ap.add_argument("--page-tokens", type=int, default=64)
+    ap.add_argument("--rank", type=int, default=512, help="latent: the latent's size")
+    ap.add_argument("--absorbed", action="store_true", help="latent: long portions over the cached latents, too")
     ap.add_argument("--window", type=int, default=0)
     ap.add_argument("--chunk", type=int, default=0, help="attention: queries see the keys of their own chunk of this many positions")
     ap.add_argument("--keep-first", type=int, default=0, dest="keep_first",
                     help="attention: with --window, a request's first tokens stay in sight")
     ap.add_argument("--sink", action="store_true", help="attention: one more term of score 0 in the softmax's denominator")
+    ap.add_argument("--slopes", action="store_true", help="attention: a distance bias, a slope per head")
+    ap.add_argument("--rectified", action="store_true", help="linear: with --dual, the rectified gate with biases instead of SwiGLU")
     ap.add_argument("--experts", type=int, default=60)
     ap.add_argument("--top-k", type=int, default=4)
     ap.add_argument("--tile", type=int, default=0, help="experts: rows of a tile instead of the engine's choice")
@@ -472,7 +556,7 @@ def main(argv=None) -> int:
         print("kernel_bench: no CUDA device", file=sys.stderr)
         return 1
     {"linear": bench_linear, "attn_decode": bench_attn_decode, "attn_chunk": bench_attn_chunk,
-     "experts": bench_experts, "sample": bench_sample, "recurrence": bench_recurrence, "head_prep": bench_head_prep, "rows": bench_rows}[args.kernel](args)
+     "experts": bench_experts, "sample": bench_sample, "recurrence": bench_recurrence, "head_prep": bench_head_prep, "rows": bench_rows, "latent": bench_latent}[args.kernel](args)
     return 0
 
 

@@ -494,6 +494,39 @@ def latent_attn(q_abs_hm, q_rot, pool, sink, out_hm, *, seg_q0, seg_qn, seg_ctx,
                 out_hm[h * T + q0 + i] = ((e / den) @ rows[:, :kv_rank]).to(out_hm.dtype)
 
 
+def latent_gather(pool, out, *, segs, n_segs, row0, seg_qn, seg_ctx, block_table, page_tokens, longest):
+    for i in range(n_segs):
+        s = int(segs[i])
+        n = int(seg_ctx[s]) + int(seg_qn[s])
+        assert n <= longest
+        for t in range(n):
+            page = int(block_table[s, t // page_tokens])
+            out[int(row0[s]) + t] = pool[page, 0, 0, t % page_tokens, : out.shape[1]] if page >= 0 else 0.0
+
+
+def attn_chunk_tc_splits(n_items, n_heads, max_ctx, n_rows=0):
+    return 1
+
+
+def attn_chunk_tc_rows(q, k, v, out, *, seg_q0, seg_qn, seg_ctx, kv_row0, items, n_items, n_heads, n_kv_heads, head_dim, window, scale,
+                       n_splits=1, part_o=None, part_ml=None, keep_first=0, sink=False, chunk=0, slopes=None):
+    assert window == 0 and keep_first == 0 and chunk == 0
+    group = n_heads // n_kv_heads
+    for seg in sorted({int(items[i, 0]) for i in range(n_items)}):
+        q0, qn, ctx, r0 = int(seg_q0[seg]), int(seg_qn[seg]), int(seg_ctx[seg]), int(kv_row0[seg])
+        for i in range(qn):
+            p = ctx + i
+            for h in range(n_heads):
+                cols = slice((h // group) * head_dim, (h // group + 1) * head_dim)
+                s = (_f(k[r0:r0 + p + 1, cols]) @ _f(q[q0 + i].view(n_heads, head_dim)[h])) * scale
+                if slopes is not None:
+                    s = s - _f(slopes)[h] * (p - torch.arange(p + 1, dtype=s.dtype))
+                if sink is not False:
+                    s = torch.cat([s, (_f(sink)[h] if isinstance(sink, torch.Tensor) else s.new_zeros(())).view(1)])
+                w = torch.softmax(s, 0)[: p + 1]
+                out[q0 + i].view(n_heads, head_dim)[h] = (w @ _f(v[r0:r0 + p + 1, cols])).to(out.dtype)
+
+
 def latent_attn_mma_takes(dtype, kv_rank, rot_dim):
     return False
 
@@ -799,7 +832,7 @@ def head_tile(n_tokens, dtype, widths_ok):
 
 
 _NAMES = ["embed_rows", "rmsnorm", "rmsnorm_adds", "attn_chunk_tc_takes", "linear", "rope_kv_write", "attn_chunk", "attn_chunk_mma", "attn_decode", "router_topk", "router_logits", "router_select",
-          "moe_sort", "route_small", "route_small_takes", "route_fused_small", "moe_combine", "gather_rows", "add_rows", "apply_penalties", "sample",
+          "moe_sort", "route_small", "route_small_takes", "route_fused_small", "moe_combine", "gather_rows", "add_rows", "latent_gather", "attn_chunk_tc_splits", "attn_chunk_tc_rows", "apply_penalties", "sample",
           "cast_rows", "rmsnorm_add", "latent_prep", "latent_q_split", "latent_attn", "heads_to_rows", "retention_scan",
           "retention_gate_norm", "head_tile", "latent_attn_mma_takes", "layernorm", "stream_update", "moe_identity",
           "gated_recurrence", "mlstm_gates", "mlstm_out", "ssm_conv", "ssm_out", "head_prep", "gate_rows", "delta_rule", "delta_out",
