@@ -21,6 +21,7 @@
 //   latent_attn     attention over the latent rows, float32 arithmetic: a sliding window (a query at position p
 //                   sees p - window < j <= p; 0 = all), and a sink per head: exp(sink[h]) joins the softmax's
 //                   denominator, without a key or a value
+//   latent_decode   the same for single new tokens on the tensor cores, a row read once for sixteen heads
 //   heads_to_rows   [head][token][d] -> [token][head * d]
 //   latent_gather   cached rows of some requests as plain rows, for portions whose heads' keys and values are expanded
 //
@@ -713,7 +714,7 @@ __global__ void __launch_bounds__(256) latent_attn_mma_kernel(LatentMmaArgs a) {
     }
 }
 
-// One block per (item, head block): the ranges' partial results, in ascending order of the ranges.
+// Blocks per (item, head block), each for LM_ROWS / gridDim.z of its rows: the ranges' partial results, in ascending order.
 __global__ void __launch_bounds__(256) latent_attn_merge_kernel(LatentMmaArgs a, int kvr) {
     __shared__ float s_w[16][LM_ROWS];   // weight of every range for every row
     __shared__ float s_inv[LM_ROWS];
@@ -744,11 +745,13 @@ __global__ void __launch_bounds__(256) latent_attn_merge_kernel(LatentMmaArgs a,
         s_inv[r] = 1.0f / l;
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < LM_ROWS * kvr; i += 256) {
-        const int r = i / kvr, d = i % kvr;
+    const int rows = LM_ROWS / gridDim.z;
+    for (int i = threadIdx.x; i < rows * kvr; i += 256) {
+        const int r = blockIdx.z * rows + i / kvr, d = i % kvr;
         const int qi = r >> a.hb_shift, h = h0 + (r & (HB - 1));
         if (qi >= nq || h >= a.H) continue;
         float acc = 0.f;
+#pragma unroll 8
         for (int sp = 0; sp < n_live; ++sp) acc += a.part_o[((unit0 + sp) * LM_ROWS + r) * kvr + d] * s_w[sp][r];
         a.out[(static_cast<size_t>(h) * a.T + row0 + qi) * kvr + d] = __float2bfloat16_rn(acc * s_inv[r]);
     }
@@ -763,7 +766,7 @@ static int launch_latent_mma(const LatentMmaArgs& a, int n_items, size_t smem, c
     const int HB = 1 << a.hb_shift;
     locus_launch(latent_attn_mma_kernel<KVR>, dim3((a.H + HB - 1) / HB, n_items, a.n_splits), dim3(256), smem, stream, a);
     if (a.n_splits > 1)
-        locus_launch(latent_attn_merge_kernel, dim3((a.H + HB - 1) / HB, n_items), dim3(256), 0, stream, a, KVR);
+        locus_launch(latent_attn_merge_kernel, dim3((a.H + HB - 1) / HB, n_items, 16), dim3(256), 0, stream, a, KVR);
     return locus_launch_status();
 }
 
@@ -807,5 +810,311 @@ extern "C" int locus_latent_attn_mma(const void* q_abs, const void* q_rot, const
         case 448: return launch_latent_mma<448>(a, n_items, smem, stream);
         case 512: return launch_latent_mma<512>(a, n_items, smem, stream);
     }
+    return LOCUS_ERR_UNSUPPORTED;
+}
+
+// ---------------------------------------------------------------------------
+// Decoding over the latent rows: one new token per request, bfloat16, mma.sync m16n8k16 with float32 accumulation.
+//
+// Reading the cache is what there is to do: a row of R = KVR + ROT elements serves all heads.  Sixteen heads are the M side of
+// every product, so a block takes sixteen heads of one request over a range of its keys (blockIdx.z) and reads each row once.
+// Eight warps; key tiles of 64 rows arrive by cp.async, three stages deep (up to 224 KB of shared memory, a block per SM).
+//   scores    warp w takes the tile's keys 8 w .. 8 w + 7; its A fragments, the sixteen queries, stay in registers for the
+//             whole range (R / 4 registers), two chains of accumulators
+//   softmax   scores go through shared memory once; every warp then forms the rows' running maximum and the whole tile's
+//             probabilities itself (the same numbers), as A fragments of the second product
+//   values    warp w sums the latent's dimensions [w KVR / 8, (w + 1) KVR / 8) over the tile's keys
+// A range leaves unnormalised sums, maxima and denominators; latent_decode_merge_kernel, a block per (head, request), adds the
+// ranges up in ascending order.  Rows in shared memory are padded by 16 bytes so that ldmatrix reads no bank twice.
+#define LD_KEYS 64
+#define LD_STAGES 3
+#define LD_HEADS 16
+#define LD_MAX_RANGES 64
+
+struct LatentDecodeArgs {
+    const bf16* q_abs;       // [H, T, KVR]
+    const bf16* q_rot;       // [T, H, ROT]
+    const bf16* pool;        // [n_pages][page_tokens][R]
+    const float* sink;       // [H] or null
+    bf16* out;               // [H, T, KVR]
+    const int* seg_q0;
+    const int* seg_ctx;
+    const int* block_table;
+    int table_stride;
+    const int* items;        // [n_items] segments with one new token
+    int T, H, page_tokens, window, n_ranges;
+    float scale;
+    float* part_o;           // [item][head block][range][16][KVR]
+    float* part_ml;          // [item][head block][range][16][2]  maximum (base 2) and denominator
+};
+
+// Key tiles of a request and how they are cut (the same in both kernels).
+__device__ __forceinline__ void ld_tiles(int p, int window, int n_ranges, int& t_lo, int& first_tile, int& n_tiles, int& per_range) {
+    t_lo = window > 0 ? max(0, p - window + 1) : 0;
+    first_tile = (t_lo / LD_KEYS) * LD_KEYS;
+    n_tiles = (p - first_tile) / LD_KEYS + 1;
+    per_range = (n_tiles + n_ranges - 1) / n_ranges;
+}
+
+template <int KVR, int ROT>
+__global__ void __launch_bounds__(256, 1) latent_decode_kernel(LatentDecodeArgs a) {
+    constexpr int R = KVR + ROT;
+    constexpr int LDS = R + 8;             // padded row, elements
+    constexpr int CH = R / 8;              // 16-byte pieces of a row
+    constexpr int NK = R / 32;             // pairs of k-steps of the scores
+    constexpr int DW = KVR / 8;            // dimensions of a warp
+    constexpr int NT = DW / 8;             // its 8-wide output tiles
+    constexpr int SLD = LD_KEYS + 4;       // padded row of scores
+    static_assert(R % 32 == 0 && KVR % 128 == 0, "whole fragments");
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    bf16* sK = reinterpret_cast<bf16*>(smem_raw);                                // [stages][64][LDS]
+    float* sS = reinterpret_cast<float*>(sK + LD_STAGES * LD_KEYS * LDS);        // [16][SLD]
+    pdl_entry();
+    pdl_trigger();
+    const int item = blockIdx.y, h0 = blockIdx.x * LD_HEADS;
+    const int seg = a.items[item];
+    const int p = a.seg_ctx[seg], row = a.seg_q0[seg];
+    const int* table = a.block_table + static_cast<size_t>(seg) * a.table_stride;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, qd = lane & 3;
+    const int P = a.page_tokens;
+    int t_lo, first_tile, n_tiles_all, per_range;
+    ld_tiles(p, a.window, a.n_ranges, t_lo, first_tile, n_tiles_all, per_range);
+    first_tile += blockIdx.z * per_range * LD_KEYS;
+    const int n_tiles = min(per_range, n_tiles_all - static_cast<int>(blockIdx.z) * per_range);
+    if (n_tiles <= 0) return;   // the merge counts the live ranges the same way
+
+    auto load_tile = [&](int it) {
+        bf16* dst = sK + (it % LD_STAGES) * LD_KEYS * LDS;
+        if (it < n_tiles) {
+            const int tile0 = first_tile + it * LD_KEYS;
+#pragma unroll
+            for (int k = 0; k < LD_KEYS / 8; ++k) {
+                const int r = warp + 8 * k, t = tile0 + r;
+                const bool ok = t >= t_lo && t <= p;
+                const int tt = ok ? t : p;   // any live position: nothing is copied when !ok
+                const bf16* src = a.pool + (static_cast<size_t>(table[tt / P]) * P + tt % P) * R;
+#pragma unroll
+                for (int c = lane; c < CH; c += 32) lm_cp16(lm_addr(dst + r * LDS + c * 8), src + c * 8, ok ? 16 : 0);
+            }
+        }
+        lm_commit();   // (an empty group keeps the count)
+    };
+    // the sixteen queries first, into the last stage's buffer, which no tile needs before they are in registers
+    bf16* sQ = sK + (LD_STAGES - 1) * LD_KEYS * LDS;
+    for (int i = tid; i < LD_HEADS * CH; i += 256) {
+        const int r = i / CH, c = i % CH;
+        const int h = h0 + r;
+        const bool ok = h < a.H;
+        const int hh = ok ? h : h0;
+        const bf16* src = c < KVR / 8 ? a.q_abs + (static_cast<size_t>(hh) * a.T + row) * KVR + c * 8
+                                      : a.q_rot + (static_cast<size_t>(row) * a.H + hh) * ROT + (c - KVR / 8) * 8;
+        lm_cp16(lm_addr(sQ + r * LDS + c * 8), src, ok ? 16 : 0);
+    }
+    lm_commit();
+#pragma unroll
+    for (int s = 0; s < LD_STAGES - 1; ++s) load_tile(s);
+    lm_wait<LD_STAGES - 1>();
+    __syncthreads();
+    uint32_t qf[2 * NK][4];
+    {
+        const uint32_t qa = lm_addr(sQ + (lane & 15) * LDS + (lane >> 4) * 8);
+#pragma unroll
+        for (int ks = 0; ks < 2 * NK; ++ks) lm_ldsm(qa + ks * 32, qf[ks][0], qf[ks][1], qf[ks][2], qf[ks][3]);
+    }
+    const float scale_log2 = a.scale * 1.4426950408889634f;
+    float o[NT][4];
+#pragma unroll
+    for (int d = 0; d < NT; ++d) o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.f;
+    float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
+
+    for (int it = 0; it < n_tiles; ++it) {
+        lm_wait<LD_STAGES - 2>();
+        __syncthreads();               // tile `it` is here, and everyone is done with the tile (and the scores) before it
+        load_tile(it + LD_STAGES - 1);
+        const bf16* tK = sK + (it % LD_STAGES) * LD_KEYS * LDS;
+        const int tile0 = first_tile + it * LD_KEYS;
+        // ---- S = Q K^T for this warp's eight keys
+        {
+            float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
+            const uint32_t ka = lm_addr(tK + (8 * warp + (lane & 7)) * LDS + (lane >> 3) * 8);
+#pragma unroll
+            for (int k2 = 0; k2 < NK; ++k2) {
+                uint32_t b0, b1, b2, b3;
+                lm_ldsm(ka + k2 * 64, b0, b1, b2, b3);
+                lm_mma(s0, qf[2 * k2][0], qf[2 * k2][1], qf[2 * k2][2], qf[2 * k2][3], b0, b1);
+                lm_mma(s1, qf[2 * k2 + 1][0], qf[2 * k2 + 1][1], qf[2 * k2 + 1][2], qf[2 * k2 + 1][3], b2, b3);
+            }
+            const int kcol = 8 * warp + 2 * qd, t = tile0 + kcol;
+            const bool ok0 = t >= t_lo && t <= p, ok1 = t + 1 >= t_lo && t + 1 <= p;
+#pragma unroll
+            for (int rr = 0; rr < 2; ++rr)
+                *reinterpret_cast<float2*>(sS + (g + 8 * rr) * SLD + kcol) =
+                    make_float2(ok0 ? (s0[2 * rr] + s1[2 * rr]) * scale_log2 : -INFINITY,
+                                ok1 ? (s0[2 * rr + 1] + s1[2 * rr + 1]) * scale_log2 : -INFINITY);
+        }
+        __syncthreads();
+        // ---- the whole tile's scores in the layout of the left operand of P C
+        float2 pz[4][4];   // [keys 16 kk ..][row g | row g + 8 | row g, keys + 8 | row g + 8, keys + 8]
+        float mx[2] = {m_run[0], m_run[1]};
+#pragma unroll
+        for (int kk = 0; kk < 4; ++kk)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                pz[kk][i] = *reinterpret_cast<const float2*>(sS + (g + 8 * (i & 1)) * SLD + kk * 16 + 8 * (i >> 1) + 2 * qd);
+                mx[i & 1] = fmaxf(mx[i & 1], fmaxf(pz[kk][i].x, pz[kk][i].y));
+            }
+        float alpha[2], m_ref[2];
+#pragma unroll
+        for (int rr = 0; rr < 2; ++rr) {
+            mx[rr] = fmaxf(mx[rr], __shfl_xor_sync(0xffffffffu, mx[rr], 1));
+            mx[rr] = fmaxf(mx[rr], __shfl_xor_sync(0xffffffffu, mx[rr], 2));
+            m_ref[rr] = mx[rr] == -INFINITY ? 0.f : mx[rr];
+            alpha[rr] = exp2f(m_run[rr] - m_ref[rr]);   // (0 in front of the first live key)
+            m_run[rr] = mx[rr];
+            l_run[rr] *= alpha[rr];
+        }
+        uint32_t pf[4][4];
+#pragma unroll
+        for (int kk = 0; kk < 4; ++kk)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const float e0 = exp2f(pz[kk][i].x - m_ref[i & 1]), e1 = exp2f(pz[kk][i].y - m_ref[i & 1]);
+                l_run[i & 1] += e0 + e1;   // this lane's share of the keys
+                pf[kk][i] = lm_pack(e0, e1);
+            }
+#pragma unroll
+        for (int d = 0; d < NT; ++d) {
+            o[d][0] *= alpha[0];
+            o[d][1] *= alpha[0];
+            o[d][2] *= alpha[1];
+            o[d][3] *= alpha[1];
+        }
+        // ---- O += P C over this warp's dimensions
+#pragma unroll
+        for (int kk = 0; kk < 4; ++kk) {
+            const uint32_t va = lm_addr(tK + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * LDS + warp * DW + (lane >> 4) * 8);
+#pragma unroll
+            for (int dp = 0; dp < DW / 16; ++dp) {
+                uint32_t b0, b1, b2, b3;
+                lm_ldsm_t(va + dp * 32, b0, b1, b2, b3);
+                lm_mma(o[2 * dp], pf[kk][0], pf[kk][1], pf[kk][2], pf[kk][3], b0, b1);
+                lm_mma(o[2 * dp + 1], pf[kk][0], pf[kk][1], pf[kk][2], pf[kk][3], b2, b3);
+            }
+        }
+    }
+    lm_wait<0>();   // (no copy is left in flight)
+    const size_t unit = (static_cast<size_t>(item) * gridDim.x + blockIdx.x) * a.n_ranges + blockIdx.z;
+#pragma unroll
+    for (int rr = 0; rr < 2; ++rr) {
+        const int r = g + 8 * rr, h = h0 + r;
+        float l = l_run[rr];
+        l += __shfl_xor_sync(0xffffffffu, l, 1);
+        l += __shfl_xor_sync(0xffffffffu, l, 2);
+        if (h >= a.H) continue;
+        if (a.n_ranges > 1) {
+            float* po = a.part_o + (unit * LD_HEADS + r) * KVR + warp * DW + 2 * qd;
+#pragma unroll
+            for (int d = 0; d < NT; ++d) *reinterpret_cast<float2*>(po + d * 8) = make_float2(o[d][2 * rr], o[d][2 * rr + 1]);
+            if (warp == 0 && qd == 0) *reinterpret_cast<float2*>(a.part_ml + (unit * LD_HEADS + r) * 2) = make_float2(m_run[rr], l);
+        } else {
+            // (a sink above every score: the sums are brought to its height, so that nothing overflows)
+            const float sk = a.sink ? a.sink[h] * 1.4426950408889634f : -INFINITY;
+            const float M = fmaxf(m_run[rr], sk), w = exp2f(m_run[rr] - M);
+            const float inv = w / (l * w + (a.sink ? exp2f(sk - M) : 0.f));
+            bf16* dst = a.out + (static_cast<size_t>(h) * a.T + row) * KVR + warp * DW + 2 * qd;
+#pragma unroll
+            for (int d = 0; d < NT; ++d)
+                *reinterpret_cast<uint32_t*>(dst + d * 8) = lm_pack(o[d][2 * rr] * inv, o[d][2 * rr + 1] * inv);
+        }
+    }
+}
+
+__global__ void __launch_bounds__(128) latent_decode_merge_kernel(LatentDecodeArgs a, int kvr) {
+    __shared__ float s_m[LD_MAX_RANGES], s_w[LD_MAX_RANGES], s_l[LD_MAX_RANGES];
+    pdl_entry();
+    pdl_trigger();
+    const int h = blockIdx.x, item = blockIdx.y, hb = h / LD_HEADS, r = h % LD_HEADS;
+    const int n_hb = (a.H + LD_HEADS - 1) / LD_HEADS;
+    const int seg = a.items[item];
+    int t_lo, first_tile, n_tiles, per_range;
+    ld_tiles(a.seg_ctx[seg], a.window, a.n_ranges, t_lo, first_tile, n_tiles, per_range);
+    const int live = (n_tiles + per_range - 1) / per_range;
+    const size_t unit0 = (static_cast<size_t>(item) * n_hb + hb) * a.n_ranges;
+    if (threadIdx.x < live) {
+        const float2 ml = *reinterpret_cast<const float2*>(a.part_ml + ((unit0 + threadIdx.x) * LD_HEADS + r) * 2);
+        s_m[threadIdx.x] = ml.x;
+        s_l[threadIdx.x] = ml.y;
+    }
+    __syncthreads();
+    float M = a.sink ? a.sink[h] * 1.4426950408889634f : -INFINITY;
+    const float sk = M;
+    for (int s = 0; s < live; ++s) M = fmaxf(M, s_m[s]);
+    if (threadIdx.x < live) s_w[threadIdx.x] = exp2f(s_m[threadIdx.x] - M);
+    __syncthreads();
+    float L = a.sink ? exp2f(sk - M) : 0.f;
+    for (int s = 0; s < live; ++s) L = fmaf(s_l[s], s_w[s], L);
+    const float inv = 1.0f / L;
+    bf16* dst = a.out + (static_cast<size_t>(h) * a.T + a.seg_q0[seg]) * kvr;
+    for (int d = threadIdx.x * 4; d < kvr; d += 512) {
+        float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+        for (int s = 0; s < live; ++s) {
+            const float4 v = __ldcg(reinterpret_cast<const float4*>(a.part_o + ((unit0 + s) * LD_HEADS + r) * kvr + d));
+            const float w = s_w[s];
+            acc.x = fmaf(v.x, w, acc.x);
+            acc.y = fmaf(v.y, w, acc.y);
+            acc.z = fmaf(v.z, w, acc.z);
+            acc.w = fmaf(v.w, w, acc.w);
+        }
+        *reinterpret_cast<uint2*>(dst + d) = make_uint2(lm_pack(acc.x * inv, acc.y * inv), lm_pack(acc.z * inv, acc.w * inv));
+    }
+}
+
+template <int KVR, int ROT>
+static int launch_latent_decode(const LatentDecodeArgs& a, int n_items, cudaStream_t stream) {
+    constexpr size_t smem = sizeof(bf16) * LD_STAGES * LD_KEYS * (KVR + ROT + 8) + sizeof(float) * LD_HEADS * (LD_KEYS + 4);
+    static bool set = false;
+    if (!set) {
+        if (cudaFuncSetAttribute(latent_decode_kernel<KVR, ROT>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)) != cudaSuccess)
+            return static_cast<int>(cudaGetLastError());
+        set = true;
+    }
+    const int n_hb = (a.H + LD_HEADS - 1) / LD_HEADS;
+    locus_launch(latent_decode_kernel<KVR, ROT>, dim3(n_hb, n_items, a.n_ranges), dim3(256), smem, stream, a);
+    if (a.n_ranges > 1) locus_launch(latent_decode_merge_kernel, dim3(a.H, n_items), dim3(128), 0, stream, a, KVR);
+    return locus_launch_status();
+}
+
+// bfloat16; kv_rank 128, 256, 384 or 512, rot_dim 0, 32 or 64.  items: [n_items] segments with exactly one new token.
+// n_ranges (1 to 64): ranges that every request's key tiles are cut into; with more than one, part_o holds n_items * head
+// blocks of 16 * n_ranges * 16 * kv_rank floats and part_ml n_items * head blocks * n_ranges * 32.
+extern "C" int locus_latent_decode(const void* q_abs, const void* q_rot, const void* pool, const float* sink, void* out,
+                                   const int* seg_q0, const int* seg_ctx, const int* block_table, int table_stride, const int* items,
+                                   int n_items, int T, int H, int kv_rank, int rot_dim, int page_tokens, int window, float scale,
+                                   int n_ranges, float* part_o, float* part_ml, cudaStream_t stream) {
+    if (n_items <= 0) return 0;
+    if (H <= 0 || page_tokens <= 0 || window < 0 || n_items > 65535 || n_ranges < 1 || n_ranges > LD_MAX_RANGES) return LOCUS_ERR_UNSUPPORTED;
+    if (n_ranges > 1 && (part_o == nullptr || part_ml == nullptr ||
+                         ((reinterpret_cast<uintptr_t>(part_o) | reinterpret_cast<uintptr_t>(part_ml)) & 15)))
+        return LOCUS_ERR_UNSUPPORTED;
+    if ((reinterpret_cast<uintptr_t>(q_abs) | reinterpret_cast<uintptr_t>(q_rot) | reinterpret_cast<uintptr_t>(pool) |
+         reinterpret_cast<uintptr_t>(out)) & 15)
+        return LOCUS_ERR_UNSUPPORTED;
+    LatentDecodeArgs a;
+    a.q_abs = static_cast<const bf16*>(q_abs); a.q_rot = static_cast<const bf16*>(q_rot); a.pool = static_cast<const bf16*>(pool);
+    a.sink = sink; a.out = static_cast<bf16*>(out); a.seg_q0 = seg_q0; a.seg_ctx = seg_ctx; a.block_table = block_table;
+    a.table_stride = table_stride; a.items = items; a.T = T; a.H = H; a.page_tokens = page_tokens; a.window = window;
+    a.n_ranges = n_ranges; a.scale = scale; a.part_o = part_o; a.part_ml = part_ml;
+#define LATENT_DECODE(RANK)                                                     \
+    do {                                                                        \
+        if (rot_dim == 0) return launch_latent_decode<RANK, 0>(a, n_items, stream);   \
+        if (rot_dim == 32) return launch_latent_decode<RANK, 32>(a, n_items, stream); \
+        if (rot_dim == 64) return launch_latent_decode<RANK, 64>(a, n_items, stream); \
+    } while (0)
+    if (kv_rank == 128) LATENT_DECODE(128);
+    if (kv_rank == 256) LATENT_DECODE(256);
+    if (kv_rank == 384) LATENT_DECODE(384);
+    if (kv_rank == 512) LATENT_DECODE(512);
+#undef LATENT_DECODE
     return LOCUS_ERR_UNSUPPORTED;
 }

@@ -1422,8 +1422,10 @@ def latent_attn(q_abs_hm: torch.Tensor, q_rot: torch.Tensor, pool: torch.Tensor,
 # Long portions: the heads' keys and values of a segment's whole context are expanded into plain rows and the portion runs on
 # the tcgen05 attention kernel.  A query-key pair then costs 2 x (key + value size) multiply-adds a head instead of 2 x 2 x rank
 # on the mma.sync kernel (sizes of 128 on a latent of 512: a quarter, on the faster pipe); the expansion costs as much as that
-# of two products per context row and is shared by the portion's queries.
-LATENT_EXPAND_FROM = 128         # new tokens of a segment from which on it is expanded
+# of two products per context row and is shared by the portion's queries.  Measured at 16 heads of 128 on a latent of 512, all
+# kernels between the queries and the output projection, over the latents / expanded: 2,048 tokens 561 / 55 us; 128 tokens
+# behind 0, 1,024 and 8,192 others 45 / 16, 77 / 34 and 307 / 91 us; 64 tokens over the latents 32, 54 and 157 us.
+LATENT_EXPAND_FROM = 64          # new tokens of a segment from which on it is expanded
 LATENT_EXPAND_ROWS = 16384       # most context rows of a step that are expanded ...
 LATENT_EXPAND_BYTES = 512 << 20  # ... and most bytes of their keys and values; segments beyond run over the latents
 
@@ -1530,6 +1532,71 @@ def latent_attn_mma(q_abs_hm: torch.Tensor, q_rot: torch.Tensor, pool: torch.Ten
     if n_splits > 1 and code == 0:
         _count_launches(1)
     _check(code, "latent_attn_mma", f"(heads {n_heads}, latent {kv_rank} + {rot_dim})")
+
+
+LATENT_DECODE_RANKS, LATENT_DECODE_ROTS = (128, 256, 384, 512), (0, 32, 64)
+LATENT_DECODE_HEADS, LATENT_DECODE_KEYS, LATENT_DECODE_MAX_RANGES = 16, 64, 64   # of a block; of a key tile
+
+
+def latent_decode_takes(dtype: torch.dtype, kv_rank: int, rot_dim: int) -> bool:
+    """Whether :func:`latent_decode` takes single tokens of this case; otherwise they run with the portions."""
+    return USE_TENSOR_CORES and dtype == torch.bfloat16 and kv_rank in LATENT_DECODE_RANKS and rot_dim in LATENT_DECODE_ROTS
+
+
+def latent_decode_ranges(n_items: int, n_heads: int, max_keys: int) -> int:
+    """Ranges every request's key tiles are cut into: a block takes one, a block per SM, so the cut with the least rounds x
+    (tiles of a range + what starting and merging one costs, in tiles), at most four blocks per SM (the scratch's size)."""
+    n_sm = _sm_count()
+    blocks = n_items * -(-n_heads // LATENT_DECODE_HEADS)
+    tiles = -(-max_keys // LATENT_DECODE_KEYS)
+    best, best_cost = 1, None
+    for n in range(1, min(LATENT_DECODE_MAX_RANGES, tiles, max(1, 4 * n_sm // blocks)) + 1):
+        cost = -(-blocks * n // n_sm) * (-(-tiles // n) + 2.0) + 0.05 * n
+        if best_cost is None or cost < best_cost - 1e-9:
+            best, best_cost = n, cost
+    return best
+
+
+def latent_decode_scratch(kv_rank: int) -> Tuple[int, int]:
+    """Floats of the two scratch buffers for any cut that :func:`latent_decode_ranges` chooses."""
+    units = 4 * _sm_count() * LATENT_DECODE_HEADS
+    return units * kv_rank, units * 2
+
+
+def latent_decode(q_abs_hm: torch.Tensor, q_rot: torch.Tensor, pool: torch.Tensor, sink: Optional[torch.Tensor],
+                  out_hm: torch.Tensor, *, seg_q0: torch.Tensor, seg_ctx: torch.Tensor, block_table: torch.Tensor,
+                  items: torch.Tensor, n_items: int, n_tokens: int, n_heads: int, kv_rank: int, rot_dim: int, page_tokens: int,
+                  window: int, scale: float, n_ranges: int = 1, part_o: Optional[torch.Tensor] = None,
+                  part_ml: Optional[torch.Tensor] = None) -> None:
+    """:func:`latent_attn` of single new tokens: ``items`` [n_items] lists segments with one new token; every cached row is
+    read once for sixteen heads.  ``n_ranges`` > 1 (:func:`latent_decode_ranges`) with scratch of
+    :func:`latent_decode_scratch` floats: the keys of every request are cut into that many ranges, merged in ascending order."""
+    _cuda_c(q_abs_hm, "q_abs_hm")
+    _cuda_c(q_rot, "q_rot")
+    _cuda_c(pool, "pool")
+    _cuda_c(out_hm, "out_hm")
+    _i32(block_table, "block_table")
+    _i32(items, "items")
+    T = n_tokens
+    _need(q_abs_hm.dtype == q_rot.dtype == pool.dtype == out_hm.dtype == torch.bfloat16, "latent_decode: bfloat16 only")
+    _need(q_abs_hm.shape[0] >= n_heads * T and q_abs_hm.shape[1] == kv_rank and out_hm.shape[0] >= n_heads * T
+          and out_hm.shape[1] == kv_rank and q_rot.shape[0] >= T and q_rot.shape[1] == n_heads * rot_dim, "latent_decode: shapes")
+    _need(pool.shape[-1] == kv_rank + rot_dim and pool.shape[-2] == page_tokens, "latent_decode: pool layout")
+    if sink is not None:
+        _need(sink.is_cuda and sink.dtype == torch.float32 and sink.numel() == n_heads and sink.is_contiguous(),
+              "latent_decode: sink must be float32 [H]")
+    if n_ranges > 1:
+        units = n_items * -(-n_heads // LATENT_DECODE_HEADS) * n_ranges * LATENT_DECODE_HEADS
+        _need(part_o is not None and part_ml is not None and part_o.is_cuda and part_ml.is_cuda
+              and part_o.dtype == part_ml.dtype == torch.float32 and part_o.numel() >= units * kv_rank and part_ml.numel() >= 2 * units,
+              "latent_decode: scratch too small for these ranges")
+    code = _lib("latent_attention").locus_latent_decode(
+        _p(q_abs_hm), _p(q_rot), _p(pool), _p(sink), _p(out_hm), _p(seg_q0), _p(seg_ctx), _p(block_table), I(block_table.shape[1]),
+        _p(items), I(n_items), I(T), I(n_heads), I(kv_rank), I(rot_dim), I(page_tokens), I(window), F(scale), I(n_ranges),
+        _p(part_o if n_ranges > 1 else None), _p(part_ml if n_ranges > 1 else None), _stream())
+    if n_ranges > 1 and code == 0:
+        _count_launches(1)
+    _check(code, "latent_decode", f"(heads {n_heads}, latent {kv_rank} + {rot_dim}, {n_ranges} key ranges)")
 
 
 def heads_to_rows(src_hm: torch.Tensor, out: torch.Tensor, *, n_tokens: int, n_heads: int) -> None:

@@ -41,73 +41,65 @@ from .base import Mixer, PagedKvSpec, PartSpec, StepPlan, TensorSource, make_par
 
 
 class LatentTiles(StepPlan):
-    """Work items of the latent attention kernels: tiles of ``tile`` queries over every segment, one token or
-    many, ordered by the position of their first query (the kernels walk the list from its end, so the tiles
-    with the most keys start first)."""
+    """Work items of the latent attention kernels, for every segment by its new tokens: tiles of ``tile`` queries
+    (``items``); with ``singles`` the segments with one new token go to a list of their own (``single_items``), which the
+    decode kernel takes; with ``max_rows`` > 0 the segments with at least ``expand_from`` new tokens, as long as the rows of
+    their contexts fit into ``max_rows`` together, go to tiles of 64 queries (``long_items``), with the segments, the first row
+    of each and the rows of all.  Tiles are ordered by the position of their first query (the kernels walk a list from its
+    end, so the tiles with the most keys start first)."""
 
-    def __init__(self, tile: int = K.LATENT_QUERY_TILE) -> None:
+    def __init__(self, tile: int = K.LATENT_QUERY_TILE, singles: bool = False, max_rows: int = 0, expand_from: int = 0) -> None:
         from ..cache import native
 
         self._lib = native.lib()
-        self.tile = int(tile)
-        self.key = ("latent_attention.tiles", self.tile)
+        self.tile, self.singles = int(tile), bool(singles)
+        self.max_rows, self.expand_from = int(max_rows), int(expand_from) if max_rows else 0
+        self.key = ("latent_attention.tiles", self.tile, self.singles, self.max_rows, self.expand_from)
 
     def capacity(self, max_tokens: int, max_segments: int) -> int:
-        return 2 * (max_tokens // self.tile + max_segments)
+        return 2 * (max_tokens // self.tile + max_tokens // K.MMA_QUERY_TILE + 2 * max_segments) + 3 * max_segments
 
-    def build(self, seg_q0, seg_qn, seg_ctx, out):
-        n = self._lib.locus_plan_query_tiles(len(seg_qn), seg_qn.ctypes.data, self.tile, 1,
-                                             out.ctypes.data, len(out))
+    def _tiles(self, seg_qn, tile, min_new, seg_ctx, out, at):
+        """Tiles of the segments with at least ``min_new`` new tokens, from ``out[at]`` on; their number."""
+        base = out.ctypes.data + 4 * at
+        n = self._lib.locus_plan_query_tiles(len(seg_qn), seg_qn.ctypes.data, tile, min_new, base, len(out) - at)
         if n < 0:
             raise ValueError("latent attention: the step has more query tiles than the plan's capacity holds")
-        self._lib.locus_sort_tiles_by_position(n, out.ctypes.data, seg_ctx.ctypes.data)
-        return {"items": (0, 2 * n, (-1, 2)), "n_items": n}
-
-
-class SplitTiles(StepPlan):
-    """Work items where long portions have their keys and values expanded: tiles of 64 queries over the segments with at least
-    ``expand_from`` new tokens (as long as the rows of their contexts fit into ``max_rows`` together), with the segments and
-    the first row of each; tiles of ``tile`` queries over all others.  Both ordered as in :class:`LatentTiles`."""
-
-    def __init__(self, tile: int, max_rows: int, expand_from: int) -> None:
-        from ..cache import native
-
-        self._lib = native.lib()
-        self.tile, self.max_rows, self.expand_from = int(tile), int(max_rows), int(expand_from)
-        self.key = ("latent_attention.split", self.tile, self.max_rows, self.expand_from)
-
-    def capacity(self, max_tokens: int, max_segments: int) -> int:
-        return 2 * (max_tokens // self.tile + max_tokens // K.MMA_QUERY_TILE + 2 * max_segments) + 2 * max_segments
+        self._lib.locus_sort_tiles_by_position(n, base, seg_ctx.ctypes.data)
+        return n
 
     def build(self, seg_q0, seg_qn, seg_ctx, out):
-        n_seg, ctx = len(seg_qn), seg_ctx.ctypes.data
-        rows, longest, long_segs = 0, 0, []
-        row0 = np.full(n_seg, -1, dtype=np.int32)
-        for s in np.nonzero(seg_qn >= self.expand_from)[0]:
-            n = int(seg_ctx[s]) + int(seg_qn[s])
-            if rows + n <= self.max_rows:
-                row0[s] = rows
-                rows += n
-                longest = max(longest, n)
-                long_segs.append(int(s))
-        is_long = row0 >= 0
-        # the segments of the other kind count as having no tokens (the helper lists none of them)
-        short = np.ascontiguousarray(np.where(is_long, 0, seg_qn), dtype=np.int32)
-        long = np.ascontiguousarray(np.where(is_long, seg_qn, 0), dtype=np.int32)
-        at, n = 0, []
-        for qn, tile in ((short, self.tile), (long, K.MMA_QUERY_TILE)):
-            base = out.ctypes.data + 4 * at
-            k = self._lib.locus_plan_query_tiles(n_seg, qn.ctypes.data, tile, 1, base, len(out) - at)
-            if k < 0:
-                raise ValueError("latent attention: the step has more query tiles than the plan's capacity holds")
-            self._lib.locus_sort_tiles_by_position(k, base, ctx)
-            n.append((at, k))
-            at += 2 * k
-        out[at:at + n_seg] = row0
-        out[at + n_seg:at + n_seg + len(long_segs)] = long_segs
-        return {"items": (n[0][0], 2 * n[0][1], (-1, 2)), "n_items": n[0][1], "long_items": (n[1][0], 2 * n[1][1], (-1, 2)),
-                "n_long_items": n[1][1], "row0": (at, n_seg, None), "long_segs": (at + n_seg, len(long_segs), None),
-                "n_long": len(long_segs), "n_rows": rows, "longest": longest}
+        n_seg, at, res = len(seg_qn), 0, {}
+        if self.singles:
+            n = self._lib.locus_plan_segments_with(n_seg, seg_qn.ctypes.data, 1, out.ctypes.data, len(out))
+            if n < 0:
+                raise ValueError("latent attention: the step has more segments than the plan's capacity holds")
+            res.update(single_items=(0, n, None), n_single_items=n)
+            at = n
+        long_segs = []
+        if self.max_rows:
+            rows, longest = 0, 0
+            row0 = np.full(n_seg, -1, dtype=np.int32)
+            for s in np.nonzero(seg_qn >= self.expand_from)[0]:
+                n = int(seg_ctx[s]) + int(seg_qn[s])
+                if rows + n <= self.max_rows:
+                    row0[s] = rows
+                    rows += n
+                    longest = max(longest, n)
+                    long_segs.append(int(s))
+            # a list is made of the segments of its kind: the others count as having no new tokens
+            long = np.ascontiguousarray(np.where(row0 >= 0, seg_qn, 0), dtype=np.int32)
+            seg_qn = np.ascontiguousarray(np.where(row0 >= 0, 0, seg_qn), dtype=np.int32)
+            n = self._tiles(long, K.MMA_QUERY_TILE, 1, seg_ctx, out, at)
+            res.update(long_items=(at, 2 * n, (-1, 2)), n_long_items=n, n_long=len(long_segs), n_rows=rows, longest=longest)
+            at += 2 * n
+            out[at:at + n_seg] = row0
+            out[at + n_seg:at + n_seg + len(long_segs)] = long_segs
+            res.update(row0=(at, n_seg, None), long_segs=(at + n_seg, len(long_segs), None))
+            at += n_seg + len(long_segs)
+        n = self._tiles(seg_qn, self.tile, 2 if self.singles else 1, seg_ctx, out, at)
+        res.update(items=(at, 2 * n, (-1, 2)), n_items=n)
+        return res
 
 
 class HeadTiles(StepPlan):
@@ -222,15 +214,16 @@ class LatentAttention(Mixer):
         return [self._query_tiles, self._head_tiles]
 
     @property
-    def _query_tiles(self) -> StepPlan:
+    def _query_tiles(self) -> LatentTiles:
         """Tiles of 16 queries for the CUDA-core kernel, or of 64 / (heads that share a block) for the tensor-core
-        kernel where it takes this mixer's sizes; where long portions are expanded, of the short segments alone."""
+        kernel where it takes this mixer's sizes; single tokens and long portions apart where their kernels do."""
         dtype = getattr(self, "_dtype", torch.float32)
         self._mma = K.latent_attn_mma_takes(dtype, self.kv_rank, self.dr)
         self._head_shift = K.latent_mma_head_shift(self.H)
         tile = 64 >> self._head_shift if self._mma else K.LATENT_QUERY_TILE
+        self._singles = K.latent_decode_takes(dtype, self.kv_rank, self.dr)
         self._max_rows = self._expand_rows(dtype)
-        return SplitTiles(tile, self._max_rows, K.LATENT_EXPAND_FROM) if self._max_rows else LatentTiles(tile)
+        return LatentTiles(tile, self._singles, self._max_rows, K.LATENT_EXPAND_FROM)
 
     @property
     def _head_tiles(self) -> HeadTiles:
@@ -277,7 +270,7 @@ class LatentAttention(Mixer):
         K.linear(cq if self.q_rank else h, self.params["w_uq"], q)
         o = rt.rows("latent.o", H * self.dv, rt.dtype, T)
         tiles = batch.plans[self._tiles_key]
-        if tiles["n_items"]:
+        if tiles["n_items"] or tiles.get("n_single_items"):
             self._attend_latents(q, o, tiles, batch, cache, gb, rt)
         if tiles.get("n_long_items"):
             self._attend_expanded(q, o, tiles, batch, cache, gb, rt)
@@ -325,13 +318,25 @@ class LatentAttention(Mixer):
         q_abs = rt.rows(f"latent.q_abs{self.kv_rank}", self.kv_rank, rt.dtype, H * T, per_token=H)
         K.linear(q_nope, self._w_uk_t, q_abs, layout=lay, n_rows=H * T, lists_ready=True)
         o_lat = rt.rows(f"latent.o_lat{self.kv_rank}", self.kv_rank, rt.dtype, H * T, per_token=H)
+        # the most keys a query of this step sees (all that the block table can describe when the step's launches must not
+        # depend on its lengths)
+        keys = gb.block_table.shape[1] * gb.page_tokens if batch.static_shapes else max(batch.longest, 1)
+        n1 = tiles.get("n_single_items", 0)
+        if n1:
+            n_ranges = K.latent_decode_ranges(n1, H, min(keys, self.window) if self.window > 0 else keys)
+            scratch = {}
+            if n_ranges > 1:
+                n_o, n_ml = K.latent_decode_scratch(self.kv_rank)
+                scratch = dict(part_o=rt.buf("latent.decode_part_o", (n_o,), torch.float32), part_ml=rt.buf("latent.decode_part_ml", (n_ml,), torch.float32))
+            K.latent_decode(q_abs, q_rot, cache.pool, self._sink, o_lat, seg_q0=batch.seg_q0, seg_ctx=batch.seg_ctx,
+                            block_table=gb.block_table, items=tiles["single_items"], n_items=n1, n_tokens=T, n_heads=H, kv_rank=self.kv_rank,
+                            rot_dim=self.dr, page_tokens=gb.page_tokens, window=self.window, scale=self.scale, n_ranges=n_ranges, **scratch)
         common = dict(seg_q0=batch.seg_q0, seg_qn=batch.seg_qn, seg_ctx=batch.seg_ctx, block_table=gb.block_table,
                       items=tiles["items"], n_items=tiles["n_items"], n_tokens=T, n_heads=H, kv_rank=self.kv_rank,
                       rot_dim=self.dr, page_tokens=gb.page_tokens, window=self.window, scale=self.scale)
-        if self._mma:
-            # the most keys a query of this step sees (all that the block table can describe when the step's
-            # launches must not depend on its lengths)
-            keys = gb.block_table.shape[1] * gb.page_tokens if batch.static_shapes else max(batch.longest, 1)
+        if not tiles["n_items"]:
+            pass
+        elif self._mma:
             if self.window > 0:
                 keys = min(keys, self.window + (64 >> self._head_shift))
             n_splits = K.latent_attn_mma_splits(tiles["n_items"], H, self._head_shift, keys)

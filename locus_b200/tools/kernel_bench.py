@@ -457,17 +457,28 @@ def bench_latent(args) -> None:
         n_o, n_ml = K.latent_attn_mma_scratch(r)
         extra = dict(n_splits=n_splits, part_o=torch.empty(n_o, device=dev), part_ml=torch.empty(n_ml, device=dev)) if n_splits > 1 else {}
         pos, fl = torch.zeros(T, dtype=torch.int32, device=dev), 2.0 * T * H * D * r
-        steps = [("latent_q_split", lambda: K.latent_q_split(q, pos, None, 1.0, q_hm, q_rot, n_heads=H, nope_dim=D, rot_dim=0, rot_pairs=0), 0, 4.0 * T * H * D),
-                 ("product into the latent space", lambda: K.linear(q_hm, w_uk_t, q_abs, layout=lay, n_rows=H * T, lists_ready=True), fl, w_uk_t.numel() * 2.0),
-                 (f"latent_attn_mma ({n_splits} key ranges)",
+        attend = (f"latent_attn_mma ({n_splits} key ranges)",
                   lambda: K.latent_attn_mma(q_abs, q_rot, pool(), None, o_lat, head_shift=shift, items=items, n_items=len(items), n_tokens=T, n_heads=H,
                                             kv_rank=r, rot_dim=0, page_tokens=P, window=0, scale=D ** -0.5, block_table=table, **meta, **extra),
-                  4.0 * keys * H * r, 2.0 * B * total * r),
+                  4.0 * keys * H * r, 2.0 * B * total * r)
+        if n == 1 and K.latent_decode_takes(dt, r, 0) and not args.absorbed:
+            one, n_ranges = i32(list(range(B))), args.key_ranges if args.key_ranges > 0 else K.latent_decode_ranges(B, H, total)
+            n_o, n_ml = K.latent_decode_scratch(r)
+            scratch = dict(part_o=torch.empty(n_o, device=dev), part_ml=torch.empty(n_ml, device=dev))
+            attend = (f"latent_decode ({n_ranges} key ranges)",
+                      lambda: K.latent_decode(q_abs, q_rot, pool(), None, o_lat, items=one, n_items=B, n_tokens=T, n_heads=H, kv_rank=r, rot_dim=0,
+                                              page_tokens=P, window=0, scale=D ** -0.5, block_table=table, seg_q0=meta["seg_q0"],
+                                              seg_ctx=meta["seg_ctx"], n_ranges=n_ranges, **scratch), 4.0 * keys * H * r, 2.0 * B * total * r)
+        steps = [("latent_q_split", lambda: K.latent_q_split(q, pos, None, 1.0, q_hm, q_rot, n_heads=H, nope_dim=D, rot_dim=0, rot_pairs=0), 0, 4.0 * T * H * D),
+                 ("product into the latent space", lambda: K.linear(q_hm, w_uk_t, q_abs, layout=lay, n_rows=H * T, lists_ready=True), fl, w_uk_t.numel() * 2.0),
+                 attend,
                  ("product out of the latent space", lambda: K.linear(o_lat, w_uv, o_hm, layout=lay, n_rows=H * T, lists_ready=True), fl, w_uv.numel() * 2.0),
                  ("heads_to_rows", lambda: K.heads_to_rows(o_hm, o, n_tokens=T, n_heads=H), 0, 4.0 * T * H * D)]
 
+    parts = [fn for _, fn, _, _ in steps]
+
     def all_of_it():
-        for _, fn, _, _ in steps:
+        for fn in parts:
             fn()
     steps.append(("all", all_of_it, 4.0 * keys * H * D, 2.0 * B * total * r))
     for name, fn, fl, by in steps:
@@ -544,7 +555,7 @@ def main(argv=None) -> int:
                     help="linear: with --token-tile, parts along K (0 = not split)")
     ap.add_argument("--cuda-cores", action="store_true", help="attn_chunk: the CUDA-core kernel")
     ap.add_argument("--key-ranges", type=int, default=-1,
-                    help="attn_chunk, tensor-core kernels: ranges the keys are cut into (default: the engine's choice)")
+                    help="attn_chunk, latent, tensor-core kernels: ranges the keys are cut into (default: the engine's choice)")
     ap.add_argument("--mma-sync", action="store_true", help="attn_chunk: the mma.sync kernel where tcgen05 would run")
     args = ap.parse_args(argv)
     if args.skinny_rows >= 0:

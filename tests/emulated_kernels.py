@@ -494,6 +494,22 @@ def latent_attn(q_abs_hm, q_rot, pool, sink, out_hm, *, seg_q0, seg_qn, seg_ctx,
                 out_hm[h * T + q0 + i] = ((e / den) @ rows[:, :kv_rank]).to(out_hm.dtype)
 
 
+def latent_decode_takes(dtype, kv_rank, rot_dim):
+    return False
+
+
+def latent_decode_ranges(n_items, n_heads, max_keys):
+    return 1
+
+
+def latent_decode(q_abs_hm, q_rot, pool, sink, out_hm, *, seg_q0, seg_ctx, block_table, items, n_items, n_tokens, n_heads, kv_rank,
+                  rot_dim, page_tokens, window, scale, n_ranges=1, part_o=None, part_ml=None):
+    pairs = torch.stack([items[:n_items], torch.zeros_like(items[:n_items])], 1)
+    latent_attn(q_abs_hm, q_rot, pool, sink, out_hm, seg_q0=seg_q0, seg_qn=torch.ones_like(seg_ctx), seg_ctx=seg_ctx, block_table=block_table,
+                items=pairs, n_items=n_items, n_tokens=n_tokens, n_heads=n_heads, kv_rank=kv_rank, rot_dim=rot_dim, page_tokens=page_tokens,
+                window=window, scale=scale)
+
+
 def latent_gather(pool, out, *, segs, n_segs, row0, seg_qn, seg_ctx, block_table, page_tokens, longest):
     for i in range(n_segs):
         s = int(segs[i])
@@ -832,7 +848,7 @@ def head_tile(n_tokens, dtype, widths_ok):
 
 
 _NAMES = ["embed_rows", "rmsnorm", "rmsnorm_adds", "attn_chunk_tc_takes", "linear", "rope_kv_write", "attn_chunk", "attn_chunk_mma", "attn_decode", "router_topk", "router_logits", "router_select",
-          "moe_sort", "route_small", "route_small_takes", "route_fused_small", "moe_combine", "gather_rows", "add_rows", "latent_gather", "attn_chunk_tc_splits", "attn_chunk_tc_rows", "apply_penalties", "sample",
+          "moe_sort", "route_small", "route_small_takes", "route_fused_small", "moe_combine", "gather_rows", "add_rows", "latent_gather", "latent_decode", "latent_decode_takes", "latent_decode_ranges", "attn_chunk_tc_splits", "attn_chunk_tc_rows", "apply_penalties", "sample",
           "cast_rows", "rmsnorm_add", "latent_prep", "latent_q_split", "latent_attn", "heads_to_rows", "retention_scan",
           "retention_gate_norm", "head_tile", "latent_attn_mma_takes", "layernorm", "stream_update", "moe_identity",
           "gated_recurrence", "mlstm_gates", "mlstm_out", "ssm_conv", "ssm_out", "head_prep", "gate_rows", "delta_rule", "delta_out",

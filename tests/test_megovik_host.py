@@ -280,18 +280,21 @@ def test_long_portions_with_expanded_keys_and_values(tmp_path, monkeypatch):
     import locus_b200.kernels as K
 
     monkeypatch.setattr(K, "LATENT_EXPAND_FROM", 8)
+    monkeypatch.setattr(K, "latent_decode_takes", lambda dtype, rank, rot: rank == 32)   # (single tokens apart in the first layer)
     monkeypatch.setattr(K, "latent_expand_rows", lambda dtype, H, dn, dr, dv, rank: 90 if dn == dv else 0)
     raw = model(48, 50, [with_mlp(latent(4, 16, 16, 32), dense(24)), with_mlp(latent(2, 24, 24, 24, q_rank=16), None)])
     case = Case("expanded", tmp_path, torch.float32, raw=raw, requests=(60, 40, 30, 70))
     runner, cache = make_runner(case, torch.float32, "cpu", page_tokens=8, n_pages=30, max_tokens=160, slots=4)
     calls, rows = [], K.attn_chunk_tc_rows
+    singles, decode = [], K.latent_decode
+    monkeypatch.setattr(K, "latent_decode", lambda *a, **kw: (singles.append(kw["items"].tolist()), decode(*a, **kw)))
     monkeypatch.setattr(K, "attn_chunk_tc_rows", lambda *a, **kw: (calls.append(sorted({int(s) for s, _ in kw["items"].tolist()})), rows(*a, **kw)))
-    steps = [[("r0", 20), ("r1", 2)], [("r0", 10), ("r1", 20), ("r2", 1)], [("r0", 30), ("r1", 18), ("r2", 28), ("r3", 50)], [("r2", 1), ("r3", 20)]]
+    steps = [[("r0", 20), ("r1", 2)], [("r0", 10), ("r1", 20), ("r2", 1)], [("r0", 30), ("r1", 18), ("r2", 28), ("r3", 50)], [("r2", 1), ("r3", 18)], [("r3", 1)], [("r3", 1)]]
     got, routed = run_steps(runner, cache, case, steps)
     compare(case, got, routed, *TOL, TIE)
     # (third step: 60 rows, 40 that do not fit, 29, 50 that do not)
     assert calls == [[0]] * 2 + [[0, 1]] * 2 + [[0, 2]] * 2 + [[1]] * 2
-    assert {pl.key[0] for pl in runner.plans.values()} == {"latent_attention.split", "latent_attention.head_tiles"}
+    assert singles == [[2], [0], [0], [0]]
 
 
 def test_pages_and_slots_are_used_again_under_a_small_pool(tmp_path):
