@@ -428,19 +428,19 @@ attn_chunk_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
             const bool need_mask = tile_first + AT_MK - 1 > p0 || tile_first < lo_last;
             float mx = -INFINITY;
             if constexpr (BIAS) {
-                // s <- s scale - slope (pq - t), two keys at a time (t - pq is an exact float32)
+                // s <- s scale + slope (t - pq), two keys at a time: the tile's first key's share (t - pq is an exact float32),
+                // then a multiple of the slope per key
                 const unsigned long long k2 = at_pair(scale_log2, scale_log2), sl2 = at_pair(slope, slope);
-                const float d0 = static_cast<float>(tile0 - pq);
-                const unsigned long long d2 = at_pair(d0, d0);
+                const float d0 = slope * static_cast<float>(tile0 - pq), d1 = slope * static_cast<float>(tile0 + 32 - pq);
+                const unsigned long long b0 = at_pair(d0, d0), b1 = at_pair(d1, d1);
 #pragma unroll
                 for (int i = 0; i < 32; i += 2) {
                     float x, y;
-                    const unsigned long long off0 = at_mul2(sl2, at_add2(d2, at_pair(static_cast<float>(i), static_cast<float>(i + 1))));
-                    at_unpair(at_fma2(at_pair(__uint_as_float(s0[i]), __uint_as_float(s0[i + 1])), k2, off0), x, y);
+                    const unsigned long long at2 = at_pair(static_cast<float>(i), static_cast<float>(i + 1));
+                    at_unpair(at_fma2(at_pair(__uint_as_float(s0[i]), __uint_as_float(s0[i + 1])), k2, at_fma2(sl2, at2, b0)), x, y);
                     s0[i] = __float_as_uint(x);
                     s0[i + 1] = __float_as_uint(y);
-                    const unsigned long long off1 = at_mul2(sl2, at_add2(d2, at_pair(static_cast<float>(i + 32), static_cast<float>(i + 33))));
-                    at_unpair(at_fma2(at_pair(__uint_as_float(s1[i]), __uint_as_float(s1[i + 1])), k2, off1), x, y);
+                    at_unpair(at_fma2(at_pair(__uint_as_float(s1[i]), __uint_as_float(s1[i + 1])), k2, at_fma2(sl2, at2, b1)), x, y);
                     s1[i] = __float_as_uint(x);
                     s1[i + 1] = __float_as_uint(y);
                 }
