@@ -11,7 +11,7 @@ query/key dimensions, values of ``v_dim``):
     score(t, j, head) = (q_nope . (W_uk c_j) + rot(q_rot) . rot(k_r_j)) * scale,   value_j = W_uv c_j
 
 Only c and rot(k_r) are cached: a row of kv_rank + rot_dim elements per token.  The heads' keys and values
-are never expanded per key: W_uk is applied to the query instead (q_abs = W_uk^T q_nope), attention runs over
+are not expanded per key: W_uk is applied to the query instead (q_abs = W_uk^T q_nope), attention runs over
 the cached rows as they are, and W_uv is applied to the attention's output (sum_j p_j c_j).  The two per-head
 products are grouped products (the heads in the place of experts) over head-major rows [head][token].
 
